@@ -7,7 +7,8 @@ from .dafolorn import DafolornConfig
 from .zeluzen import ZeluzenConfig
 from .benarax import BenaraxConfig
 from .radalix import RadalixConfig
+from .vononex import VononexConfig
 
 __all__ = ["LayerSpec", "ModelPlan", "PartSpec", "ScheduleEntry", "SubPart", "default_schedule", "prenorm_layer", "ConfigError",
            "config_from_dict", "load_config", "register_architecture", "registered_architectures",
-           "resolve_architecture", "Qwen2Config", "DafolornConfig", "ZeluzenConfig", "BenaraxConfig", "RadalixConfig"]
+           "resolve_architecture", "Qwen2Config", "DafolornConfig", "ZeluzenConfig", "BenaraxConfig", "RadalixConfig", "VononexConfig"]

@@ -19,6 +19,12 @@ and reads the keys and values another layer's cache holds (`own_kv` False), a sh
 every channel of q, k and v right behind the projection (`conv_taps`; the last taps - 1 projected rows are the
 request's state), a query multiplier 1 + coef ln(floor((p + 1) / every) + 1) at position p (`q_temp`), a gate
 sigmoid(W_g h) on the heads' outputs in front of the output projection (`gate`), and other tensor names (`names`).
+
+Three more go through one kernel of their own (`ctx.kernels.row_norm_rope_append`), together with biases: a norm of the
+query rows and of the key rows as a whole, all heads together, in front of the rotation, with a weight per element
+(`qk_norm` with `over: "row"`); a learned factor per head on the scores (`head_temp`, multiplied into the queries); and values
+that are turned by their own position over their whole head (`value_position`), cached so, with each head's output turned
+back by the query's position.  A bias on the output projection (`o_bias`) travels with the unadded output.
 """
 from __future__ import annotations
 
@@ -27,7 +33,7 @@ import math
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import KVCacheSpec, Mixer, StateSpec, WeightBuffers, build_part, register_part
+from .base import KVCacheSpec, Mixer, StateSpec, WeightBuffers, WeightedSum, build_part, register_part
 
 
 def materialized_rows(kernels, h):
@@ -42,12 +48,14 @@ class Attention(Mixer):
     position (a PartSpec of role `position`, or None), qkv_bias (True, False or
     "if_present"), invent_bias (with "if_present": whether random-weights mode makes
     the biases up; default True), scale (None for 1/sqrt(head_dim)), v_head_dim (None: head_dim),
-    qk_norm (None, or {eps}), chunk (None or int), sink (bool, or "learned": a tensor [heads]), own_kv (default True),
+    qk_norm (None, or {eps, over: "head" (default) or "row"}), chunk (None or int), sink (bool, or "learned": a tensor [heads]), own_kv (default True),
     conv_taps (None or int), q_temp (None, or {coef, every}), gate (None or "sigmoid"),
-    names (tensor names of q, k, v, o, q_bias, k_bias, v_bias, q_norm, k_norm, sink, gate, q_conv, k_conv, v_conv)."""
+    head_temp (bool), value_position (a PartSpec of role `position` that turns whole value heads, or None), o_bias (bool),
+    names (tensor names of q, k, v, o, q_bias, k_bias, v_bias, o_bias, q_norm, k_norm, sink, gate, temp, q_conv, k_conv,
+    v_conv)."""
 
     _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
-              "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
+              "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias", "temp": "temp",
               "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sink", "gate": "gate_proj.weight",
               "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight"}
 
@@ -68,8 +76,14 @@ class Attention(Mixer):
         self.nkv = int(p["num_kv_heads"])
         self.d = int(p["head_dim"])
         self.dv = int(p["v_head_dim"]) if p.get("v_head_dim") is not None else self.d
+        self.row_norm = bool(p.get("qk_norm")) and p["qk_norm"].get("over", "head") == "row"
+        self.head_temp = bool(p.get("head_temp", False))
+        self.o_bias = bool(p.get("o_bias", False))
+        vpos = p.get("value_position")
+        self.value_position = build_part("position", vpos) if vpos is not None else None
+        self.by_rows = self.row_norm or self.head_temp or self.value_position is not None      # row_norm_rope_append's options
         self.general = (any(p.get(k) for k in ("qk_norm", "chunk", "sink", "conv_taps", "q_temp", "gate"))
-                        or self.dv != self.d or not p.get("own_kv", True))
+                        or self.dv != self.d or not p.get("own_kv", True) or self.by_rows or self.o_bias)
         if self.general:                   # the general kernels take any even size up to 256
             for size in (self.d, self.dv):
                 if size <= 0 or size % 2 or size > 256:
@@ -103,12 +117,16 @@ class Attention(Mixer):
             raise ValueError(f"attention: unknown gate {self.gate!r} (known: sigmoid)")
         if self.general and self.qkv_bias == "if_present":
             self.qkv_bias = False
-        if self.general and self.qkv_bias:
+        if self.general and self.qkv_bias and not self.by_rows:
             raise ValueError("attention: biases together with head norms, chunks, a sink or a shared cache are not built")
+        if self.by_rows and (not self.own_kv or self.taps is not None or self.q_temp is not None
+                             or (self.qk_norm_eps is not None and not self.row_norm)):
+            raise ValueError("attention: a norm over rows, a factor per head or turned values beside a shared cache, a "
+                             "convolution, a query multiplier or a norm per head are not built")
         self.names = dict(self._NAMES)
         self.names.update(p.get("names") or {})
         self.w_qkv = self.b_qkv = self.w_o = self.q_norm_w = self.k_norm_w = None
-        self.sink_values = self.w_gate = self.w_conv = None
+        self.sink_values = self.w_gate = self.w_conv = self.temp = self.b_o = None
 
     # ---------------------------------------------------------------- declarations
     def cache_spec(self):
@@ -146,9 +164,13 @@ class Attention(Mixer):
             for side, size in (("q", q), ("k", k), ("v", v)):
                 specs[n[side + "_bias"]] = TensorSpec((size,), optional=optional, invent=self.invent_bias)
         if self.qk_norm_eps is not None:
-            specs[n["q_norm"]] = TensorSpec((self.d,), init="ones")
+            specs[n["q_norm"]] = TensorSpec((q if self.row_norm else self.d,), init="ones")
             if self.own_kv:
-                specs[n["k_norm"]] = TensorSpec((self.d,), init="ones")
+                specs[n["k_norm"]] = TensorSpec((k if self.row_norm else self.d,), init="ones")
+        if self.head_temp:
+            specs[n["temp"]] = TensorSpec((self.nq,), init="ones")
+        if self.o_bias:
+            specs[n["o_bias"]] = TensorSpec((self.hidden,))
         if self.learned_sink:
             specs[n["sink"]] = TensorSpec((self.nq,))
         if self.gate is not None:
@@ -158,17 +180,28 @@ class Attention(Mixer):
                 specs[n[side + "_conv"]] = TensorSpec((size, self.taps))
         return specs
 
-    def load(self, tensors, dtype, device):
+    def projection_rows(self) -> int:
+        """Rows of the stacked projection, for a mixer that stacks it with another one's."""
+        return sum(self._sizes())
+
+    def load(self, tensors, dtype, device, projection=None):
+        """`projection`: room for the stacked projection that somebody else owns (see `projection_rows`)."""
         n = self.names
         q, k, v = self._sizes()
         sides = [("q", q)] + ([("k", k), ("v", v)] if self.own_kv else [])
         has_bias = any(n[side + "_bias"] in tensors for side, _ in sides)
-        layout = {"w_qkv": ((q + k + v, self.hidden), dtype), "w_o": ((self.hidden, self.nq * self.dv), dtype)}
+        layout = {"w_o": ((self.hidden, self.nq * self.dv), dtype)}
+        if projection is None:
+            layout["w_qkv"] = ((q + k + v, self.hidden), dtype)
         if has_bias:
             layout["b_qkv"] = ((q + k + v,), torch.float32)               # added in float32
         if self.qk_norm_eps is not None:
-            layout["q_norm"] = ((self.d,), torch.float32)
-            layout["k_norm"] = ((self.d,), torch.float32)
+            layout["q_norm"] = ((q if self.row_norm else self.d,), torch.float32)
+            layout["k_norm"] = ((k if self.row_norm else self.d,), torch.float32)
+        if self.head_temp:
+            layout["temp"] = ((self.nq,), torch.float32)
+        if self.o_bias:
+            layout["b_o"] = ((self.hidden,), torch.float32)
         if self.learned_sink:
             layout["sink"] = ((self.nq,), torch.float32)
         if self.gate is not None:
@@ -176,6 +209,12 @@ class Attention(Mixer):
         if self.taps is not None:
             layout["w_conv"] = ((q + k + v, self.taps), torch.float32)
         self.buffers = buf = WeightBuffers(device, layout)
+        if self.head_temp:
+            buf["temp"].copy_(tensors[n["temp"]])
+            self.temp = buf["temp"]
+        if self.o_bias:
+            buf["b_o"].copy_(tensors[n["o_bias"]])
+            self.b_o = buf["b_o"]
         if self.learned_sink:
             buf["sink"].copy_(tensors[n["sink"]])
             self.sink_values = buf["sink"]
@@ -188,9 +227,10 @@ class Attention(Mixer):
                 buf["w_conv"][at:at + size].copy_(tensors[n[side + "_conv"]])
                 at += size
             self.w_conv = buf["w_conv"]
+        w_qkv = buf["w_qkv"] if projection is None else projection
         at = 0
         for side, size in sides:                                          # each projection into its rows of the stack
-            buf["w_qkv"][at:at + size].copy_(tensors[n[side]])
+            w_qkv[at:at + size].copy_(tensors[n[side]])
             if has_bias:
                 b = tensors.get(n[side + "_bias"])
                 if b is None:
@@ -199,7 +239,7 @@ class Attention(Mixer):
                     buf["b_qkv"][at:at + size].copy_(b)
             at += size
         buf["w_o"].copy_(tensors[n["o"]])
-        self.w_qkv, self.w_o = buf["w_qkv"], buf["w_o"]
+        self.w_qkv, self.w_o = w_qkv, buf["w_o"]
         self.b_qkv = buf["b_qkv"] if has_bias else None
         if self.qk_norm_eps is not None:
             buf["q_norm"].copy_(tensors[n["q_norm"]])
@@ -214,8 +254,11 @@ class Attention(Mixer):
         return make(ctx) if make is not None else {}
 
     # --------------------------------------------------------------------- forward
-    def forward(self, h, ctx, cache):
+    def forward(self, h, ctx, cache, projected=None):
+        """`projected` = (rows, first column): the stacked projection's result, when somebody else made it."""
         k = ctx.kernels
+        if self.by_rows:
+            return self._forward_by_rows(h, ctx, cache, projected)
         qkv = k.linear(h, self.w_qkv, allow_partial=True)                    # [T, (nq + 2 nkv) d], maybe in K slices
         rotary = self.position.rotary(ctx.device) if self.position is not None else None
         if not self.general:
@@ -236,4 +279,22 @@ class Attention(Mixer):
                         sink=self.sink_values if self.learned_sink else self.sink, dv=self.dv)   # [T, nq dv]
         if self.gate is not None:
             a = k.gate_mul(a, k.linear(materialized_rows(k, h), self.w_gate), self.gate)
-        return k.linear(a, self.w_o, allow_partial=True)
+        return self._output(k, a)
+
+    def _output(self, k, a):
+        y = k.linear(a, self.w_o, allow_partial=True)
+        return y if self.b_o is None else WeightedSum([(1.0, y, self.b_o)])
+
+    def _forward_by_rows(self, h, ctx, cache, projected):
+        k = ctx.kernels
+        rows, col0 = (k.linear(h, self.w_qkv, allow_partial=True), 0) if projected is None else projected
+        rotary = self.position.rotary(ctx.device) if self.position is not None else None
+        turn = self.value_position.rotary(ctx.device) if self.value_position is not None else None
+        # the queries, and what turns the values' sum back: (cos, sin) of every token's angles
+        q, back = k.row_norm_rope_append(rows, col0, self.b_qkv, rotary, turn, self.temp, self.nq, self.nkv, self.d, self.dv,
+                                         ctx, cache, q_norm=self.q_norm_w, k_norm=self.k_norm_w, norm_eps=self.qk_norm_eps or 0.0)
+        a = k.attention(q, self.nq, self.nkv, self.d, self.window, self.scale, ctx, cache, chunk=self.chunk,
+                        sink=self.sink_values if self.learned_sink else self.sink, dv=self.dv, turn_back=back)   # [T, nq dv]
+        if self.gate is not None:
+            a = k.gate_mul(a, k.linear(materialized_rows(k, h), self.w_gate), self.gate)
+        return self._output(k, a)

@@ -79,11 +79,47 @@ class VectorScaledDelta:
         ctx.kernels.residual_add_vectors(x, self.a, self.s_a, self.b, self.s_b, self.b2)
 
 
+class WeightedSum:
+    """A sublayer's output as up to two terms c * (y + bias): y a tensor or a PartialSum, c a number, bias a float32 vector
+    along the row or None.  The kernel that adds it to the stream does all of it in the same pass."""
+
+    def __init__(self, terms):
+        self.terms = [(float(c), y, bias) for c, y, bias in terms]
+        if not 1 <= len(self.terms) <= 2:
+            raise ValueError(f"a weighted sum of {len(self.terms)} terms (one or two are built)")
+
+    @classmethod
+    def of(cls, y) -> "WeightedSum":
+        return y if isinstance(y, cls) else cls([(1.0, y, None)])
+
+    def scaled(self, factor: float):
+        return [(factor * c, y, bias) for c, y, bias in self.terms]
+
+    def add_to(self, x: torch.Tensor, ctx) -> None:
+        ctx.kernels.norm_of_sum(x, 1.0, self.terms, None, 0.0)
+
+
+class NormOfSum:
+    """A sublayer's output whose sum with the stream is normed as a whole: x becomes the RMS norm of alpha x + output, times
+    a weight.  A block hands it on as `pending`; `add_to` replaces x, and with `out_dtype` also returns the new rows in
+    that dtype for a sublayer that reads them."""
+
+    def __init__(self, y, alpha: float, weight: torch.Tensor, eps: float):
+        self.sum, self.alpha, self.weight, self.eps = WeightedSum.of(y), float(alpha), weight, float(eps)
+
+    def add_to(self, x: torch.Tensor, ctx, out_dtype=None):
+        return ctx.kernels.norm_of_sum(x, self.alpha, self.sum.terms, self.weight, self.eps, out_dtype=out_dtype)
+
+
+# deltas that join the stream through a kernel of their own, unlike plain tensors and PartialSums
+UNADDED = (NormedDelta, VectorScaledDelta, WeightedSum, NormOfSum)
+
+
 def settle_pending(x: torch.Tensor, pending, ctx) -> None:
-    """x += pending, whatever kind of delta it is."""
+    """x += pending (or what else the kind of delta does to x)."""
     if pending is None:
         return
-    if isinstance(pending, (NormedDelta, VectorScaledDelta)):
+    if isinstance(pending, UNADDED):
         pending.add_to(x, ctx)
     else:
         ctx.kernels.residual_add(x, pending)

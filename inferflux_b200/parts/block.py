@@ -10,7 +10,7 @@ from typing import Optional
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import Block, NormedDelta, StateSpec, StreamMerge, VectorScaledDelta, register_part, settle_pending
+from .base import UNADDED, Block, NormedDelta, NormOfSum, StateSpec, StreamMerge, VectorScaledDelta, register_part, settle_pending
 from .norm import RMSNorm
 
 
@@ -19,7 +19,7 @@ class PreNormBlock(Block):
     sub_parts = {"norm_mixer": "norm", "mixer": "mixer", "norm_ffn": "norm", "ffn": "ffn"}
 
     def forward(self, x, pending, ctx, cache):
-        if isinstance(pending, NormedDelta):                         # the layer before norms its output itself
+        if isinstance(pending, UNADDED):                             # the layer before norms or scales its output itself
             pending.add_to(x, ctx)
             pending = None
         fused = getattr(ctx.kernels, "fused_prenorm_layer", None)    # a kernel table may run the whole layer itself
@@ -293,10 +293,51 @@ class ParallelNormsBlock(Block):
 
 def _settled(x, pending, ctx):
     """What is left to add inside the next norm kernel: a plain delta is; one with a norm or vectors of its own is added here."""
-    if isinstance(pending, (NormedDelta, VectorScaledDelta)):
+    if isinstance(pending, UNADDED):
         pending.add_to(x, ctx)
         return None
     return pending
+
+
+@register_part("block", "norm_of_sum")
+class NormOfSumBlock(Block):
+    """The norm behind the sum; the sublayers read the residual stream itself:
+
+        x = norm_m(alpha x + mixer(x));   x = norm_f(alpha x + ffn(x))
+
+    params: alpha, ffn (False: the layer ends after the mixer).  Parts: mixer, norm_mixer and, with a feed-forward, ffn,
+    norm_ffn.  A sublayer's output (K slices, biases, a pair's two outputs with their weights) travels unadded with its norm
+    (`NormOfSum`); the sum, the norm and the rounding of x to the run's dtype for the next sublayer are one kernel."""
+
+    def __init__(self, spec, parts):
+        self.has_ffn = bool(spec.params.get("ffn", True))
+        self.alpha = float(spec.params.get("alpha", 1.0))
+        names = {"mixer": "mixer", "norm_mixer": "norm"}
+        if self.has_ffn:
+            names.update({"ffn": "ffn", "norm_ffn": "norm"})
+        self.sub_parts = names
+        super().__init__(spec, parts)
+        for name, role in names.items():
+            if role == "norm" and (not isinstance(parts[name], RMSNorm) or parts[name].groups != 1):
+                raise ValueError(f"norm_of_sum block: {name} must be an RMS norm of the whole row (its weight and eps go into "
+                                 "a fused kernel)")
+
+    @staticmethod
+    def _rows(x, pending, reader, ctx):
+        """Settle what is pending and give the reader its rows."""
+        as_stream = reader.takes_stream or ctx.dtype == torch.float32
+        if isinstance(pending, NormOfSum) and not as_stream:
+            return pending.add_to(x, ctx, out_dtype=ctx.dtype)
+        settle_pending(x, pending, ctx)
+        return x if as_stream else ctx.kernels.cast_rows(x, ctx.dtype)
+
+    def forward(self, x, pending, ctx, cache):
+        h = self._rows(x, pending, self.mixer, ctx)
+        pending = NormOfSum(self.mixer.forward(h, ctx, cache), self.alpha, self.norm_mixer.weight, self.norm_mixer.eps)
+        if not self.has_ffn:
+            return x, pending
+        h = self._rows(x, pending, self.ffn, ctx)
+        return x, NormOfSum(self.ffn.forward(h, ctx), self.alpha, self.norm_ffn.weight, self.norm_ffn.eps)
 
 
 @register_part("merge", "linear_reinject")

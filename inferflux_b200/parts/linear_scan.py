@@ -1,5 +1,5 @@
-"""Two mixers that keep, per head, a matrix of state S (key channels x value channels) which every token decays and
-writes to, S <- diag(w_t) S + k_t v_t^T, and reads with the new S, o_t = S^T q_t.  Both run on the same scan kernel
+"""Mixers that keep, per head, a matrix of state S (key channels x value channels) which every token decays and
+writes to, S <- diag(w_t) S + k_t v_t^T, and reads with the new S, o_t = S^T q_t.  All run on the same scan kernel
 (`ctx.kernels.decay_scan`), which turns the raw decay inputs into decays itself, in float32.
 
 `decayed_linear_attention`: a decay per key channel from a low-rank projection,
@@ -14,6 +14,11 @@ writes to, S <- diag(w_t) S + k_t v_t^T, and reads with the new S, o_t = S^T q_t
     dt = softplus(dt + dt_bias),  w = exp(-exp(A_log) dt),  k = dt B,  q = C,  v = x       o += D x
     y = W_o (groupnorm(o * silu(z)) * norm)                     the gate in front of the norm, the norm over equal parts
 
+`retention`: a decay per head that is a constant of the design, queries and keys rotated by their position,
+
+    q = rot(W_q h),  k = rot(W_k h) / sqrt(key_dim),  v = W_v h;  w = decay[head]
+    y = W_o ((o / rms(o) per head) * silu(W_g h))
+
 S (float32) and the convolution's last taps - 1 input rows are the request's state: a slot of fixed size, whatever the
 length, zeroed when a request is admitted.  The projections take h in the run's dtype and hand their results over
 in float32; the decays, the step size, the state, the norms and the gates are float32.
@@ -24,7 +29,7 @@ import torch
 
 from ..weights.loader import TensorSpec
 from .attention import materialized_rows
-from .base import Mixer, StateSpec, WeightBuffers, register_part
+from .base import Mixer, StateSpec, WeightBuffers, build_part, register_part
 
 
 @register_part("mixer", "decayed_linear_attention")
@@ -168,3 +173,74 @@ class StateSpace(Mixer):
         y = k.gated_groupnorm(o, zx[:, :inner], buf["norm"], self.eps, groups=self.norm_groups, gate_first=True,
                               out_dtype=ctx.dtype)
         return k.linear(y, self.w_o, out_dtype=f32)
+
+
+@register_part("mixer", "retention")
+class Retention(Mixer):
+    """params: hidden_size, num_heads, key_dim, value_dim, decay (one number a head), position (a PartSpec of role
+    `position`, or None), norm_eps, names (tensor names of q, k, v, g, o)."""
+
+    _NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.heads = int(p["num_heads"])
+        self.dk = int(p["key_dim"])
+        self.dv = int(p["value_dim"])
+        if min(self.hidden, self.heads, self.dk, self.dv) <= 0:
+            raise ValueError("retention: sizes must be positive")
+        if self.dk > 512:
+            raise ValueError(f"retention: a key size of {self.dk} is beyond the kernel's 512")
+        self.decay_values = [float(v) for v in p["decay"]]
+        if len(self.decay_values) != self.heads:
+            raise ValueError(f"retention: {len(self.decay_values)} decays for {self.heads} heads")
+        pos = p.get("position")
+        self.position = build_part("position", pos) if pos is not None else None
+        self.eps = float(p.get("norm_eps", 1e-6))
+        self.names = dict(self._NAMES)
+        self.names.update(p.get("names") or {})
+        self.w_stack = self.w_o = self.decay = None
+
+    def state_spec(self):
+        """S of every head as [head, value channel, key channel]."""
+        return StateSpec((self.heads * self.dk * self.dv,), torch.float32)
+
+    def param_specs(self):
+        n, K, V, C = self.names, self.heads * self.dk, self.heads * self.dv, self.hidden
+        return {n["q"]: TensorSpec((K, C)), n["k"]: TensorSpec((K, C)), n["v"]: TensorSpec((V, C)), n["g"]: TensorSpec((V, C)),
+                n["o"]: TensorSpec((C, V))}
+
+    def projection_rows(self) -> int:
+        return 2 * self.heads * (self.dk + self.dv)
+
+    def load(self, tensors, dtype, device, projection=None):
+        """`projection`: room for the stacked projection that somebody else owns (see `projection_rows`)."""
+        n, K, V, C = self.names, self.heads * self.dk, self.heads * self.dv, self.hidden
+        layout = {"o": ((C, V), dtype), "decay": ((self.heads,), torch.float32)}
+        if projection is None:
+            layout["stack"] = ((2 * K + 2 * V, C), dtype)       # q, k, v, g one below the other: one product
+        self.buffers = buf = WeightBuffers(device, layout)
+        self.w_stack = buf["stack"] if projection is None else projection
+        at = 0
+        for s, rows in (("q", K), ("k", K), ("v", V), ("g", V)):
+            self.w_stack[at:at + rows].copy_(tensors[n[s]])
+            at += rows
+        buf["o"].copy_(tensors[n["o"]])
+        buf["decay"].copy_(torch.tensor(self.decay_values, dtype=torch.float64))
+        self.w_o, self.decay = buf["o"], buf["decay"]
+
+    def forward(self, h, ctx, cache, projected=None):
+        """`projected` = (rows, first column): the stacked projection's result, when somebody else made it."""
+        k = ctx.kernels
+        f32 = torch.float32
+        K, V = self.heads * self.dk, self.heads * self.dv
+        if projected is None:
+            projected = (k.linear(materialized_rows(k, h), self.w_stack, out_dtype=f32, allow_partial=True), 0)
+        rotary = self.position.rotary(ctx.device) if self.position is not None else None
+        proj = k.rotate_rows(*projected, self.projection_rows(), self.heads, self.dk, rotary, self.dk ** -0.5, ctx)   # q k v g
+        o = k.decay_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], None, cache.state, ctx, heads=self.heads,
+                         groups=self.heads, dk=self.dk, dv=self.dv, decay="constant", rate=self.decay)                # [T, V] float32
+        y = k.gated_groupnorm(o, proj[:, 2 * K + V:], None, self.eps, groups=self.heads, gate_first=False, out_dtype=ctx.dtype)
+        return k.linear(y, self.w_o, allow_partial=True)

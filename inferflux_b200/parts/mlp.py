@@ -8,7 +8,7 @@ import math
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import FeedForward, WeightBuffers, register_part
+from .base import FeedForward, WeightBuffers, WeightedSum, register_part
 
 
 @register_part("ffn", "swiglu")
@@ -48,6 +48,57 @@ class SwiGLU(FeedForward):
         k = ctx.kernels
         act = k.linear_swiglu(h, self.w_gate_up)         # [T, I] = silu(h Wg^T) * (h Wu^T)
         return k.linear(act, self.w_down, allow_partial=True)
+
+
+@register_part("ffn", "gated_mlp")
+class GatedMLP(FeedForward):
+    """W_down (act(W_gate h + b_gate) * (W_up h + b_up)) + b_down.
+    params: hidden_size, intermediate_size, activation (`gelu_tanh`: z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))), bias (all
+    three or none), names (tensor names of gate, up, down, gate_bias, up_bias, down_bias).  The down projection's bias
+    travels with the unadded output."""
+
+    _NAMES = {"gate": "gate", "up": "up", "down": "down", "gate_bias": "gate.b", "up_bias": "up.b", "down_bias": "down.b"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden = int(spec.params["hidden_size"])
+        self.inter = int(spec.params["intermediate_size"])
+        self.activation = str(spec.params.get("activation", "gelu_tanh"))
+        if self.activation != "gelu_tanh":
+            raise ValueError(f"gated_mlp: unknown activation {self.activation!r} (known: gelu_tanh)")
+        self.bias = bool(spec.params.get("bias", False))
+        self.names = dict(self._NAMES)
+        self.names.update(spec.params.get("names") or {})
+        self.w_gate_up = self.w_down = self.b_gate_up = self.b_down = None
+
+    def param_specs(self):
+        n, F, C = self.names, self.inter, self.hidden
+        specs = {n["gate"]: TensorSpec((F, C)), n["up"]: TensorSpec((F, C)), n["down"]: TensorSpec((C, F))}
+        if self.bias:
+            specs.update({n["gate_bias"]: TensorSpec((F,)), n["up_bias"]: TensorSpec((F,)), n["down_bias"]: TensorSpec((C,))})
+        return specs
+
+    def load(self, tensors, dtype, device):
+        n, F, C = self.names, self.inter, self.hidden
+        layout = {"w_gate_up": ((2 * F, C), dtype), "w_down": ((C, F), dtype)}
+        if self.bias:
+            layout.update({"b_gate_up": ((2 * F,), torch.float32), "b_down": ((C,), torch.float32)})
+        self.buffers = buf = WeightBuffers(device, layout)
+        buf["w_gate_up"][:F].copy_(tensors[n["gate"]])
+        buf["w_gate_up"][F:].copy_(tensors[n["up"]])
+        buf["w_down"].copy_(tensors[n["down"]])
+        if self.bias:
+            buf["b_gate_up"][:F].copy_(tensors[n["gate_bias"]])
+            buf["b_gate_up"][F:].copy_(tensors[n["up_bias"]])
+            buf["b_down"].copy_(tensors[n["down_bias"]])
+            self.b_gate_up, self.b_down = buf["b_gate_up"], buf["b_down"]
+        self.w_gate_up, self.w_down = buf["w_gate_up"], buf["w_down"]
+
+    def forward(self, h, ctx):
+        k = ctx.kernels
+        act = k.linear_geglu(h, self.w_gate_up, self.b_gate_up)      # [T, F], the activation in the product's epilogue where it can be
+        y = k.linear(act, self.w_down, allow_partial=True)
+        return y if self.b_down is None else WeightedSum([(1.0, y, self.b_down)])
 
 
 def _softplus(v: float) -> float:

@@ -6,6 +6,10 @@
 The left mixer may keep a key/value cache and state, the right one state only; the layer's state row per request
 is [the left one's, then the right one's].  The result is float32: the norms, the weights and the sum happen in one
 kernel, and the block adds it to the stream as it is.
+
+With `unadded` (plain only) the two outputs travel on as they are with their weights (`WeightedSum`), for a block whose
+norm kernel adds them.  With `joint_projection` the two mixers' stacked projections lie one below the other and a step
+of few rows makes both in one product.
 """
 from __future__ import annotations
 
@@ -14,7 +18,8 @@ import dataclasses
 import torch
 
 from ..weights.loader import TensorSpec
-from .base import Mixer, StateSpec, build_part, register_part
+from .attention import materialized_rows
+from .base import Mixer, StateSpec, WeightedSum, build_part, register_part
 
 
 def _floats(spec) -> int:
@@ -31,7 +36,8 @@ def _floats(spec) -> int:
 @register_part("mixer", "pair")
 class PairMixer(Mixer):
     """params: hidden_size, left, right (PartSpecs of role `mixer`; tensors under `left.` / `right.`), combine
-    (`plain` or `normed`), left_weight, right_weight (a, b), norm_eps, names (tensor names of left_norm, right_norm)."""
+    (`plain` or `normed`), left_weight, right_weight (a, b), norm_eps, unadded, joint_projection (both mixers must take `projected` rows), names
+    (tensor names of left_norm, right_norm)."""
 
     _NAMES = {"left_norm": "left_norm.weight", "right_norm": "right_norm.weight"}
 
@@ -46,6 +52,11 @@ class PairMixer(Mixer):
             raise ValueError(f"pair: unknown combine {self.combine!r} (known: plain, normed)")
         self.a, self.b = float(p.get("left_weight", 1.0)), float(p.get("right_weight", 1.0))
         self.eps = float(p.get("norm_eps", 1e-6))
+        self.unadded = bool(p.get("unadded", False))
+        if self.unadded and self.combine != "plain":
+            raise ValueError("pair: outputs that are normed before they are added cannot travel unadded")
+        self.joint = bool(p.get("joint_projection", False))
+        self.w_joint = None
         self.names = dict(self._NAMES)
         self.names.update(p.get("names") or {})
         if self.right.cache_spec() is not None:
@@ -74,9 +85,14 @@ class PairMixer(Mixer):
         return specs
 
     def load(self, tensors, dtype, device):
+        rooms = {}
+        if self.joint:
+            split, total = self.left.projection_rows(), self.left.projection_rows() + self.right.projection_rows()
+            self.w_joint = torch.empty((total, self.hidden), dtype=dtype, device=device)
+            rooms = {"left.": {"projection": self.w_joint[:split]}, "right.": {"projection": self.w_joint[split:]}}
         for side, part in (("left.", self.left), ("right.", self.right)):
             part.load({n[len(side):]: t for n, t in tensors.items() if n.startswith(side) and n[len(side):] in part.param_specs()},
-                      dtype, device)
+                      dtype, device, **rooms.get(side, {}))
         if self.combine == "normed":
             self.w_left = tensors[self.names["left_norm"]].to(device=device, dtype=torch.float32).contiguous()
             self.w_right = tensors[self.names["right_norm"]].to(device=device, dtype=torch.float32).contiguous()
@@ -90,6 +106,13 @@ class PairMixer(Mixer):
             raise ValueError("pair: the layer's state row does not fit the two mixers")
         left_cache = dataclasses.replace(cache, state=st[:, :lf] if lf else None)
         right_cache = dataclasses.replace(cache, kv=None, block_table=None, state=st[:, lf:lf + rf] if rf else None)
-        yl = self.left.forward(h, ctx, left_cache)
-        yr = self.right.forward(h, ctx, right_cache)
+        if self.joint and k.joins_projections(h):
+            rows = k.linear(materialized_rows(k, h), self.w_joint, out_dtype=torch.float32, allow_partial=True)
+            yl = self.left.forward(h, ctx, left_cache, projected=(rows, 0))
+            yr = self.right.forward(h, ctx, right_cache, projected=(rows, self.left.projection_rows()))
+        else:
+            yl = self.left.forward(h, ctx, left_cache)
+            yr = self.right.forward(h, ctx, right_cache)
+        if self.unadded:
+            return WeightedSum(WeightedSum.of(yl).scaled(self.a) + WeightedSum.of(yr).scaled(self.b))
         return k.pair_combine(k.materialize(yl), k.materialize(yr), self.w_left, self.w_right, self.a, self.b, self.eps)

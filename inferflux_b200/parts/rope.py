@@ -20,8 +20,8 @@ class RotaryEncoding(PositionEncoding):
     original/wavelength; or {kind: "ramp", factor, original, fast, slow}: with index(t) = rotary_dim *
     ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(index(fast)), 0) and hi = min(ceil(index(slow)),
     rotary_dim - 1), frequency i is blended towards f_i / factor by clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
-    and cos and sin are multiplied by 0.1 ln(factor) + 1).  The table is worked out in double precision and
-    kept in float32."""
+    and cos and sin are multiplied by 0.1 ln(factor) + 1), wide_table (default False; True: an unscaled table too is worked
+    out in double precision before it is kept in float32, as a scaled one always is)."""
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -33,6 +33,7 @@ class RotaryEncoding(PositionEncoding):
         if self.rotary_dim <= 0 or self.rotary_dim % 2:
             raise ValueError(f"rope: rotary_dim must be positive and even, got {self.rotary_dim}")
         self.interleaved = pairing == "interleaved"
+        self.wide_table = bool(spec.params.get("wide_table", False))
         scaling = spec.params.get("scaling")
         self.scaling = None
         self.ramp = None
@@ -77,7 +78,7 @@ class RotaryEncoding(PositionEncoding):
 
     def rotary(self, device):
         if self._table is None or self._table.inv_freq.device != torch.device(device):
-            if self.scaling is None and self.ramp is None:
+            if self.scaling is None and self.ramp is None and not self.wide_table:
                 exponent = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32) / self.rotary_dim
                 inv_freq = (1.0 / (self.theta ** exponent)).to(torch.float32)
             else:

@@ -167,8 +167,53 @@ class PlainKernels:
                 cache.kv[page, 1, :, off, :dv] = v.to(cache.kv.dtype)
         return q.to(qkv.dtype).reshape(T, nq * d).contiguous()
 
-    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None):
+    def row_norm_rope_append(self, rows, col0, bias, rotary, turn, temp, nq, nkv, d, dv, ctx, cache, q_norm=None, k_norm=None,
+                             norm_eps=0.0):
+        """Columns col0 .. of `rows`: [nq heads of d | nkv key heads of d | nkv value heads of dv], plus `bias`; the query part
+        and the key part RMS-normed as a whole (weights of their full size; None: no norm), turned by `rotary`, the queries
+        times `temp` per head; the values turned by `turn`; keys and values to the cache.  Returns (queries [T, nq d] in the
+        cache's dtype, what turns a sum of values back: None, or (float32 [T, dv/2, 2] of cos and sin, interleaved))."""
+        A, T = self.acc, rows.shape[0]
+        nQ, nK, nV = nq * d, nkv * d, nkv * dv
+        x = rows[:, col0:col0 + nQ + nK + nV].to(A)
+        if bias is not None:
+            x = x + bias.to(A)
+        pos = ctx.positions.long()
+
+        def row_norm(v, w):
+            return v if w is None else v * torch.rsqrt((v * v).mean(-1, keepdim=True) + norm_eps) * w.to(A)
+        q = self._turn(row_norm(x[:, :nQ], q_norm).view(T, nq, d), rotary, pos)
+        if temp is not None:
+            q = q * temp.to(A)[None, :, None]
+        k = self._turn(row_norm(x[:, nQ:nQ + nK], k_norm).view(T, nkv, d), rotary, pos)
+        v = self._turn(x[:, nQ + nK:].view(T, nkv, dv), turn, pos)
+        if cache.writes:
+            P = cache.page_size
+            slot = ctx.req_slot.long()[ctx.token_req.long()]
+            page = cache.block_table[slot, pos // P].long()
+            cache.kv[page, 0, :, pos % P, :d] = k.to(cache.kv.dtype)
+            cache.kv[page, 1, :, pos % P, :dv] = v.to(cache.kv.dtype)
+        back = None
+        if turn is not None:
+            ang = pos.to(torch.float32)[:, None] * turn.inv_freq[None, :]
+            back = (torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1), turn.interleaved)
+        return q.to(cache.kv.dtype).reshape(T, nQ).contiguous(), back
+
+    @staticmethod
+    def _turn_back(out, turn_back):
+        """out [T, heads, dv]: every head turned by minus the angles whose (cos, sin) `turn_back` holds."""
+        table, interleaved = turn_back
+        cos, sin = table[..., 0].to(out.dtype)[:, None, :], table[..., 1].to(out.dtype)[:, None, :]
+        half = out.shape[-1] // 2
+        u, v = (out[..., 0::2], out[..., 1::2]) if interleaved else (out[..., :half], out[..., half:])
+        a, b = u * cos + v * sin, v * cos - u * sin
+        return torch.stack([a, b], dim=-1).flatten(-2) if interleaved else torch.cat([a, b], dim=-1)
+
+    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None, turn_back=None):
         dv = d if dv is None else dv
+        if turn_back is not None:                            # in the accumulation's dtype, rounded once
+            wide = self.attention(q.to(self.acc), nq, nkv, d, window, scale, ctx, cache, chunk=chunk, sink=sink, dv=dv)
+            return self._turn_back(wide.view(-1, nq, dv), turn_back).to(q.dtype).reshape(-1, nq * dv)
         T = q.shape[0]
         P = cache.page_size
         if chunk or torch.is_tensor(sink) or sink or dv != d or cache.kv.shape[-1] != d:
@@ -351,8 +396,9 @@ class PlainKernels:
         return (a.to(self.acc) * gate).to(a.dtype)
 
     def decay_scan(self, q, k, v, raw, state, ctx, heads, groups, dk, dv, decay, tau=1.0, q_scale=1.0, step_bias=None,
-                   log_rate=None, skip=None):
-        """Per request and head a float32 matrix S, kept in `state` [slots, heads dv dk] as [head, value channel, key
+                   log_rate=None, skip=None, rate=None):
+        """decay `constant`: w = rate[h] whatever the token, no raw input.
+        Per request and head a float32 matrix S, kept in `state` [slots, heads dv dk] as [head, value channel, key
         channel]: S <- diag(w_t) S + k_t v_t^T, o_t = S^T (q_scale q_t) with the new S.  q, k: float32 [T, groups dk]
         (head h reads group h // (heads / groups)); v: [T, heads dv]; returns float32 [T, heads dv].
         decay `sigmoid_root`: raw [T, heads dk], w = sigmoid(raw)^(1/tau).
@@ -370,6 +416,8 @@ class PlainKernels:
             dt = torch.nn.functional.softplus(raw.to(A) + step_bias.to(A), threshold=30.0)
             w = torch.exp(-torch.exp(log_rate.to(A)) * dt)[:, :, None].expand(T, heads, dk)
             ka = ka * dt[:, :, None]
+        elif decay == "constant":
+            w = rate.to(A)[None, :, None].expand(T, heads, dk)
         else:
             raise ValueError(decay)
         out = torch.empty((T, heads, dv), dtype=A)
@@ -396,7 +444,7 @@ class PlainKernels:
         T, C = ya.shape
         parts = ya.reshape(T, groups, C // groups)
         normed = parts * torch.rsqrt((parts * parts).mean(-1, keepdim=True) + eps)
-        wa = w.to(A)
+        wa = torch.ones(C, dtype=A) if w is None else w.to(A)
         normed = (normed * wa).reshape(T, C) if wa.numel() == C // groups else normed.reshape(T, C) * wa
         if not gate_first:
             normed = normed * ga
@@ -419,6 +467,58 @@ class PlainKernels:
             bb = b.to(A) if b2 is None else b.to(A) + b2.to(A)
             total = total + (bb if s_b is None else bb * s_b.to(A))
         x += total.to(torch.float32)
+
+    # ------------------------------------------- norms of sums, retention, elementwise recurrence, gated gelu
+    def norm_of_sum(self, x, alpha, terms, w, eps, out_dtype=None):
+        """x <- n(alpha x + sum c (y + bias)) for the terms (c, y, bias), n the RMS norm times w (w None: x is the sum
+        itself), in place; with `out_dtype` also returns the new rows in that dtype."""
+        total = alpha * x.to(self.acc)
+        for c, y, bias in terms:
+            total = total + c * (y.to(self.acc) if bias is None else y.to(self.acc) + bias.to(self.acc))
+        if w is not None:
+            total = total * torch.rsqrt((total * total).mean(-1, keepdim=True) + eps) * w.to(self.acc)
+        x.copy_(total.to(torch.float32))
+        return None if out_dtype is None else x.to(out_dtype)
+
+    joint_rows = 8                     # steps of at most so many tokens make a pair's two projections in one product
+
+    def joins_projections(self, h):
+        return h.shape[0] <= self.joint_rows
+
+    def rotate_rows(self, rows, col0, width, heads, dk, rotary, k_scale, ctx):
+        """float32 [T, width] from columns col0 .. of `rows`: heads of dk (queries), heads of dk (keys), the rest; queries
+        and keys turned by the position, keys times k_scale behind it."""
+        T, K = rows.shape[0], heads * dk
+        x = rows[:, col0:col0 + width].to(self.acc)
+        pos = ctx.positions.long()
+        q = self._turn(x[:, :K].view(T, heads, dk), rotary, pos).reshape(T, K)
+        k = self._turn(x[:, K:2 * K].view(T, heads, dk), rotary, pos).reshape(T, K) * k_scale
+        return torch.cat([q, k, x[:, 2 * K:]], dim=-1).to(torch.float32)
+
+    def gated_scan(self, rows, bias, state, width, ctx, out_dtype):
+        """rows [T, 3 width] = z, x, g (bias [2 width] joins z and x): S <- (1 - sigmoid(z)) S + sigmoid(z) c with c = x + 1/2
+        where x >= 0 and sigmoid(x) where x < 0; returns S silu(g); S per request in `state` [slots, >= width], moved on."""
+        A = self.acc
+        z, u = (rows[:, :2 * width].to(A) + bias.to(A)).split(width, dim=1)
+        g = rows[:, 2 * width:3 * width].to(A)
+        c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+        keep, take = torch.sigmoid(-z), torch.sigmoid(z) * c
+        out = torch.empty_like(z)
+        cu, slots = ctx.cu_seqlens.tolist(), ctx.req_slot.tolist()
+        for r in range(ctx.num_requests):
+            S = state[slots[r], :width].to(A)
+            for t in range(cu[r], cu[r + 1]):
+                S = keep[t] * S + take[t]
+                out[t] = S
+            state[slots[r], :width] = S.to(state.dtype)
+        return (out * g * torch.sigmoid(g)).to(out_dtype)
+
+    def linear_geglu(self, a, w_gate_up, bias):
+        """gelu_tanh(a Wg^T + bg) * (a Wu^T + bu) with gate and up stacked."""
+        both = self.linear(a, w_gate_up, bias=bias, out_dtype=self.acc)
+        g, u = both.chunk(2, dim=-1)
+        g = 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
+        return (g * u).to(a.dtype)
 
     # ------------------------------------------------------- mixture of experts
     def moe_route(self, z, correction, top, of_chosen=False, kind=None, floor=0.0):
