@@ -20,6 +20,7 @@
 //   d_v, d_row   values of another size than the keys; both lie in cache rows of d_row elements
 //                (a multiple of 8 that holds either; what lies behind a row's d or d_v elements is zero)
 //   chunk        > 0: a query at position p sees the keys from (p / chunk) * chunk on, not from 0
+//   turn_back    float2 [tokens, d_v / 2]: a head's output is turned back by the token's angles (see TurnBack)
 //   sink         1: the softmax's denominator holds one more unit, a key of score 0 without a value
 #include "common.cuh"
 
@@ -68,7 +69,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
                                          const int* __restrict__ rows, T* __restrict__ out, int num_tokens, int nq,
                                          int nkv, int d, int d_v, int d_row,
                                          int page_size, int max_blocks, int num_pages, int window, int chunk,
-                                         int sink, const float* __restrict__ sink_values, float scale) {
+                                         int sink, const float* __restrict__ sink_values, float scale, TurnBack turn) {
   __shared__ __align__(16) float q_s[kWarpsPerBlock][kMaxHeadDim];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * kWarpsPerBlock + warp;
@@ -130,6 +131,23 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
   }
   const float inv = l > 0.0f ? 1.0f / l : 0.0f;
   T* orow = out + ((size_t)t * nq + h) * d_v;
+  if (turn.table != nullptr) {                             // the head's row through shared memory: pairs meet there
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kMaxHeadDim / 32; ++i) {
+      const int e = lane + 32 * i;
+      if (e < d_v) q_s[warp][e] = acc[i] * inv;
+    }
+    __syncwarp();
+    for (int m = lane; m < d_v / 2; m += 32) {
+      const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + d_v / 2;
+      float u = q_s[warp][e0], v = q_s[warp][e1];
+      TurnBack::apply(turn.table[(size_t)t * (d_v / 2) + m], u, v);
+      orow[e0] = from_f32<T>(u);
+      orow[e1] = from_f32<T>(v);
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < kMaxHeadDim / 32; ++i) {
     const int e = lane + 32 * i;
@@ -145,8 +163,11 @@ extern "C" int ifx_attention_generic_sink(const void* q, const void* kv_pool, co
                                           const int* positions, const int* token_req, const int* req_slot,
                                           const int* rows, void* out, int num_tokens, int nq, int nkv, int d, int d_v,
                                           int d_row, int page_size, int max_blocks, int num_pages, int window, int chunk,
-                                          int sink, const float* sink_values, float scale, int dtype, cudaStream_t stream) {
+                                          int sink, const float* sink_values, float scale, const float* turn_back,
+                                          int turn_interleaved, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  if (turn_back != nullptr && d_v % 2) return IFX_E_BADARG;
+  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
   if (nq <= 0 || nkv <= 0 || nq % nkv || d <= 0 || d_v <= 0 || d_row % 8 || d_row > kMaxHeadDim || d > d_row ||
       d_v > d_row || page_size <= 0 || max_blocks <= 0 || chunk < 0)
     return IFX_E_BADARG;
@@ -155,12 +176,12 @@ extern "C" int ifx_attention_generic_sink(const void* q, const void* kv_pool, co
   if (dtype == IFX_DT_F32)
     attention_generic_kernel<float><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
         (const float*)q, (const float*)kv_pool, block_table, positions, token_req, req_slot, rows, (float*)out,
-        num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, window, chunk, sink, sink_values, scale);
+        num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, window, chunk, sink, sink_values, scale, turn);
   else if (dtype == IFX_DT_BF16)
     attention_generic_kernel<__nv_bfloat16><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv_pool, block_table, positions, token_req, req_slot,
         rows, (__nv_bfloat16*)out, num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, window,
-        chunk, sink, sink_values, scale);
+        chunk, sink, sink_values, scale, turn);
   else
     return IFX_E_DTYPE;
   IFX_CHECK_LAUNCH();
@@ -173,8 +194,8 @@ extern "C" int ifx_attention_generic_ex(const void* q, const void* kv_pool, cons
                                         int d_row, int page_size, int max_blocks, int num_pages, int window, int chunk,
                                         int sink, float scale, int dtype, cudaStream_t stream) {
   return ifx_attention_generic_sink(q, kv_pool, block_table, positions, token_req, req_slot, rows, out, num_tokens, nq, nkv,
-                                    d, d_v, d_row, page_size, max_blocks, num_pages, window, chunk, sink, nullptr, scale, dtype,
-                                    stream);
+                                    d, d_v, d_row, page_size, max_blocks, num_pages, window, chunk, sink, nullptr, scale, nullptr,
+                                    0, dtype, stream);
 }
 
 extern "C" int ifx_attention_generic(const void* q, const void* kv_pool, const int* block_table,

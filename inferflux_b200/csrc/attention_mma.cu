@@ -98,11 +98,24 @@ struct PageMap {
 };
 
 // ------------------------------------------------------------- prompt portions
+// The finished rows of a key head's G query heads ([G][D] in shared memory), turned back and stored.
+template <int D>
+__device__ __forceinline__ void store_turned(const float* rows_s, bf16* out, const TurnBack& turn, int t, int G, int tid, int threads) {
+  for (int idx = tid; idx < G * (D / 2); idx += threads) {
+    const int row = idx / (D / 2), m = idx % (D / 2);
+    const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + D / 2;
+    float u = rows_s[row * D + e0], v = rows_s[row * D + e1];
+    TurnBack::apply(turn.table[(size_t)t * (D / 2) + m], u, v);
+    out[row * D + e0] = __float2bfloat16_rn(u);
+    out[row * D + e1] = __float2bfloat16_rn(v);
+  }
+}
+
 template <int D, int KT>
 __global__ void __launch_bounds__(128)
 attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool, const int* __restrict__ block_table,
                     const int* __restrict__ tiles, const int* __restrict__ req_slot, bf16* __restrict__ out, int nq,
-                    int nkv, int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window,
+                    int nkv, int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn,
                     float scale_log2, int tbl_cap) {
   constexpr int LDS = D + 8;            // shared-memory row stride in elements
   constexpr int CPR = D / 8;            // 16-byte chunks per row
@@ -274,6 +287,27 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
   }
   const float i_lo = l_lo > 0.0f ? 1.0f / l_lo : 0.0f, i_hi = l_hi > 0.0f ? 1.0f / l_hi : 0.0f;
   const int r_lo = warp * 16 + (lane >> 2), r_hi = r_lo + 8;
+  if (turn.table != nullptr) {                          // both elements of a pair lie in this thread
+    const float2* cs_lo = turn.table + (size_t)(row0 + min(r_lo, rows - 1)) * (D / 2);
+    const float2* cs_hi = turn.table + (size_t)(row0 + min(r_hi, rows - 1)) * (D / 2);
+    if (turn.interleaved) {
+#pragma unroll
+      for (int n = 0; n < D / 8; ++n) {
+        const int m = n * 4 + (lane & 3);
+        TurnBack::apply(cs_lo[m], o[n][0], o[n][1]);
+        TurnBack::apply(cs_hi[m], o[n][2], o[n][3]);
+      }
+    } else {
+#pragma unroll
+      for (int n = 0; n < D / 16; ++n) {
+        const int m = n * 8 + 2 * (lane & 3);
+        TurnBack::apply(cs_lo[m], o[n][0], o[n + D / 16][0]);
+        TurnBack::apply(cs_lo[m + 1], o[n][1], o[n + D / 16][1]);
+        TurnBack::apply(cs_hi[m], o[n][2], o[n + D / 16][2]);
+        TurnBack::apply(cs_hi[m + 1], o[n][3], o[n + D / 16][3]);
+      }
+    }
+  }
 #pragma unroll
   for (int n = 0; n < D / 8; ++n) {
     const int col = n * 8 + 2 * (lane & 3);
@@ -291,7 +325,7 @@ template <int D, int STAGES>
 __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool, const int* __restrict__ block_table,
                    const int4* __restrict__ decode_meta, bf16* __restrict__ out, int nq, int nkv, int page_size,
-                   int page_shift, int max_blocks, int num_pages, KeyMask window, float scale_log2, int tbl_cap) {
+                   int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn, float scale_log2, int tbl_cap) {
   constexpr int LDS = D + 8;
   constexpr int CPR = D / 8;
   constexpr int STAGE_ELEMS = 2 * 16 * LDS;             // K tile then V tile
@@ -491,10 +525,11 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
         L += f * c_l[w * 16 + row];
       }
     }
-    const int head = g * G + row;
     if (num_splits == 1) {
       if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-      out[((size_t)t * nq + head) * D + dim] = __float2bfloat16_rn(L > 0.0f ? O / L : 0.0f);
+      const float v = L > 0.0f ? O / L : 0.0f;
+      if (turn.table != nullptr) fin_o[row * D + dim] = v;      // turned back below, where the pairs meet
+      else out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(v);
     } else {
       fin_o[row * D + dim] = O;
       if (dim == 0) {
@@ -503,14 +538,19 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
       }
     }
   }
-  if (num_splits == 1) return;
+  if (num_splits == 1) {
+    if (turn.table != nullptr) {
+      __syncthreads();
+      store_turned<D>(fin_o, out + ((size_t)t * nq + g * G) * D, turn, t, G, tid, 128);
+    }
+    return;
+  }
   // ---- merge over the cluster: block `split` takes dims [split * D / n, (split + 1) * D / n) of every
   //      head and reads all blocks' (maximum, sum, output) through distributed shared memory, in block order
   cg::cluster_group cluster = cg::this_cluster();
   cluster.sync();
-  const int DS = D / num_splits;
-  for (int idx = tid; idx < G * DS; idx += 128) {
-    const int row = idx / DS, dim = split * DS + idx % DS;
+  // every block's share of dimension `dim` of head `row`, merged
+  auto merged = [&](int row, int dim) -> float {
     float ms[8], ls[8], os[8];
 #pragma unroll
     for (int c = 0; c < 8; ++c) {
@@ -536,7 +576,25 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
       }
     }
     if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-    out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(L > 0.0f ? O / L : 0.0f);
+    return L > 0.0f ? O / L : 0.0f;
+  };
+  if (turn.table != nullptr) {                          // a block takes pairs: both elements and the query's angle
+    const int PS = D / 2 / num_splits;
+    for (int idx = tid; idx < G * PS; idx += 128) {
+      const int row = idx / PS, m = split * PS + idx % PS;
+      const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + D / 2;
+      float u = merged(row, e0), v = merged(row, e1);
+      TurnBack::apply(turn.table[(size_t)t * (D / 2) + m], u, v);
+      bf16* o_row = out + ((size_t)t * nq + g * G + row) * D;
+      o_row[e0] = __float2bfloat16_rn(u);
+      o_row[e1] = __float2bfloat16_rn(v);
+    }
+  } else {
+    const int DS = D / num_splits;
+    for (int idx = tid; idx < G * DS; idx += 128) {
+      const int row = idx / DS, dim = split * DS + idx % DS;
+      out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(merged(row, dim));
+    }
   }
   cluster.sync();                                       // nobody leaves while its shared memory is being read
 }
@@ -555,7 +613,7 @@ __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16* __restrict__ q,
                        const int* __restrict__ block_table, const int4* __restrict__ decode_meta,
                        bf16* __restrict__ out, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                       int num_pages, KeyMask window, float scale_log2, int tbl_cap, int* __restrict__ error_flag) {
+                       int num_pages, KeyMask window, TurnBack turn, float scale_log2, int tbl_cap, int* __restrict__ error_flag) {
   constexpr int LDS = D + 8;
   constexpr int CPR = D / 8;
   constexpr int HALVES = D / 64;
@@ -793,7 +851,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
     }
     if (num_splits == 1) {
       if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-    out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(L > 0.0f ? O / L : 0.0f);
+      const float v = L > 0.0f ? O / L : 0.0f;
+      if (turn.table != nullptr) fin_o[row * D + dim] = v;      // turned back below, where the pairs meet
+      else out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(v);
     } else {
       fin_o[row * D + dim] = O;
       if (dim == 0) {
@@ -802,12 +862,17 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
       }
     }
   }
-  if (num_splits == 1) return;
+  if (num_splits == 1) {
+    if (turn.table != nullptr) {
+      __syncthreads();
+      store_turned<D>(fin_o, out + ((size_t)t * nq + g * G) * D, turn, t, G, tid, THREADS);
+    }
+    return;
+  }
   cg::cluster_group cluster = cg::this_cluster();
   cluster.sync();
-  const int DS = D / num_splits;
-  for (int idx = tid; idx < G * DS; idx += THREADS) {
-    const int row = idx / DS, dim = split * DS + idx % DS;
+  // every block's share of dimension `dim` of head `row`, merged
+  auto merged = [&](int row, int dim) -> float {
     float ms[16], ls[16], os[16];
 #pragma unroll
     for (int c = 0; c < 16; ++c) {
@@ -833,7 +898,25 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
       }
     }
     if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-    out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(L > 0.0f ? O / L : 0.0f);
+    return L > 0.0f ? O / L : 0.0f;
+  };
+  if (turn.table != nullptr) {                          // a block takes pairs: both elements and the query's angle
+    const int PS = D / 2 / num_splits;
+    for (int idx = tid; idx < G * PS; idx += THREADS) {
+      const int row = idx / PS, m = split * PS + idx % PS;
+      const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + D / 2;
+      float u = merged(row, e0), v = merged(row, e1);
+      TurnBack::apply(turn.table[(size_t)t * (D / 2) + m], u, v);
+      bf16* o_row = out + ((size_t)t * nq + g * G + row) * D;
+      o_row[e0] = __float2bfloat16_rn(u);
+      o_row[e1] = __float2bfloat16_rn(v);
+    }
+  } else {
+    const int DS = D / num_splits;
+    for (int idx = tid; idx < G * DS; idx += THREADS) {
+      const int row = idx / DS, dim = split * DS + idx % DS;
+      out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(merged(row, dim));
+    }
   }
   cluster.sync();
 }
@@ -841,7 +924,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
 template <int D, int STAGES, int WARPS>
 int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const int* block_table, const int4* decode_meta,
                              bf16* out, int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                             int num_pages, KeyMask window, float scale_log2, int num_splits, int max_keys, int* error_flag,
+                             int num_pages, KeyMask window, TurnBack turn, float scale_log2, int num_splits, int max_keys, int* error_flag,
                              cudaStream_t stream) {
   constexpr int stage_bytes = WARPS * STAGES * 2 * 16 * D * 2;
   constexpr int merge_bytes = (WARPS * 16 * D + 2 * WARPS * 16) * 4;
@@ -870,7 +953,7 @@ int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const i
   }
   return launch_pdl(attn_decode_tma_kernel<D, STAGES, WARPS>, dim3(num_items, nkv, num_splits), dim3(WARPS * 32),
                     (size_t)smem, stream, num_splits, pool_map, q, block_table, decode_meta, out, nq, nkv, page_size,
-                    page_shift, max_blocks, num_pages, window, scale_log2, tbl_cap, error_flag);
+                    page_shift, max_blocks, num_pages, window, turn, scale_log2, tbl_cap, error_flag);
 }
 
 // Four warps with three 16-key tiles in flight each (96 KB a block at head size 128) feed the HBM when two blocks
@@ -882,13 +965,13 @@ int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const i
 template <int D>
 int launch_decode_tma(const CUtensorMap& pool_map, const bf16* q, const int* block_table, const int4* decode_meta,
                       bf16* out, int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                      int num_pages, KeyMask window, float scale_log2, int num_splits, int max_keys, int* error_flag,
+                      int num_pages, KeyMask window, TurnBack turn, float scale_log2, int num_splits, int max_keys, int* error_flag,
                       cudaStream_t stream) {
   constexpr int STAGES = D <= 128 ? 3 : 2;
   const long long blocks = (long long)num_items * nkv * num_splits;
   const int keys_per_block = max_keys / (num_splits > 0 ? num_splits : 1);
 #define ARGS pool_map, q, block_table, decode_meta, out, num_items, nq, nkv, page_size, page_shift, max_blocks, num_pages, \
-             window, scale_log2, num_splits, max_keys, error_flag, stream
+             window, turn, scale_log2, num_splits, max_keys, error_flag, stream
   if (D <= 128 && blocks <= 104 && keys_per_block >= 8 * 16) return launch_decode_tma_stages<D, STAGES, 8>(ARGS);
   return launch_decode_tma_stages<D, STAGES, 4>(ARGS);
 #undef ARGS
@@ -897,7 +980,7 @@ int launch_decode_tma(const CUtensorMap& pool_map, const bf16* q, const int* blo
 template <int D>
 int launch_prefill(const bf16* q, const bf16* kv_pool, const int* block_table, const int* tiles, const int* req_slot,
                    bf16* out, int num_tiles, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                   int num_pages, KeyMask window, float scale_log2, int max_keys, cudaStream_t stream) {
+                   int num_pages, KeyMask window, TurnBack turn, float scale_log2, int max_keys, cudaStream_t stream) {
   constexpr int KT = 64;                                // keys per tile
   constexpr int tile_bytes = (64 + 4 * KT) * (D + 8) * 2;
   int tbl_cap = max_keys / page_size + 2;               // entries a tile can need
@@ -911,7 +994,7 @@ int launch_prefill(const bf16* q, const bf16* kv_pool, const int* block_table, c
   }
   dim3 grid(num_tiles * 4, nq);
   attn_prefill_kernel<D, KT><<<grid, 128, smem, stream>>>(q, kv_pool, block_table, tiles, req_slot, out, nq, nkv, page_size,
-                                                      page_shift, max_blocks, num_pages, window, scale_log2, tbl_cap);
+                                                      page_shift, max_blocks, num_pages, window, turn, scale_log2, tbl_cap);
   IFX_CHECK_LAUNCH();
   return 0;
 }
@@ -919,7 +1002,7 @@ int launch_prefill(const bf16* q, const bf16* kv_pool, const int* block_table, c
 template <int D>
 int launch_decode(const bf16* q, const bf16* kv_pool, const int* block_table, const int4* decode_meta, bf16* out,
                   int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks, int num_pages,
-                  KeyMask window, float scale_log2, int num_splits, int max_keys, cudaStream_t stream) {
+                  KeyMask window, TurnBack turn, float scale_log2, int num_splits, int max_keys, cudaStream_t stream) {
   constexpr int STAGES = D <= 128 ? 3 : 2;
   constexpr int stage_bytes = 4 * STAGES * 2 * 16 * (D + 8) * 2;
   constexpr int merge_bytes = (4 * 16 * D + 2 * 4 * 16) * 4;
@@ -949,7 +1032,7 @@ int launch_decode(const bf16* q, const bf16* kv_pool, const int* block_table, co
   cfg.attrs = attr;
   cfg.numAttrs = num_splits > 1 ? 1 : 0;
   cudaError_t e = cudaLaunchKernelEx(&cfg, attn_decode_kernel<D, STAGES>, q, kv_pool, block_table, decode_meta, out, nq,
-                                     nkv, page_size, page_shift, max_blocks, num_pages, window, scale_log2, tbl_cap);
+                                     nkv, page_size, page_shift, max_blocks, num_pages, window, turn, scale_log2, tbl_cap);
   if (e != cudaSuccess) return (int)e;
   return 0;
 }
@@ -990,12 +1073,15 @@ int ifx_attention_mma_supports(int d) {
 // max_keys: no request of the step holds more keys than this (sizes the shared-memory copy of the block table).
 // chunk, sink: see KeyMask.
 // sink_values: null, or one learned number per query head (float32 [nq]) that takes the place of the sink's score 0.
+// turn_back: null, or float2 [tokens, d / 2], see TurnBack.
 int ifx_attention_prefill_bf16_sink(const void* q, const void* kv_pool, const int* block_table, const int* tiles,
                                     const int* req_slot, void* out, int num_tiles, int nq, int nkv, int d, int page_size,
                                     int max_blocks, int num_pages, int window_size, int chunk, int sink,
-                                    const float* sink_values, float scale, int max_keys, int* error_flag,
+                                    const float* sink_values, float scale, const float* turn_back,
+                                   int turn_interleaved, int max_keys, int* error_flag,
                                     cudaStream_t stream) {
   const KeyMask window{window_size, chunk, sink, sink_values};
+  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
   if (num_tiles <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || max_blocks <= 0 || nq > 65535 || !(scale > 0.0f))
     return IFX_E_BADARG;                                  // the kernels take the maximum before scaling
@@ -1003,7 +1089,7 @@ int ifx_attention_prefill_bf16_sink(const void* q, const void* kv_pool, const in
   const int ps = shift_of(page_size);
 #define CALL(DD)                                                                                                   \
   launch_prefill<DD>((const bf16*)q, (const bf16*)kv_pool, block_table, tiles, req_slot, (bf16*)out, num_tiles, nq, \
-                     nkv, page_size, ps, max_blocks, num_pages, window, scale_log2, max_keys, stream)
+                     nkv, page_size, ps, max_blocks, num_pages, window, turn, scale_log2, max_keys, stream)
   IFX_DISPATCH_D(d, CALL)
 #undef CALL
 }
@@ -1013,7 +1099,7 @@ int ifx_attention_prefill_bf16_ex(const void* q, const void* kv_pool, const int*
                                   int max_blocks, int num_pages, int window_size, int chunk, int sink, float scale,
                                   int max_keys, int* error_flag, cudaStream_t stream) {
   return ifx_attention_prefill_bf16_sink(q, kv_pool, block_table, tiles, req_slot, out, num_tiles, nq, nkv, d, page_size,
-                                         max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, max_keys, error_flag,
+                                         max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, max_keys, error_flag,
                                          stream);
 }
 
@@ -1038,9 +1124,10 @@ int ifx_attention_decode_max_splits(int d, int page_size) {
 // max_keys: no token of the step sees more keys than this.
 int ifx_attention_decode_bf16_sink(const void* q, const void* kv_pool, const int* block_table, const int* decode_meta,
                                    void* out, int num_items, int nq, int nkv, int d, int page_size, int max_blocks,
-                                   int num_pages, int window_size, int chunk, int sink, const float* sink_values, float scale,
-                                   int num_splits, int max_keys, int* error_flag, cudaStream_t stream) {
+                                   int num_pages, int window_size, int chunk, int sink, const float* sink_values, float scale, const float* turn_back,
+                                   int turn_interleaved, int num_splits, int max_keys, int* error_flag, cudaStream_t stream) {
   const KeyMask window{window_size, chunk, sink, sink_values};
+  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
   if (num_items <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv || nq / nkv > 16 || page_size <= 0 || max_blocks <= 0 || nkv > 65535 ||
       nq > 65535)
@@ -1058,7 +1145,7 @@ int ifx_attention_decode_bf16_sink(const void* q, const void* kv_pool, const int
     if (rc) return rc;
 #define CALL_TMA(DD)                                                                                              \
   return launch_decode_tma<DD>(pool_map, (const bf16*)q, block_table, (const int4*)decode_meta, (bf16*)out,       \
-                               num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, scale_log2,      \
+                               num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn, scale_log2,      \
                                num_splits, max_keys, error_flag, stream)
     if (d == 64) CALL_TMA(64);
     if (d == 128) CALL_TMA(128);
@@ -1067,7 +1154,7 @@ int ifx_attention_decode_bf16_sink(const void* q, const void* kv_pool, const int
   }
 #define CALL(DD)                                                                                                  \
   launch_decode<DD>((const bf16*)q, (const bf16*)kv_pool, block_table, (const int4*)decode_meta, (bf16*)out,     \
-                    num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, scale_log2, num_splits,     \
+                    num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn, scale_log2, num_splits,     \
                     max_keys, stream)
   IFX_DISPATCH_D(d, CALL)
 #undef CALL
@@ -1078,7 +1165,7 @@ int ifx_attention_decode_bf16_ex(const void* q, const void* kv_pool, const int* 
                                  int num_pages, int window_size, int chunk, int sink, float scale, int num_splits,
                                  int max_keys, int* error_flag, cudaStream_t stream) {
   return ifx_attention_decode_bf16_sink(q, kv_pool, block_table, decode_meta, out, num_items, nq, nkv, d, page_size,
-                                        max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, num_splits, max_keys,
+                                        max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, num_splits, max_keys,
                                         error_flag, stream);
 }
 

@@ -75,6 +75,14 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&r)[32]) {
         "=r"(u[25]), "=r"(u[26]), "=r"(u[27]), "=r"(u[28]), "=r"(u[29]), "=r"(u[30]), "=r"(u[31])
       : "r"(taddr));
 }
+__device__ __forceinline__ void tmem_ld16f(uint32_t taddr, float (&r)[16]) {
+  uint32_t* u = reinterpret_cast<uint32_t*>(r);
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+      : "=r"(u[0]), "=r"(u[1]), "=r"(u[2]), "=r"(u[3]), "=r"(u[4]), "=r"(u[5]), "=r"(u[6]), "=r"(u[7]), "=r"(u[8]),
+        "=r"(u[9]), "=r"(u[10]), "=r"(u[11]), "=r"(u[12]), "=r"(u[13]), "=r"(u[14]), "=r"(u[15])
+      : "r"(taddr));
+}
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -125,7 +133,7 @@ __global__ void __launch_bounds__(kThreads)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap pool_map,
                             const int* __restrict__ block_table, const int* __restrict__ tiles,
                             const int* __restrict__ req_slot, bf16* __restrict__ out, int nq, int nkv, int page_size,
-                            int page_shift, int max_blocks, int num_pages, KeyMask window, float scale_log2,
+                            int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn, float scale_log2,
                             int* __restrict__ error_flag) {
   using L = PrefillLayout<D>;
   constexpr int HALVES = L::HALVES, SLOTS = L::SLOTS;
@@ -386,6 +394,50 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
       if (window.sink && m_ref > -INFINITY) l_run += exp2f(window.sink_log2(h) - m_ref * scale_log2);     // the sink's share
       const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
       bf16* dst = out + ((size_t)(row0 + q * kBM + row) * nq + h) * D;
+      if (turn.table != nullptr) {                         // 16 pairs at a time: 32 columns, or 16 and their 16 partners
+        const float4* cs4 = reinterpret_cast<const float4*>(turn.table + (size_t)(row0 + q * kBM + min(row, max(rows_q - 1, 0))) * (D / 2));
+        const int apart = turn.interleaved ? 16 : D / 2;
+#pragma unroll 1
+        for (int m0 = 0; m0 < D / 2; m0 += 16) {
+          const int c = turn.interleaved ? 2 * m0 : m0;
+          float lo[16], hi[16];
+          tmem_ld16f(o_addr + c, lo);
+          tmem_ld16f(o_addr + c + apart, hi);
+          tmem_wait_ld();
+          if (turn.interleaved) {
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+              const float4 a = cs4[(m0 + j) >> 1], b = cs4[(m0 + 8 + j) >> 1];
+              TurnBack::apply(make_float2(a.x, a.y), lo[2 * j], lo[2 * j + 1]);
+              TurnBack::apply(make_float2(a.z, a.w), lo[2 * j + 2], lo[2 * j + 3]);
+              TurnBack::apply(make_float2(b.x, b.y), hi[2 * j], hi[2 * j + 1]);
+              TurnBack::apply(make_float2(b.z, b.w), hi[2 * j + 2], hi[2 * j + 3]);
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; j += 2) {
+              const float4 a = cs4[(m0 + j) >> 1];
+              TurnBack::apply(make_float2(a.x, a.y), lo[j], hi[j]);
+              TurnBack::apply(make_float2(a.z, a.w), lo[j + 1], hi[j + 1]);
+            }
+          }
+          if (row < rows_q) {
+#pragma unroll
+            for (int j = 0; j < 16; j += 8) {
+              uint4 vl, vh;
+              __nv_bfloat162* l2 = reinterpret_cast<__nv_bfloat162*>(&vl);
+              __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&vh);
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                l2[e] = __floats2bfloat162_rn(lo[j + 2 * e] * inv, lo[j + 2 * e + 1] * inv);
+                h2[e] = __floats2bfloat162_rn(hi[j + 2 * e] * inv, hi[j + 2 * e + 1] * inv);
+              }
+              *reinterpret_cast<uint4*>(dst + c + j) = vl;
+              *reinterpret_cast<uint4*>(dst + c + apart + j) = vh;
+            }
+          }
+        }
+      } else
 #pragma unroll 1
       for (int c = 0; c < D; c += 32) {
         float t[32];
@@ -415,7 +467,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 template <int D>
 static int launch_prefill_tcgen05(const bf16* q, int num_tokens, const bf16* kv_pool, const int* block_table,
                                   const int* tiles, const int* req_slot, bf16* out, int num_tiles, int nq, int nkv,
-                                  int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window,
+                                  int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn,
                                   float scale_log2, int* error_flag, cudaStream_t stream) {
   CUtensorMap q_map, pool_map;
   int rc = make_tensor_map_bf16(&q_map, q, num_tokens, nq * D, kBM);
@@ -432,7 +484,7 @@ static int launch_prefill_tcgen05(const bf16* q, int num_tokens, const bf16* kv_
   }
   return launch_pdl(attn_prefill_tcgen05_kernel<D>, dim3(nq, num_tiles), dim3(kThreads), smem, stream, 1, q_map,
                     pool_map, block_table, tiles, req_slot, out, nq, nkv, page_size, page_shift, max_blocks,
-                    num_pages, window, scale_log2, error_flag);
+                    num_pages, window, turn, scale_log2, error_flag);
 }
 
 }  // namespace ifx
@@ -450,11 +502,14 @@ int ifx_attention_prefill_tcgen05_supports(int d, int page_size) {
 // flat row, rows <= 256, first position).
 // chunk, sink: see KeyMask (common.cuh).
 // sink_values: null, or one learned number per query head (float32 [nq]) that takes the place of the sink's score 0.
+// turn_back: null, or float2 [tokens, d / 2], see TurnBack.
 int ifx_attention_prefill_tcgen05_sink(const void* q, int num_tokens, const void* kv_pool, const int* block_table,
                                        const int* tiles, const int* req_slot, void* out, int num_tiles, int nq, int nkv,
                                        int d, int page_size, int max_blocks, int num_pages, int window_size, int chunk,
-                                       int sink, const float* sink_values, float scale, int* error_flag, cudaStream_t stream) {
+                                       int sink, const float* sink_values, float scale, const float* turn_back,
+                                   int turn_interleaved, int* error_flag, cudaStream_t stream) {
   const KeyMask window{window_size, chunk, sink, sink_values};
+  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
   if (num_tiles <= 0) return 0;
   if (!ifx_attention_prefill_tcgen05_supports(d, page_size) || nq <= 0 || nkv <= 0 || nq % nkv || max_blocks <= 0 ||
       num_tiles > 65535 || !(scale > 0.0f) || error_flag == nullptr)
@@ -464,10 +519,10 @@ int ifx_attention_prefill_tcgen05_sink(const void* q, int num_tokens, const void
   const float scale_log2 = scale * 1.4426950408889634f;
   if (d == 64)
     return launch_prefill_tcgen05<64>((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot,
-                                      (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window,
+                                      (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn,
                                       scale_log2, error_flag, stream);
   return launch_prefill_tcgen05<128>((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot,
-                                     (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window,
+                                     (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn,
                                      scale_log2, error_flag, stream);
 }
 
@@ -476,7 +531,7 @@ int ifx_attention_prefill_tcgen05_ex(const void* q, int num_tokens, const void* 
                                      int d, int page_size, int max_blocks, int num_pages, int window_size, int chunk,
                                      int sink, float scale, int* error_flag, cudaStream_t stream) {
   return ifx_attention_prefill_tcgen05_sink(q, num_tokens, kv_pool, block_table, tiles, req_slot, out, num_tiles, nq, nkv, d,
-                                            page_size, max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, error_flag,
+                                            page_size, max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, error_flag,
                                             stream);
 }
 

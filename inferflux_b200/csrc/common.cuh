@@ -96,6 +96,30 @@ struct KeyMask {
   __device__ __forceinline__ bool any() const { return window > 0 || chunk > 0; }
 };
 
+// Values that were turned by their own position before they were summed: the sum is turned back by the query's.  `table`
+// [tokens, size / 2] holds cos and sin of the query's angles (null: nothing is turned); pairs are (m, m + size / 2), or
+// neighbours with `interleaved`.
+struct TurnBack {
+  const float2* table;
+  int interleaved;
+  __device__ __forceinline__ static void apply(float2 cs, float& u, float& v) {
+    const float a = u * cs.x + v * cs.y, b = v * cs.x - u * cs.y;
+    u = a;
+    v = b;
+  }
+};
+
+// The tanh form of gelu, z/2 (1 + tanh(s (z + 0.044715 z^3))) with s = sqrt(2/pi), as z sigmoid(2 s (z + 0.044715 z^3)).
+__device__ __forceinline__ float gelu_tanh_f32(float z) {
+  const float u = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.0f + expf(-u));
+}
+// The same with the fast exponential and division: a few float32 ulps, for results that are rounded to bfloat16.
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float u = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return __fdividef(z, 1.0f + __expf(fminf(-u, 80.0f)));
+}
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 

@@ -9,6 +9,7 @@
 //   DECAY_CHANNEL   raw [T, heads dk]:  w = sigmoid(raw)^(1 / tau) = exp(logsigmoid(raw) / tau), one per key channel
 //   DECAY_STEP      raw [T, heads]:     dt = softplus(raw + step_bias[h]);  w = exp(-exp(log_rate[h]) dt) for the
 //                                       whole head;  k_t is multiplied by dt
+//   DECAY_CONSTANT  no raw input:       w = rate[h], whatever the token
 //
 // All inputs are float32 rows that may be wider than what is read (row strides in elements, pointers already at the
 // first column).  The state lives in a slot per request, [head, value channel, key channel] (a column of S is
@@ -24,7 +25,7 @@
 
 namespace ifx {
 
-enum { DECAY_CHANNEL = 0, DECAY_STEP = 1 };
+enum { DECAY_CHANNEL = 0, DECAY_STEP = 1, DECAY_CONSTANT = 2 };
 
 struct DecayScanArgs {
   const float* q; long long q_stride;
@@ -34,7 +35,8 @@ struct DecayScanArgs {
   float* state; long long state_slot_stride;
   const int* req_slot; const int* cu_seqlens;
   float* out;                                  // [T, heads dv]
-  const float* step_bias; const float* log_rate; const float* skip;     // per head, DECAY_STEP (skip: either mode)
+  const float* step_bias; const float* log_rate; const float* skip;     // per head, DECAY_STEP (skip: any mode)
+  const float* rate;                           // per head, DECAY_CONSTANT
   int heads, groups, dk, dv;
   int ks, cols, chunk;                         // lanes per column, columns per block, staged tokens
   float inv_tau, q_scale;
@@ -74,7 +76,7 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(const DecayScanArgs a) 
   const int DKP = R * KS;                                    // key channels, padded to the lanes (a power of two)
   const int lg = 31 - __clz(DKP);
   const int ROW = padded(DKP);                               // floats from one token's row to the next
-  const size_t w_floats = MODE == DECAY_CHANNEL ? (size_t)CH * ROW : (size_t)2 * CH;
+  const size_t w_floats = MODE == DECAY_CHANNEL ? (size_t)CH * ROW : (MODE == DECAY_STEP ? (size_t)2 * CH : 0);
   const size_t buf_floats = ((size_t)2 * CH * ROW + w_floats + (size_t)CH * CB + 3) / 4 * 4;
   const int tid = threadIdx.x, nthreads = blockDim.x;
   const int s = tid % KS, jl = tid / KS;
@@ -92,6 +94,7 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(const DecayScanArgs a) 
   const float skip = a.skip ? a.skip[h] : 0.0f;
   const float rate = MODE == DECAY_STEP ? expf(a.log_rate[h]) : 0.0f;
   const float sbias = MODE == DECAY_STEP ? a.step_bias[h] : 0.0f;
+  const float constant = MODE == DECAY_CONSTANT ? a.rate[h] : 0.0f;
 
   auto fetch = [&](int t0, float* buf) {                     // the raw rows of tokens t0 .. t0 + m - 1 on their way
     const int m = min(CH, n - t0);
@@ -162,7 +165,7 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(const DecayScanArgs a) 
         sq[at] *= a.q_scale;
         if (MODE == DECAY_CHANNEL) {
           if (!a.ready) sw[at] = expf(log_sigmoid(sw[at]) * a.inv_tau);
-        } else {
+        } else if (MODE == DECAY_STEP) {
           sk[at] *= sw[CH + tt];
         }
       } else {                                               // padding: nothing is written, nothing is read out
@@ -185,7 +188,7 @@ __global__ void __launch_bounds__(256) decay_scan_kernel(const DecayScanArgs a) 
       for (int u = 0; u < U; ++u) {
         const int tu = tt + min(u, cnt - 1);
         vv[u] = (live && u < cnt) ? sv[tu * CB + jl] : 0.0f;
-        wall[u] = MODE == DECAY_STEP ? sw[tu] : 0.0f;
+        wall[u] = MODE == DECAY_STEP ? sw[tu] : constant;
         rowat[u] = tu * ROW + lane_at;
         acc[u] = 0.0f;
       }
@@ -296,21 +299,22 @@ int ifx_decay_scan_split(int dk, int* R_out, int* KS_out) {
 }
 
 // mode 0: a decay per key channel (raw [T, heads dk], tau); mode 1: a decay per head from a step size (raw [T, heads],
-// step_bias, log_rate per head; k is multiplied by the step).  skip (per head, may be null): out += skip v.
+// step_bias, log_rate per head; k is multiplied by the step); mode 2: a constant decay per head (rate; raw is not read).  skip (per head, may be null): out += skip v.
 // blocks_wanted: how many blocks the caller would like at least (the SMs to fill); value channels are cut over more
 // blocks while there are fewer.
 // scratch (may be null): room for the step's decays, num_tokens * heads * dk floats (mode 0) or num_tokens * 2 heads
 // (mode 1); with it, steps with long spans make their decays in a pass of their own over all SMs.
-int ifx_decay_scan(const float* q, long long q_stride, const float* k, long long k_stride, const float* v, long long v_stride,
+int ifx_decay_scan_rate(const float* q, long long q_stride, const float* k, long long k_stride, const float* v, long long v_stride,
                    const float* raw, long long raw_stride, float* state, long long state_slot_stride, const int* req_slot,
                    const int* cu_seqlens, float* out, const float* step_bias, const float* log_rate, const float* skip,
                    int num_requests, int num_tokens, int max_span, int heads, int groups, int dk, int dv, int mode, float tau,
-                   float q_scale, int blocks_wanted, float* scratch, cudaStream_t stream) {
+                   float q_scale, int blocks_wanted, float* scratch, const float* rate, cudaStream_t stream) {
   if (num_requests <= 0) return 0;
-  if (heads <= 0 || groups <= 0 || heads % groups || dk <= 0 || dv <= 0 || (mode != 0 && mode != 1) || max_span <= 0)
+  if (heads <= 0 || groups <= 0 || heads % groups || dk <= 0 || dv <= 0 || mode < 0 || mode > 2 || max_span <= 0)
     return IFX_E_BADARG;
   if (mode == 0 && !(tau > 0.0f)) return IFX_E_BADARG;
   if (mode == 1 && (step_bias == nullptr || log_rate == nullptr)) return IFX_E_BADARG;
+  if (mode == 2 && rate == nullptr) return IFX_E_BADARG;
   if (heads > 65535) return IFX_E_TOOBIG;
   int R = 0, KS = 0;
   const int rc = ifx_decay_scan_split(dk, &R, &KS);
@@ -320,8 +324,8 @@ int ifx_decay_scan(const float* q, long long q_stride, const float* k, long long
   // nothing and more blocks bring the states in sooner.
   int cols = 256 / KS;
   if (cols > dv) cols = dv;
-  const bool ready = scratch != nullptr && max_span >= 64;
-  if (ready) {
+  const bool ready = mode == 2 ? max_span >= 64 : scratch != nullptr && max_span >= 64;      // no decays to make while staging
+  if (ready && mode != 2) {
     const int per_row = mode == 0 ? heads * dk : heads;
     const size_t total = (size_t)num_tokens * per_row;
     const unsigned blocks = (unsigned)((total + 255) / 256 > 148 * 8 ? 148 * 8 : (total + 255) / 256);
@@ -350,19 +354,31 @@ int ifx_decay_scan(const float* q, long long q_stride, const float* k, long long
   a.q = q; a.q_stride = q_stride; a.k = k; a.k_stride = k_stride; a.v = v; a.v_stride = v_stride;
   a.raw = raw; a.raw_stride = raw_stride; a.state = state; a.state_slot_stride = state_slot_stride;
   a.req_slot = req_slot; a.cu_seqlens = cu_seqlens; a.out = out; a.step_bias = step_bias; a.log_rate = log_rate;
-  a.skip = skip; a.heads = heads; a.groups = groups; a.dk = dk; a.dv = dv; a.ks = KS; a.cols = cols; a.chunk = chunk;
+  a.skip = skip; a.rate = rate; a.heads = heads; a.groups = groups; a.dk = dk; a.dv = dv; a.ks = KS; a.cols = cols; a.chunk = chunk;
   a.inv_tau = mode == 0 ? 1.0f / tau : 0.0f;
   a.q_scale = q_scale;
   a.ready = ready ? 1 : 0;
   auto by16 = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-  a.vec = (dk % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && (mode == 1 || raw_stride % 4 == 0) && by16(q) && by16(k) &&
-           (mode == 1 || by16(raw))) ? 1 : 0;
+  a.vec = (dk % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && (mode != 0 || raw_stride % 4 == 0) && by16(q) && by16(k) &&
+           (mode != 0 || by16(raw))) ? 1 : 0;
   dim3 grid((unsigned)num_requests, (unsigned)heads, (unsigned)zsplits);
-  const int lrc = mode == 0 ? launch_decay_scan<DECAY_CHANNEL>(a, R, grid, threads, smem, stream)
-                            : launch_decay_scan<DECAY_STEP>(a, R, grid, threads, smem, stream);
+  const int lrc = mode == 0   ? launch_decay_scan<DECAY_CHANNEL>(a, R, grid, threads, smem, stream)
+                  : mode == 1 ? launch_decay_scan<DECAY_STEP>(a, R, grid, threads, smem, stream)
+                              : launch_decay_scan<DECAY_CONSTANT>(a, R, grid, threads, smem, stream);
   if (lrc) return lrc;
   IFX_CHECK_LAUNCH();
   return 0;
+}
+
+int ifx_decay_scan(const float* q, long long q_stride, const float* k, long long k_stride, const float* v, long long v_stride,
+                   const float* raw, long long raw_stride, float* state, long long state_slot_stride, const int* req_slot,
+                   const int* cu_seqlens, float* out, const float* step_bias, const float* log_rate, const float* skip,
+                   int num_requests, int num_tokens, int max_span, int heads, int groups, int dk, int dv, int mode, float tau,
+                   float q_scale, int blocks_wanted, float* scratch, cudaStream_t stream) {
+  if (mode != 0 && mode != 1) return IFX_E_BADARG;
+  return ifx_decay_scan_rate(q, q_stride, k, k_stride, v, v_stride, raw, raw_stride, state, state_slot_stride, req_slot, cu_seqlens,
+                             out, step_bias, log_rate, skip, num_requests, num_tokens, max_span, heads, groups, dk, dv, mode, tau,
+                             q_scale, blocks_wanted, scratch, nullptr, stream);
 }
 
 }  // extern "C"

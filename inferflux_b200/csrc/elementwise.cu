@@ -308,6 +308,17 @@ __global__ void scale_rows_kernel(const T* __restrict__ pre, const float* __rest
 // ------------------------------------------------------------------- SiLU*up
 // in [rows, 2*inter] = gate | up;  out[r, i] = silu(gate) * up, silu(g) = g / (1 + exp(-g)).
 template <typename T>
+__global__ void geglu_mul_kernel(const T* __restrict__ in, const float* __restrict__ bias, T* __restrict__ out, int inter, size_t total) {
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = idx / inter;
+    const int i = (int)(idx - r * inter);
+    const float g = to_f32(in[r * 2 * inter + i]) + (bias ? bias[i] : 0.0f);
+    const float u = to_f32(in[r * 2 * inter + inter + i]) + (bias ? bias[inter + i] : 0.0f);
+    out[idx] = from_f32<T>(gelu_tanh_f32(g) * u);
+  }
+}
+
+template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ in, T* __restrict__ out, int inter, size_t total) {
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= total) return;
@@ -561,6 +572,22 @@ int ifx_reduce_partial(const float* part, const float* bias, void* out, int rows
   else if (dtype == IFX_DT_BF16)
     reduce_partial_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(part, bias, (__nv_bfloat16*)out, total, cols,
                                                                      num_splits);
+  else
+    return IFX_E_DTYPE;
+  IFX_CHECK_LAUNCH();
+  return 0;
+}
+
+// gate_up [rows, 2 inter] (+ bias [2 inter], may be null) -> gelu_tanh(gate) * up, in the same dtype
+int ifx_geglu_mul(const void* gate_up, const float* bias, void* out, int rows, int inter, int dtype, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (inter <= 0) return IFX_E_BADARG;
+  const size_t total = (size_t)rows * inter;
+  const unsigned blocks = (unsigned)((total + 255) / 256 > 148 * 16 ? 148 * 16 : (total + 255) / 256);
+  if (dtype == IFX_DT_BF16)
+    geglu_mul_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gate_up, bias, (__nv_bfloat16*)out, inter, total);
+  else if (dtype == IFX_DT_F32)
+    geglu_mul_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gate_up, bias, (float*)out, inter, total);
   else
     return IFX_E_DTYPE;
   IFX_CHECK_LAUNCH();

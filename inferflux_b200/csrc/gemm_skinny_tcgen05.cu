@@ -17,7 +17,7 @@
 //                PARTIAL  part[split, m, n] = acc in float32, for consumers that add
 //                         the K slices themselves (residual + norm, bias + rotation),
 //                SWIGLU   two accumulators (gate rows and up rows of the same
-//                         outputs): out[m, n] = silu(gate) * up,
+//                         outputs): out[m, n] = silu(gate) * up, or gelu(gate + bias) * (up + bias),
 //                SWIGLU64 the same for a narrow product: 64 gate rows and 64 up rows share
 //                         one accumulator (lanes 0-63 and 64-127), so that twice as many
 //                         blocks stream the weights; the up half crosses to the gate half's
@@ -42,7 +42,8 @@ constexpr int kTileN = 128;       // weight rows per block (MMA M)
 constexpr int kTileK = 64;        // bf16 elements per k-block = one 128-byte swizzle row
 
 enum { MODE_STORE = 0, MODE_PARTIAL = 1, MODE_SWIGLU = 2, MODE_SWIGLU64 = 3 };
-enum { ACT_NONE = 0, ACT_XIELU = 1 };                  // an activation on the stored result of MODE_STORE
+// an activation on the stored result of MODE_STORE, or (GEGLU) in place of SiLU on the gate of MODE_SWIGLU / SWIGLU64
+enum { ACT_NONE = 0, ACT_XIELU = 1, ACT_GEGLU = 2 };
 
 __device__ __forceinline__ uint64_t make_smem_desc(uint32_t addr) {
   // K-major tile of 128-byte rows, 128-byte swizzle: 8-row groups 1024 bytes apart.
@@ -216,7 +217,9 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
     if (!ok && lane == 0) atomicExch(error_flag, 3);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    const float b = (MODE == MODE_STORE && bias != nullptr && n < N) ? bias[n] : 0.0f;
+    constexpr bool GLU = MODE == MODE_SWIGLU || MODE == MODE_SWIGLU64;
+    const float b = ((MODE == MODE_STORE || GLU) && bias != nullptr && n < N) ? bias[n] : 0.0f;
+    const float b_up = (GLU && bias != nullptr && n < N) ? bias[up_row_offset + n] : 0.0f;
 #pragma unroll
     for (int c = 0; c < NPAD; c += 16) {
       if (c >= M) break;                                         // uniform over the block
@@ -249,14 +252,16 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
           if (m >= M) break;
           const float rs = row_sumsq != nullptr ? row_scale[m] : 1.0f;
           float v = __uint_as_float(g[j]) * rs;
-          if (MODE == MODE_SWIGLU || MODE == MODE_SWIGLU64) {
-            const float up = __uint_as_float(u[j]) * rs;
-            v = __fdividef(v, 1.0f + __expf(-v)) * up;       // a few float32 ulps, far below the bfloat16 rounding
+          if (GLU) {
+            const float up = __uint_as_float(u[j]) * rs + b_up;
+            v += b;
+            v = (act_kind == ACT_GEGLU ? gelu_tanh_fast(v)
+                                       : __fdividef(v, 1.0f + __expf(-v))) * up;     // a few float32 ulps, far below the bfloat16 rounding
           }
           if (MODE == MODE_PARTIAL) {
             partials[((size_t)split * M + m) * N + n] = v;
           } else {
-            float r = v + b;
+            float r = GLU ? v : v + b;
             if (MODE == MODE_STORE && act_kind == ACT_XIELU)     // a z^2 + z/2 above zero, b (e^z - 1 - z) + z/2 below
               r = r > 0.0f ? fmaf(act_a * r, r, 0.5f * r) : fmaf(act_b, (__expf(r) - 1.0f) - r, 0.5f * r);
             if (out_is_f32) reinterpret_cast<float*>(out)[(size_t)m * N + n] = r;
@@ -366,7 +371,8 @@ static int gemm_skinny_any(const void* act, const void* W, const float* bias, vo
                           const float* row_sumsq, int sumsq_chunks, float eps, int* error_flag, cudaStream_t stream,
                           int act_kind, float act_a, float act_b) {
   if (M <= 0 || N <= 0) return 0;
-  if (act_kind != ACT_NONE && (act_kind != ACT_XIELU || mode != MODE_STORE)) return IFX_E_BADARG;
+  if (act_kind != ACT_NONE && !(act_kind == ACT_XIELU && mode == MODE_STORE) && !(act_kind == ACT_GEGLU && mode == MODE_SWIGLU))
+    return IFX_E_BADARG;
   if (K <= 0 || M > 256 || splits <= 0 || splits > 65535 || error_flag == nullptr) return IFX_E_BADARG;
   if (mode == MODE_STORE && splits != 1) return IFX_E_BADARG;
   if (mode == MODE_SWIGLU && (splits != 1 || out_is_f32)) return IFX_E_BADARG;
@@ -414,4 +420,12 @@ extern "C" int ifx_gemm_skinny_act(const void* act, const void* W, const float* 
                                    int act_kind, float act_a, float act_b, int* error_flag, cudaStream_t stream) {
   return gemm_skinny_any(act, W, bias, out, nullptr, M, N, K, w_rows, 1, MODE_STORE, 0, out_is_f32, row_sumsq,
                          sumsq_chunks, eps, error_flag, stream, act_kind, act_a, act_b);
+}
+
+// mode 2 with the tanh form of gelu on the gate and biases: W holds N gate rows at 0 and N up rows at N, bias (may be null)
+// [2 N] likewise; out[M, N] = gelu(act . Wg^T + bg) * (act . Wu^T + bu), bfloat16.
+extern "C" int ifx_gemm_skinny_geglu(const void* act, const void* W, const float* bias, void* out, int M, int N, int K,
+                                     int* error_flag, cudaStream_t stream) {
+  return gemm_skinny_any(act, W, bias, out, nullptr, M, N, K, 2 * N, 1, MODE_SWIGLU, N, 0, nullptr, 0, 0.0f, error_flag, stream,
+                         ACT_GEGLU, 0.0f, 0.0f);
 }

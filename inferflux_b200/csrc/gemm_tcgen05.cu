@@ -6,6 +6,7 @@
 //   SWIGLU   W holds N gate rows and, `up_row_offset` rows further, N up rows;
 //            out[m, n] = silu(acc_gate) * acc_up               (bfloat16; no [M, 2N] round trip,
 //                                                               no separate activation kernel)
+//   GEGLU    the same with gelu(acc_gate + bias) * (acc_up + bias), the tanh form
 //   GROUP_RELU2  rows are sorted into groups of whole 128-row tiles; tile mt multiplies with the weight rows
 //            [tile_group[mt] * group_rows, + N) of a stack of matrices (a negative entry: the tile is unused and
 //            skipped);  out[m, n] = relu(acc)^2                 (bfloat16)
@@ -34,7 +35,7 @@ namespace ifx {
 constexpr int kBM = 128, kBN = 256, kBK = 64, kGemmStages = 4;
 constexpr uint32_t kABytes = kBM * kBK * 2, kBBytes = kBN * kBK * 2, kStageBytes = kABytes + kBBytes;
 
-enum { GEMM_STORE = 0, GEMM_SWIGLU = 1, GEMM_GROUP_RELU2 = 2, GEMM_GROUP_SCALE = 3, GEMM_GROUP_GLU = 4 };
+enum { GEMM_STORE = 0, GEMM_SWIGLU = 1, GEMM_GROUP_RELU2 = 2, GEMM_GROUP_SCALE = 3, GEMM_GROUP_GLU = 4, GEMM_GEGLU = 5 };
 
 __device__ __forceinline__ uint64_t gemm_smem_desc(uint32_t addr) {
   // K-major tile of 128-byte rows, 128-byte swizzle: 8-row groups 1024 bytes apart.
@@ -72,8 +73,9 @@ __global__ void __launch_bounds__(192, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     __nv_bfloat16* __restrict__ out, int M, int N, int K, int up_row_offset, int m_tiles, int n_tiles,
                     int* __restrict__ error_flag, const int* __restrict__ tile_group, int group_rows,
-                    const float* __restrict__ row_scale, float glu_limit, float glu_slope, float glu_offset) {
-  constexpr bool PAIRED = MODE == GEMM_SWIGLU || MODE == GEMM_GROUP_GLU;   // a tile is 128 gate rows and their 128 up rows
+                    const float* __restrict__ row_scale, float glu_limit, float glu_slope, float glu_offset,
+                    const float* __restrict__ bias) {
+  constexpr bool PAIRED = MODE == GEMM_SWIGLU || MODE == GEMM_GEGLU || MODE == GEMM_GROUP_GLU;   // a tile is 128 gate rows and their 128 up rows
   constexpr int OUT_COLS = PAIRED ? kBN / 2 : kBN;                  // output columns a tile makes
   constexpr bool GROUPED = MODE == GEMM_GROUP_RELU2 || MODE == GEMM_GROUP_SCALE || MODE == GEMM_GROUP_GLU;
   extern __shared__ unsigned char smem_raw[];
@@ -204,6 +206,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         for (int j = 0; j < 16; ++j) {
           v[j] = __uint_as_float(g[j]);
           if (MODE == GEMM_SWIGLU) v[j] = __fdividef(v[j], 1.0f + __expf(-v[j])) * __uint_as_float(u[j]);
+          if (MODE == GEMM_GEGLU) {
+            const int n = min(n0 + c + j, N - 1);                     // the last tile may hang over
+            const float bg = bias ? bias[n] : 0.0f, bu = bias ? bias[N + n] : 0.0f;
+            v[j] = gelu_tanh_fast(v[j] + bg) * (__uint_as_float(u[j]) + bu);
+          }
           if (MODE == GEMM_GROUP_GLU) {                               // g sigmoid(slope g) (u + 1), g cut from above, u on both sides
             const float gate = fminf(v[j], glu_limit);
             const float up = fminf(fmaxf(__uint_as_float(u[j]), -glu_limit), glu_limit);
@@ -262,8 +269,9 @@ static int gemm_sm_count() {
 template <int MODE>
 static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mw, void* out, int M, int N, int K, int up_row_offset,
                        int* error_flag, cudaStream_t stream, const int* tile_group = nullptr, int group_rows = 0,
-                       const float* row_scale = nullptr, float glu_limit = 0.0f, float glu_slope = 0.0f, float glu_offset = 1.0f) {
-  constexpr int OUT_COLS = (MODE == GEMM_SWIGLU || MODE == GEMM_GROUP_GLU) ? kBN / 2 : kBN;
+                       const float* row_scale = nullptr, float glu_limit = 0.0f, float glu_slope = 0.0f, float glu_offset = 1.0f,
+                       const float* bias = nullptr) {
+  constexpr int OUT_COLS = (MODE == GEMM_SWIGLU || MODE == GEMM_GEGLU || MODE == GEMM_GROUP_GLU) ? kBN / 2 : kBN;
   const size_t smem = 1024 + (size_t)kGemmStages * kStageBytes + (2 * kGemmStages + 4) * 8 + 16;
   static bool configured = false;
   if (!configured) {
@@ -276,7 +284,7 @@ static int launch_gemm(const CUtensorMap& ma, const CUtensorMap& mw, void* out, 
   const int grid = tiles < gemm_sm_count() ? tiles : gemm_sm_count();
   gemm_tcgen05_kernel<MODE><<<grid, 192, smem, stream>>>(ma, mw, reinterpret_cast<__nv_bfloat16*>(out), M, N, K,
                                                          up_row_offset, m_tiles, n_tiles, error_flag, tile_group,
-                                                         group_rows, row_scale, glu_limit, glu_slope, glu_offset);
+                                                         group_rows, row_scale, glu_limit, glu_slope, glu_offset, bias);
   IFX_CHECK_LAUNCH();
   return 0;
 }
@@ -349,4 +357,17 @@ extern "C" int ifx_gemm_tcgen05_grouped_glu(const void* act, const void* W, void
                                             const int* tile_group, float limit, float slope, int* error_flag,
                                             cudaStream_t stream) {
   return ifx_gemm_tcgen05_grouped_glu_offset(act, W, out, M, ff, K, groups, tile_group, limit, slope, 1.0f, error_flag, stream);
+}
+
+// out [M, N] bfloat16 = gelu(act . W[:N]^T + bias[:N]) * (act . W[N:]^T + bias[N:]), the tanh form; W [2 N, K], bias [2 N] or null.
+extern "C" int ifx_gemm_tcgen05_geglu(const void* act, const void* W, const float* bias, void* out, int M, int N, int K,
+                                      int* error_flag, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K <= 0 || K % 8 || error_flag == nullptr || out == nullptr) return IFX_E_BADARG;
+  CUtensorMap ma, mw;
+  int rc = weight_tensor_map(&mw, W, 2 * N, K, 128);
+  if (rc) return rc;
+  rc = make_tensor_map_bf16(&ma, act, M, K, kBM);
+  if (rc) return rc;
+  return launch_gemm<GEMM_GEGLU>(ma, mw, out, M, N, K, N, error_flag, stream, nullptr, 0, nullptr, 0.0f, 0.0f, 1.0f, bias);
 }

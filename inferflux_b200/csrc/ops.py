@@ -163,7 +163,9 @@ class CudaKernels:
                    "ifx_moe_route_kind", "ifx_moe_experts_glu", "ifx_gemm_tcgen05_grouped_glu_offset", "ifx_norm_rope_append_ex",
                    "ifx_attention_generic_sink", "ifx_short_conv_ex", "ifx_decay_scan", "ifx_decay_scan_split", "ifx_bigram_add",
                    "ifx_rmsnorm_pair", "ifx_gate_mul", "ifx_gated_groupnorm", "ifx_pair_combine", "ifx_residual_add_vectors",
-                   "ifx_attention_prefill_tcgen05_sink", "ifx_attention_prefill_bf16_sink", "ifx_attention_decode_bf16_sink"):
+                   "ifx_attention_prefill_tcgen05_sink", "ifx_attention_prefill_bf16_sink", "ifx_attention_decode_bf16_sink",
+                   "ifx_norm_of_sum", "ifx_row_norm_rope_append", "ifx_rotate_rows", "ifx_gated_scan", "ifx_decay_scan_rate",
+                   "ifx_geglu_mul", "ifx_gemm_skinny_geglu", "ifx_gemm_tcgen05_geglu"):
             getattr(self.lib, fn).restype = ctypes.c_int
         self.lib.ifx_delta_rule_scratch_floats.restype = ctypes.c_longlong
         self.lib.ifx_sample_scratch_bytes.restype = ctypes.c_longlong
@@ -410,6 +412,30 @@ class CudaKernels:
                 and a.data_ptr() % 16 == 0 and w_gate_up.data_ptr() % 16 == 0 and a.is_contiguous()):
             return self.linear_tiles(a, w_gate_up, swiglu=True)        # many rows: own tcgen05 tiles, activation fused
         return self.silu_mul(self.linear(a, w_gate_up))
+
+    def linear_geglu(self, a, w_gate_up, bias):
+        """gelu_tanh(a . Wg^T + bg) * (a . Wu^T + bu) with Wg and Wu stacked in w_gate_up [2 I, K] and the biases (float32, or
+        None) likewise: the activation in the product's epilogue as in `linear_swiglu`, else the product followed by the
+        activation kernel."""
+        T, K = a.shape
+        inter = w_gate_up.shape[0] // 2
+        _need(a.dtype == w_gate_up.dtype and w_gate_up.shape[1] == K and a.is_contiguous() and w_gate_up.is_contiguous()
+              and (bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * inter)),
+              "linear_geglu: bad operands")
+        if (T and a.dtype == torch.bfloat16 and K % 8 == 0 and a.data_ptr() % 16 == 0 and w_gate_up.data_ptr() % 16 == 0):
+            few = T <= self.SKINNY_MAX_ROWS
+            if few or (self.swiglu_tiles and K <= self.SWIGLU_TILES_MAX_K):
+                out = torch.empty((T, inter), dtype=torch.bfloat16, device=a.device)
+                product = self.lib.ifx_gemm_skinny_geglu if few else self.lib.ifx_gemm_tcgen05_geglu
+                _check(product(_ptr(a), _ptr(w_gate_up), _ptr(bias), _ptr(out), T, inter, K, _ptr(self.error_flag), _stream()),
+                       "linear_geglu")
+                self.launches += 1
+                return out
+        both = self.linear(a, w_gate_up)
+        out = torch.empty((T, inter), dtype=a.dtype, device=a.device)
+        _check(self.lib.ifx_geglu_mul(_ptr(both), _ptr(bias), _ptr(out), T, inter, _DT[a.dtype], _stream()), "geglu_mul")
+        self.launches += 1
+        return out
 
     def linear_xielu(self, a, w, a_pos, a_neg):
         """xielu(a . w^T): for few bfloat16 rows and a product wide enough to fill the SMs without K slices, the
@@ -726,17 +752,19 @@ class CudaKernels:
         self.launches += 1
         return q_out
 
-    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None):
+    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None, turn_back=None):
         """Every token attends its request's keys up to its own position (or the last
         `window` of them) through the block table.  float32: the per-token kernel
         whose additions depend on the position only.  bfloat16: the tiled kernels,
         one launch for the prompt portions and one for the single decoded tokens.
         `chunk`: a query at position p sees keys from (p // chunk) * chunk on; `sink`: one more unit in the
         softmax's denominator (True), or exp of a learned number per head (a float32 tensor [nq]); `dv`: the values'
-        head size if it is not `d`."""
-        if (chunk or torch.is_tensor(sink) or sink or (dv is not None and dv != d)
+        head size if it is not `d`; `turn_back`: what `row_norm_rope_append` returned for values that were turned, so that
+        every head's output is turned back by the query's position before it is rounded."""
+        if (turn_back is not None or chunk or torch.is_tensor(sink) or sink or (dv is not None and dv != d)
                 or (cache.kv is not None and cache.kv.shape[-1] != d)):      # cache rows longer than a head
-            return self._attention_masked(q, nq, nkv, d, d if dv is None else dv, window, chunk, sink, scale, ctx, cache)
+            return self._attention_masked(q, nq, nkv, d, d if dv is None else dv, window, chunk, sink, scale, ctx, cache,
+                                          turn_back)
         T = q.shape[0]
         kv, table = cache.kv, cache.block_table
         _need(kv is not None and table is not None, "attention: the mixer has no key/value cache")
@@ -797,8 +825,9 @@ class CudaKernels:
             splits = 8
         return splits
 
-    def _attention_masked(self, q, nq, nkv, d, dv, window, chunk, sink, scale, ctx, cache):
-        """Attention with a chunk mask, a sink or values of their own size: the per-token kernel."""
+    def _attention_masked(self, q, nq, nkv, d, dv, window, chunk, sink, scale, ctx, cache, turn_back=None):
+        """Attention with a chunk mask, a sink, values of their own size or turned values: the tiled kernels where they take
+        the sizes, else the per-token kernel."""
         T = q.shape[0]
         kv, table = cache.kv, cache.block_table
         _need(kv is not None and table is not None, "attention: the mixer has no key/value cache")
@@ -813,6 +842,9 @@ class CudaKernels:
         if sink_values is not None:
             _need(sink_values.dtype == torch.float32 and sink_values.numel() == nq and sink_values.is_contiguous(),
                   "attention: the learned sink is float32 [heads]")
+        back, neighbours = (None, 0) if turn_back is None else (turn_back[0], int(bool(turn_back[1])))
+        _need(back is None or (back.dtype == torch.float32 and back.is_contiguous() and tuple(back.shape) == (T, dv // 2, 2)),
+              "attention: cos and sin of the values' angles are float32 [tokens, dv / 2, 2]")
         if (q.dtype == torch.bfloat16 and d == dv == d_row and nq // nkv <= 16 and self.lib.ifx_attention_mma_supports(d)
                 and os.environ.get("INFERFLUX_B200_MASKED_TILES", "1") != "0"):
             # the tiled kernels: prompt portions on mma.sync tiles, single tokens on the cluster kernel
@@ -822,7 +854,7 @@ class CudaKernels:
                     ctx.extra_len[name] = len(vals)
             num_tiles = ctx.extra_len["attn.prefill_tiles"] // 4
             common = (cache.page_size, table.shape[1], kv.shape[0], win, int(chunk or 0),
-                      int(sink_values is not None or bool(sink)), _ptr(sink_values), ctypes.c_float(scale))
+                      int(sink_values is not None or bool(sink)), _ptr(sink_values), ctypes.c_float(scale), _ptr(back), neighbours)
             if num_tiles and self.tensor_core_prefill and self.lib.ifx_attention_prefill_tcgen05_supports(d, cache.page_size):
                 _check(self.lib.ifx_attention_prefill_tcgen05_sink(
                     _ptr(q), T, _ptr(kv), _ptr(table), _ptr(ctx.extra["attn.prefill_tiles"]), _ptr(ctx.req_slot), _ptr(out),
@@ -852,7 +884,7 @@ class CudaKernels:
             _ptr(q), _ptr(kv), _ptr(table), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(ctx.req_slot), _ptr(None),
             _ptr(out), T, nq, nkv, d, dv, d_row, cache.page_size, table.shape[1], kv.shape[0],
             0 if window is None else int(window), int(chunk or 0), int(sink_values is not None or bool(sink)),
-            _ptr(sink_values), ctypes.c_float(scale), _DT[q.dtype], _stream()), "attention (masked)")
+            _ptr(sink_values), ctypes.c_float(scale), _ptr(back), neighbours, _DT[q.dtype], _stream()), "attention (masked)")
         self.launches += 1
         return out
 
@@ -1450,48 +1482,53 @@ class CudaKernels:
         return ctypes.c_void_p(t.data_ptr()), ctypes.c_longlong(t.stride(0))
 
     def decay_scan(self, q, k, v, raw, state, ctx, heads, groups, dk, dv, decay, tau=1.0, q_scale=1.0, step_bias=None,
-                   log_rate=None, skip=None):
+                   log_rate=None, skip=None, rate=None):
         """Per request and head a float32 matrix S, kept in `state` [slots, >= heads dv dk] as [head, value channel, key
         channel]: S <- diag(w_t) S + k_t v_t^T, o_t = S^T (q_scale q_t) with the new S.  q, k: float32 [T, groups dk]
         (head h reads group h // (heads / groups)); v: [T, heads dv]; rows may be slices of wider rows.  Returns
         float32 [T, heads dv].
         decay `sigmoid_root`: raw [T, heads dk], w = sigmoid(raw)^(1/tau).
         decay `softplus_step`: raw [T, heads], dt = softplus(raw + step_bias), w = exp(-exp(log_rate) dt) for the whole
-        head, k is multiplied by dt, and skip[h] v_t is added to o_t."""
+        head, k is multiplied by dt, and skip[h] v_t is added to o_t.
+        decay `constant`: raw None, w = rate[h] whatever the token."""
         T = q.shape[0]
-        _need(decay in ("sigmoid_root", "softplus_step"), f"decay_scan: unknown decay {decay!r}")
-        mode = 0 if decay == "sigmoid_root" else 1
+        modes = {"sigmoid_root": 0, "softplus_step": 1, "constant": 2}
+        _need(decay in modes, f"decay_scan: unknown decay {decay!r}")
+        mode = modes[decay]
+        _need((raw is None) == (mode == 2) == (rate is not None), "decay_scan: a constant decay comes from `rate`, any other from `raw`")
         _need(q.shape[1] == groups * dk and k.shape[1] == groups * dk and v.shape[1] == heads * dv
-              and raw.shape[1] == (heads * dk if mode == 0 else heads) and k.shape[0] == T and v.shape[0] == T and raw.shape[0] == T,
+              and k.shape[0] == T and v.shape[0] == T
+              and (raw is None or tuple(raw.shape) == (T, heads * dk if mode == 0 else heads)),
               "decay_scan: the rows do not fit the head counts")
         _need(state is not None and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * dv * dk,
               "decay_scan: the state does not fit the heads")
-        for vec in (step_bias, log_rate, skip):
+        for vec in (step_bias, log_rate, skip, rate):
             _need(vec is None or (vec.dtype == torch.float32 and vec.numel() == heads and vec.is_contiguous()),
                   "decay_scan: per-head vectors are float32 [heads]")
         out = torch.empty((T, heads * dv), dtype=torch.float32, device=q.device)
         scratch = None                                     # steps with long spans make their decays in a pass of their own
-        if ctx.max_span >= 64:
+        if ctx.max_span >= 64 and mode != 2:
             scratch = torch.empty(T * (heads * dk if mode == 0 else 2 * heads), dtype=torch.float32, device=q.device)
-        _check(self.lib.ifx_decay_scan(*self._rows_f32(q, "decay_scan q"), *self._rows_f32(k, "decay_scan k"),
-                                       *self._rows_f32(v, "decay_scan v"), *self._rows_f32(raw, "decay_scan raw"), _ptr(state),
+        _check(self.lib.ifx_decay_scan_rate(*self._rows_f32(q, "decay_scan q"), *self._rows_f32(k, "decay_scan k"),
+                                       *self._rows_f32(v, "decay_scan v"),
+                                       *(self._rows_f32(raw, "decay_scan raw") if raw is not None else (_ptr(None), _LL(0))), _ptr(state),
                                        ctypes.c_longlong(state.stride(0)), _ptr(ctx.req_slot), _ptr(ctx.cu_seqlens), _ptr(out),
                                        _ptr(step_bias), _ptr(log_rate), _ptr(skip), ctx.num_requests, T, int(ctx.max_span), int(heads),
                                        int(groups), int(dk), int(dv), mode, ctypes.c_float(tau), ctypes.c_float(q_scale), 296,
-                                       _ptr(scratch), _stream()), "decay_scan")
+                                       _ptr(scratch), _ptr(rate), _stream()), "decay_scan")
         self.launches += 1 + int(scratch is not None)
         return out
 
     def gated_groupnorm(self, y, gate, w, eps, groups, gate_first, out_dtype):
         """Rows of y (float32 [T, C]) in `groups` equal parts, each over its own root mean square, times w (of size C, or
-        of a part's size and then the same for every part) and silu(gate) (float32 rows, maybe a slice of wider ones):
+        of a part's size and then the same for every part; None: no weight) and silu(gate) (float32 rows, maybe a slice of wider ones):
         the gate multiplies before the norm (`gate_first`) or behind it."""
         T, C = y.shape
-        _need(y.dtype == torch.float32 and y.is_contiguous() and tuple(gate.shape) == (T, C) and w.dtype == torch.float32
-              and w.is_contiguous() and C % groups == 0 and w.numel() in (C, C // groups), "gated_groupnorm: bad operands")
+        _need(y.dtype == torch.float32 and y.is_contiguous() and tuple(gate.shape) == (T, C) and C % groups == 0
+              and (w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() in (C, C // groups))), "gated_groupnorm: bad operands")
         out = torch.empty((T, C), dtype=out_dtype, device=y.device)
         gp, gs = self._rows_f32(gate, "gated_groupnorm gate")
-        _check(self.lib.ifx_gated_groupnorm(_ptr(y), gp, gs, _ptr(w), int(w.numel()), ctypes.c_float(eps), _ptr(out), T, C,
+        _check(self.lib.ifx_gated_groupnorm(_ptr(y), gp, gs, _ptr(w), 0 if w is None else int(w.numel()), ctypes.c_float(eps), _ptr(out), T, C,
                                             int(groups), int(bool(gate_first)), _DT[out_dtype], _stream()), "gated_groupnorm")
         self.launches += 1
         return out
@@ -1522,6 +1559,108 @@ class CudaKernels:
                                                  _DT[b.dtype] if b is not None else 0, _ptr(s_b), T, C, _stream()),
                "residual_add_vectors")
         self.launches += 1
+
+    # ------------------------------------------- norms of sums, rotated rows, an elementwise recurrence
+    def norm_of_sum(self, x, alpha, terms, w, eps, out_dtype=None):
+        """x <- n(alpha x + sum c (y + bias)), float32 and in place, for one or two terms (c, y, bias): y a tensor or a
+        PartialSum, bias float32 along the row or None; n the RMS norm times w (w None: x is the sum itself).  With
+        `out_dtype` also returns the new rows in that dtype."""
+        T, H = x.shape
+        _need(x.dtype == torch.float32 and x.is_contiguous() and 1 <= len(terms) <= 2
+              and (w is None or (w.dtype == torch.float32 and w.numel() == H and w.is_contiguous())), "norm_of_sum: bad operands")
+        flat = []
+        for c, y, bias in list(terms) + [(0.0, None, None)] * (2 - len(terms)):
+            splits = 1
+            if isinstance(y, PartialSum):
+                _need(tuple(y.shape) == (T, H), "norm_of_sum: partial sums do not match x")
+                y, splits = y.parts, y.splits
+            _need((y is None or (tuple(y.shape[-2:]) == (T, H) and y.is_contiguous()))
+                  and (bias is None or (bias.dtype == torch.float32 and bias.numel() == H and bias.is_contiguous())),
+                  "norm_of_sum: a term does not match x")
+            flat += [_ptr(y), 0 if y is None else _DT[y.dtype], splits, ctypes.c_float(c), _ptr(bias)]
+        out = None if out_dtype is None else torch.empty((T, H), dtype=out_dtype, device=x.device)
+        _check(self.lib.ifx_norm_of_sum(_ptr(x), ctypes.c_float(alpha), *flat, _ptr(w), ctypes.c_float(eps), _ptr(out),
+                                        0 if out is None else _DT[out_dtype], T, H, _stream()), "norm_of_sum")
+        self.launches += 1
+        return out
+
+    def joins_projections(self, h):
+        """Whether two stacked projections of the same rows run as one product: for few bfloat16 rows, where the time is the
+        weights' way in; with many rows each keeps an output dtype of its own."""
+        return h.dtype == torch.bfloat16 and h.shape[0] <= self.SKINNY_MAX_ROWS
+
+    @staticmethod
+    def _row_source(rows):
+        """(plain pointer, dtype code, partial pointer, splits, row length) of a tensor or PartialSum."""
+        if isinstance(rows, PartialSum):
+            return _ptr(None), 0, _ptr(rows.parts), rows.splits, rows.parts.shape[-1]
+        _need(rows.is_contiguous(), "projected rows must be contiguous")
+        return _ptr(rows), _DT[rows.dtype], _ptr(None), 1, rows.shape[-1]
+
+    def row_norm_rope_append(self, rows, col0, bias, rotary, turn, temp, nq, nkv, d, dv, ctx, cache, q_norm=None, k_norm=None,
+                             norm_eps=0.0):
+        """Columns col0 .. of `rows` (a tensor or PartialSum): [nq heads of d | nkv key heads of d | nkv value heads of dv],
+        plus `bias`; the query part and the key part RMS-normed as a whole (weights of their full size; None: no norm),
+        turned by `rotary`, the queries times `temp` per head; the values turned by `turn` over their whole heads; keys and
+        values to the cache.  Returns (queries [T, nq d] in the cache's dtype, what `attention` takes as `turn_back`)."""
+        T = rows.shape[0]
+        kv, table = cache.kv, cache.block_table
+        _need(kv is not None and table is not None and kv.shape[1] == 2 and kv.shape[2] == nkv and kv.shape[-1] >= max(d, dv),
+              "row_norm_rope_append: the cache does not fit the heads")
+        for v, n in ((bias, nq * d + nkv * (d + dv)), (q_norm, nq * d), (k_norm, nkv * d), (temp, nq)):
+            _need(v is None or (v.dtype == torch.float32 and v.numel() == n and v.is_contiguous()),
+                  "row_norm_rope_append: biases, norm weights and factors are float32 of their full size")
+        for table_, size in ((rotary, d), (turn, dv)):
+            _need(table_ is None or (table_.magnitude == 1.0 and table_.rotary_dim <= size), "row_norm_rope_append: a table does not fit")
+        _need(turn is None or turn.rotary_dim == dv, "row_norm_rope_append: values are turned as a whole")
+        src, code, part, splits, ld = self._row_source(rows)
+        dev = kv.device
+        q_out = torch.empty((T, nq * d), dtype=kv.dtype, device=dev)
+        back = None if turn is None else torch.empty((T, dv // 2, 2), dtype=torch.float32, device=dev)
+        _check(self.lib.ifx_row_norm_rope_append(
+            src, code, part, splits, _LL(ld), int(col0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), ctypes.c_float(norm_eps),
+            _ptr(None if rotary is None else rotary.inv_freq), 0 if rotary is None else int(rotary.rotary_dim),
+            int(rotary is not None and rotary.interleaved), _ptr(None if turn is None else turn.inv_freq),
+            int(turn is not None and turn.interleaved), _ptr(temp), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(ctx.req_slot),
+            _ptr(table), table.shape[1], cache.page_size, kv.shape[0], _ptr(kv), _ptr(q_out), _ptr(back), T, nq, nkv, d, dv,
+            kv.shape[-1], int(bool(cache.writes)), _DT[kv.dtype], _stream()), "row_norm_rope_append")
+        self.launches += 1
+        return q_out, (None if back is None else (back, turn.interleaved))
+
+    def rotate_rows(self, rows, col0, width, heads, dk, rotary, k_scale, ctx):
+        """float32 [T, width] from columns col0 .. of `rows` (a float32 tensor, which is then changed in place where it has
+        just these columns, or a PartialSum): heads of dk (queries), heads of dk (keys), the rest; queries and keys turned
+        by the position, keys times k_scale behind it."""
+        T = rows.shape[0]
+        src, code, part, splits, ld = self._row_source(rows)
+        plain = not isinstance(rows, PartialSum)
+        _need(not plain or rows.dtype == torch.float32, "rotate_rows: float32 rows")
+        _need(rotary is None or (rotary.magnitude == 1.0 and rotary.rotary_dim <= dk), "rotate_rows: the table does not fit")
+        device = rows.device if plain else rows.parts.device
+        out = rows if plain and ld == width and col0 == 0 else torch.empty((T, width), dtype=torch.float32, device=device)
+        _check(self.lib.ifx_rotate_rows(
+            src, part, splits, _LL(ld), int(col0), _ptr(None if rotary is None else rotary.inv_freq),
+            0 if rotary is None else int(rotary.rotary_dim), int(rotary is not None and rotary.interleaved), _ptr(ctx.positions),
+            _ptr(out), T, int(width), int(heads), int(dk), ctypes.c_float(k_scale), _stream()), "rotate_rows")
+        self.launches += 1
+        return out
+
+    def gated_scan(self, rows, bias, state, width, ctx, out_dtype):
+        """rows [T, 3 width] (float32 or PartialSum) = z, x, g; `bias` (float32 [2 width]) joins z and x:
+        S <- (1 - sigmoid(z)) S + sigmoid(z) c with c = x + 1/2 where x >= 0 and sigmoid(x) where x < 0; returns S silu(g) in
+        `out_dtype`.  S per request in `state` (float32 [slots, >= width]), moved on."""
+        T = rows.shape[0]
+        _need(tuple(rows.shape) == (T, 3 * width) and bias.dtype == torch.float32 and bias.numel() == 2 * width
+              and state is not None and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= width,
+              "gated_scan: bad operands")
+        src, splits = (rows.parts, rows.splits) if isinstance(rows, PartialSum) else (rows, 1)
+        _need(src.dtype == torch.float32 and src.is_contiguous(), "gated_scan: float32 rows")
+        out = torch.empty((T, width), dtype=out_dtype, device=src.device)
+        _check(self.lib.ifx_gated_scan(_ptr(src), splits, _ptr(bias), _ptr(state), _LL(state.stride(0)), _ptr(ctx.req_slot),
+                                       _ptr(ctx.cu_seqlens), _ptr(out), ctx.num_requests, T, int(ctx.max_span), int(width),
+                                       _DT[out_dtype], _stream()), "gated_scan")
+        self.launches += 1
+        return out
 
     # ---------------------------------------------------------------- sampling
     def argmax(self, logits):

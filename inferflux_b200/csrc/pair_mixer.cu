@@ -4,7 +4,7 @@
 //                         the token before a span's first one is the request's state, which takes the span's last token
 //   rmsnorm_pair          two RMS norms of the same float32 rows (one sum of squares, two weights)
 //   gate_mul              a * sigmoid(g) or a * silu(g)
-//   gated_groupnorm       rows in equal parts, each over its own root mean square, times a weight and silu(gate), the
+//   gated_groupnorm       rows in equal parts, each over its own root mean square, times a weight (or none) and silu(gate), the
 //                         gate in front of the norm or behind it
 //   pair_combine          c_a a + c_b b, or c_a a / rms(a) * w_a + c_b b / rms(b) * w_b; the result is float32
 //   residual_add_vectors  x += s_a * a + s_b * (b + b2), vectors along the row
@@ -122,7 +122,7 @@ __global__ void __launch_bounds__(256) gated_groupnorm_kernel(const float* __res
       const float sg = gv / (1.0f + expf(-gv));
       float v = yr[c];
       if (gate_first) v *= sg;
-      v = v * inv * w[w_size == C ? c : e];
+      v = v * inv * (w ? w[w_size == C ? c : e] : 1.0f);
       if (!gate_first) v *= sg;
       store_from_f32(out, out_dtype, (size_t)t * C + c, v);
     }
@@ -158,7 +158,7 @@ __global__ void __launch_bounds__(512) gated_groupnorm_wide_kernel(const float* 
       const float sg = gv / (1.0f + expf(-gv));
       float v = yr[c];
       if (gate_first) v *= sg;
-      v = v * inv * w[w_size == C ? c : e];
+      v = v * inv * (w ? w[w_size == C ? c : e] : 1.0f);
       if (!gate_first) v *= sg;
       store_from_f32(out, out_dtype, (size_t)t * C + c, v);
     }
@@ -262,7 +262,7 @@ int ifx_gate_mul(const void* a, const void* g, void* out, long long total, int d
 int ifx_gated_groupnorm(const float* y, const float* gate, long long gate_stride, const float* w, int w_size, float eps,
                         void* out, int T, int C, int groups, int gate_first, int out_dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (C <= 0 || groups <= 0 || C % groups || (w_size != C && w_size != C / groups) || gate_stride < C) return IFX_E_BADARG;
+  if (C <= 0 || groups <= 0 || C % groups || (w != nullptr && w_size != C && w_size != C / groups) || gate_stride < C) return IFX_E_BADARG;
   if (out_dtype != IFX_DT_F32 && out_dtype != IFX_DT_BF16) return IFX_E_DTYPE;
   const int part = C / groups;
   if (groups < 8 && part > 64) {                            // few long parts: a block per row takes them in turn
