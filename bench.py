@@ -1298,6 +1298,216 @@ def run_design_radalix(args, pk):
     return 0
 
 
+# ---------------------------------------------------------------- Vononex beside Radalix and the Qwen2 shape
+def vononex_config(shape, layers=0):
+    """Vononex at the sizes of `radalix_config`: two layers of attention (the Qwen2 shape's heads of 128 over its key/value
+    heads, wholly rotated) beside a retention (heads of 64 keys x 128 values), then a gated elementwise recurrence twice as
+    wide as the model; every layer with a dense feed-forward of the Qwen2 shape's size."""
+    from inferflux_b200.config import VononexConfig
+    s = DESIGN_SHAPES[shape]
+    q = qwen7b_config(s["qwen"])
+    w, n = s["width"], layers or q.num_hidden_layers
+    mlp = {"kind": "dense", "ff": q.intermediate_size}
+    heads = w // 128
+    pair = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": s["heads"], "kv_heads": q.num_key_value_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                 "rot": {"base": 500000.0, "dims": 128}},
+        "right": {"heads": heads, "dim": 64, "vdim": 128, "rot": {"base": 10000.0, "dims": 64},
+                  "decay": [1.0 - 2.0 ** (-5.0 - 5.0 * h / heads) for h in range(heads)]},
+        "left_scale": 0.7, "right_scale": 0.7}}
+    gru = {"type": "mingru", "mixer": {"width": 2 * w}, "mlp": mlp}
+    return VononexConfig.from_dict({"architecture": "Vononex", "vocab": s["vocab"], "width": w, "norm": {"eps": 1e-6},
+                                    "postln_alpha": 2.0, "layers": [gru if i % 3 == 2 else pair for i in range(n)]})
+
+
+def vononex_costs(cfg, batch, context, tokens):
+    """(bytes a decode step must read or write, FLOPs of a prefill of `tokens`): matrices, recurrent state in and out, cached
+    keys and values."""
+    w, step_bytes, flops = cfg.width, 0, 0
+    for layer in cfg.layers:
+        m = layer["mixer"]
+        params = 3 * w * layer["mlp"]["ff"] if layer["mlp"] else 0
+        if layer["type"] == "mingru":
+            params += 4 * w * m["width"]
+            step_bytes += 2 * batch * m["width"] * 4
+        else:
+            l, r = m["left"], m["right"]
+            qd, kd, vd = l["heads"] * l["dim"], l["kv_heads"] * l["dim"], l["kv_heads"] * l["vdim"]
+            state = r["heads"] * r["dim"] * r["vdim"]
+            params += w * (qd + kd + vd + l["heads"] * l["vdim"]) + w * r["heads"] * (2 * r["dim"] + 3 * r["vdim"])
+            step_bytes += batch * context * (kd + vd) * 2 + 2 * batch * state * 4
+            flops += 2 * l["heads"] * (l["dim"] + l["vdim"]) * (tokens * (tokens + 1) // 2) + 4 * tokens * state
+        step_bytes += 2 * params
+        flops += 2 * tokens * params
+    return step_bytes + 2 * cfg.vocab * w, flops + 2 * cfg.vocab * w
+
+
+def vononex_kernels(kernels, vcfg, pk, batch, context, tokens):
+    """The new design's kernels beside the like kernels of the closest models, each alone at the layer's sizes: attention
+    whose sum is turned back beside attention with a sink and plain attention, rows normed and turned beside bias and rotation,
+    the scan with a constant decay beside the one with a decay per key channel, the elementwise scan, the norm of a sum
+    beside the norm of a sublayer's output, the gelu-gated product with biases beside the SiLU-gated one."""
+    import torch
+    from inferflux_b200.cache import CacheManager
+    from inferflux_b200.config import ScheduleEntry
+    from inferflux_b200.csrc.ops import PartialSum
+    from inferflux_b200.engine.batch import StepContext, StepEntry
+    from inferflux_b200.parts import KVCacheSpec
+    from inferflux_b200.parts.base import RotaryTable
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    mix = next(l for l in vcfg.layers if l["type"] == "parallel")["mixer"]
+    left, ret = mix["left"], mix["right"]
+    W = next(l for l in vcfg.layers if l["type"] == "mingru")["mixer"]["width"]
+    w, ff = vcfg.width, vcfg.layers[0]["mlp"]["ff"]
+    page, out = 16, {}
+
+    def row(name, fn, bytes_=0, flops=0):
+        ms = _event_times(fn)
+        roof = max(bytes_ / hbm, flops / tf)
+        out[name] = {"us": round(ms * 1000, 1), "roofline_us": round(roof * 1e6, 1), "frac": round(roof / (ms * 1e-3), 3),
+                     "bound": "hbm" if bytes_ / hbm >= flops / tf else "tensor"}
+
+    def ctx_for(cache, spans, providers=()):
+        entries, starts, slots = [], [], []
+        for rid, n in spans:
+            if rid not in cache:
+                cache.add_request(rid)
+            start = cache.length(rid)
+            cache.reserve(rid, start + n)
+            entries.append(StepEntry(rid, [0] * n, []))
+            starts.append(start)
+            slots.append(cache.slot(rid))
+        ctx = StepContext.build(kernels, bf, dev, entries, starts, slots, cache.drain_table_updates(), providers=providers)
+        for g, (idx, pg) in zip(cache.groups, ctx.table_updates):
+            kernels.scatter_i32(g.table, idx, pg)
+        for (rid, n), start in zip(spans, starts):
+            cache.commit(rid, start + n)
+        return ctx
+
+    class _Sections:                                       # asks the kernel table for the attention kernels' work lists
+        def step_sections(self, ctx):
+            return ctx.kernels.attention_sections(ctx)
+
+    nq, nkv, d = left["heads"], left["kv_heads"], left["dim"]
+    rot = RotaryTable(torch.tensor([left["rot"]["base"] ** (-2.0 * i / d) for i in range(d // 2)], device=dev), d, False)
+    rot_r = RotaryTable(torch.tensor([ret["rot"]["base"] ** (-2.0 * i / ret["dim"]) for i in range(ret["dim"] // 2)], device=dev), ret["dim"], False)
+    ones = lambda n: torch.ones(n, device=dev)
+    for what, spans_a, spans_b in (("decode", [(f"r{i}", context - 1) for i in range(batch)], [(f"r{i}", 1) for i in range(batch)]),
+                                   ("prefill", [], [("p", tokens)])):
+        T, R = sum(n for _r, n in spans_b), len(spans_b)
+        tag = f"{T} rows" if what == "decode" else f"{T} rows "
+        keys = sum((context if what == "decode" else (n * (n + 1)) // 2) for _r, n in spans_b)
+        pages = (batch * context if what == "decode" else tokens) // page + 2 * batch + 2
+        cached = batch * context if what == "decode" else tokens
+        cache = CacheManager([(KVCacheSpec(nkv, d, None), None)], page_size=page, num_pages=pages, max_seqs=batch,
+                             max_seq_len=max(context, tokens) + 16, dtype=bf, device=dev)
+        cache.groups[0].pool.normal_()
+        if spans_a:
+            ctx_for(cache, spans_a)
+        ctx = ctx_for(cache, spans_b, providers=[_Sections()])
+        view = cache.view(ScheduleEntry(0, 0))
+        splits = 8 if what == "decode" else 0
+        mk = lambda n, dt=bf: PartialSum(torch.randn(splits, T, n, device=dev), dt) if splits else torch.randn(T, n, device=dev).to(dt)
+        size = lambda n, dt=bf: T * n * (4 * splits if splits else (2 if dt == bf else 4))
+        # rows in front of attention
+        width = (nq + 2 * nkv) * d
+        qkv, bias = mk(width), torch.randn(width, device=dev)
+        run = lambda: kernels.row_norm_rope_append(qkv, 0, bias, rot, rot, ones_q[1], nq, nkv, d, d, ctx, view, q_norm=ones_q[0], k_norm=ones_k)
+        ones_q, ones_k = (ones(nq * d), ones(nq)), ones(nkv * d)
+        row(f"row norms, rotation, turned values, cache write, {tag}", run, bytes_=size(width) + 2 * T * width + T * d * 4)
+        row(f"bias, rotation, cache write (the Qwen2 model's), {tag}", lambda: kernels.rope_append(qkv, bias, rot, nq, nkv, d, ctx, view),
+            bytes_=size(width) + 2 * T * width)
+        # attention
+        q, back = run()
+        cost = dict(bytes_=cached * nkv * 2 * d * 2 + 2 * T * nq * d * 2, flops=4 * nq * d * keys)
+        row(f"attention, sum turned back, {what}", lambda: kernels.attention(q, nq, nkv, d, None, d ** -0.5, ctx, view, turn_back=back), **cost)
+        row(f"attention with a plain sink (Radalix's kernels), {what}", lambda: kernels.attention(q, nq, nkv, d, None, d ** -0.5, ctx, view, sink=True), **cost)
+        row(f"plain attention (the Qwen2 model's), {what}", lambda: kernels.attention(q, nq, nkv, d, None, d ** -0.5, ctx, view), **cost)
+        # the retention: rows turned, the scan, the gated norm
+        H, dk, dv = ret["heads"], ret["dim"], ret["vdim"]
+        rw = 2 * H * (dk + dv)
+        proj = mk(rw, f32)
+        row(f"retention's queries and keys turned, {tag}", lambda: kernels.rotate_rows(proj, 0, rw, H, dk, rot_r, dk ** -0.5, ctx),
+            bytes_=(size(rw, f32) + T * rw * 4) if splits else T * 2 * H * dk * 8)
+        state = torch.zeros(batch, H * dk * dv, device=dev)
+        wide = torch.randn(T, rw, device=dev) * 0.1
+        cut = (wide[:, :H * dk], wide[:, H * dk:2 * H * dk], wide[:, 2 * H * dk:2 * H * dk + H * dv])
+        rate, raw = torch.full((H,), 0.99, device=dev), torch.randn(T, H * dk, device=dev)
+        row(f"scan, constant decay, {tag}", lambda: kernels.decay_scan(*cut, None, state, ctx, heads=H, groups=H, dk=dk, dv=dv, decay="constant", rate=rate),
+            bytes_=2 * R * H * dk * dv * 4 + T * H * (2 * dk + 2 * dv) * 4)
+        row(f"scan, decay per key channel (Radalix's), {tag}", lambda: kernels.decay_scan(*cut, raw, state, ctx, heads=H, groups=H, dk=dk, dv=dv,
+                                                                                         decay="sigmoid_root", tau=16.0),
+            bytes_=2 * R * H * dk * dv * 4 + T * H * (3 * dk + 2 * dv) * 4)
+        o, wn = torch.randn(T, H * dv, device=dev), ones(dv)
+        row(f"gated norm per head, no weight, {tag}", lambda: kernels.gated_groupnorm(o, wide[:, 2 * H * dk + H * dv:], None, 1e-6, H, False, bf), bytes_=T * H * dv * 10)
+        row(f"gated norm per head, weight (Radalix's), {tag}", lambda: kernels.gated_groupnorm(o, wide[:, 2 * H * dk + H * dv:], wn, 1e-6, H, False, bf), bytes_=T * H * dv * 10)
+        # the elementwise recurrence
+        zxg, zb, gstate = mk(3 * W, f32), torch.zeros(2 * W, device=dev), torch.zeros(batch, W, device=dev)
+        row(f"elementwise gated scan, {tag}", lambda: kernels.gated_scan(zxg, zb, gstate, W, ctx, bf), bytes_=size(3 * W, f32) + T * W * 2 + 2 * R * W * 4)
+        del cache, zxg, proj, wide
+        # norms of sums
+        x, wr, b1 = torch.randn(T, w, device=dev), ones(w), torch.randn(w, device=dev)
+        y1, y2 = mk(w), mk(w)
+        row(f"norm of a sum, one term with a bias, {tag}", lambda: kernels.norm_of_sum(x, 2.0, [(1.0, y1, b1)], wr, 1e-6, out_dtype=bf), bytes_=size(w) + T * w * 10)
+        row(f"norm of a sum, a pair's two terms, {tag}", lambda: kernels.norm_of_sum(x, 2.0, [(0.7, y1, b1), (0.7, y2, None)], wr, 1e-6, out_dtype=bf),
+            bytes_=2 * size(w) + T * w * 10)
+        row(f"norm of a sublayer's output, added (Zeluzen's), {tag}", lambda: kernels.postnorm_add(x, y1, wr, 1e-6, out_dtype=bf, cast_out=True), bytes_=size(w) + T * w * 10)
+        # the feed-forward's first product
+        h = torch.randn(T, w, device=dev).to(bf)
+        gu, gb = (torch.randn(2 * ff, w, device=dev) * 0.02).to(bf), torch.zeros(2 * ff, device=dev)
+        cost = dict(bytes_=2 * ff * w * 2 + T * (w + ff) * 2, flops=4 * T * ff * w)
+        row(f"gelu-gated product with biases, {tag}", lambda: kernels.linear_geglu(h, gu, gb), **cost)
+        row(f"SiLU-gated product (the Qwen2 model's), {tag}", lambda: kernels.linear_swiglu(h, gu), **cost)
+        del gu
+    kernels.check_errors()
+    return out
+
+
+def run_design_vononex(args, pk):
+    """`--design vononex`: decode and prefill throughput of the design at real layer sizes beside Radalix (the closest model:
+    pairs of attention and a matrix-state scan, but mixtures of experts) and the Qwen2 shape (the same dense feed-forward) at
+    equal width, layer count and vocabulary, and its kernels beside the like kernels, one JSON line."""
+    import torch
+    page, batch, context = 16, args.batch, min(args.context, 4096)
+    steps, warmup = max(1, args.steps), max(3, args.warmup)
+    result = {"metric": "decode and prefill tokens/s of another design beside the closest models at equal size",
+              "design": args.design, "dtype": "bf16", "n_gpus": 1, "data": "synthetic: random weights, uniform random token ids",
+              "batch": batch, "context": context, "prefill_tokens": PREFILL_TOKENS, "peaks": pk["source"], "shapes": {}}
+    kernels_table = None
+    for shape in ([args.shape] if args.shape in DESIGN_SHAPES and args.shape != "7b" else sorted(DESIGN_SHAPES)):
+        entry = {}
+        for name in ("vononex", "radalix", "qwen2"):
+            if name == "qwen2":
+                cfg = qwen7b_config(DESIGN_SHAPES[shape]["qwen"])
+                cfg.num_hidden_layers = args.layers or cfg.num_hidden_layers
+            else:
+                cfg = (vononex_config if name == "vononex" else radalix_config)(shape, args.layers)
+            longest = context + 4 * (warmup + 3 * steps) + 16 + batch
+            if name == "qwen2":
+                cfg.max_position_embeddings = max(cfg.max_position_embeddings, longest)
+            engine = _engine(cfg, page, batch, longest)
+            r = time_decode(engine, cfg, batch, steps, warmup, repeats=3, context=context, e2e=False)
+            pre_ms = time_prefill(engine, cfg, PREFILL_TOKENS, warmup=2, reps=5)
+            if name == "qwen2":
+                step_bytes = weight_bytes(cfg, batch) + batch * r["ctx"] * kv_bytes_per_token(cfg)
+                flops = prefill_flops(cfg, PREFILL_TOKENS)
+            else:
+                step_bytes, flops = (vononex_costs if name == "vononex" else radalix_costs)(cfg, batch, r["ctx"], PREFILL_TOKENS)
+            entry[name] = {"decode_tok_s": round(batch * 1000.0 / r["dev_ms"], 1), "decode_ms_per_step": round(r["dev_ms"], 3),
+                           "decode_hbm_frac": round(step_bytes / (r["dev_ms"] * 1e-3) / 1e9 / pk["hbm_gbs"], 3),
+                           "launches_per_step": round(r["launches"], 1),
+                           "prefill_tok_s": round(PREFILL_TOKENS * 1000.0 / pre_ms, 1), "prefill_ms": round(pre_ms, 2),
+                           "prefill_tensor_frac": round(flops / (pre_ms * 1e-3) / 1e12 / pk["bf16_tflops"], 3)}
+            if name == "vononex" and kernels_table is None:
+                kernels_table = vononex_kernels(engine.kernels, cfg, pk, batch, context, PREFILL_TOKENS)
+                entry["kernels"] = kernels_table
+            del engine
+            torch.cuda.empty_cache()
+        result["shapes"][shape] = entry
+    print(json.dumps(result))
+    return 0
+
 
 def _engine(cfg, page, slots, longest, pages=None, chunk=2048):
     import torch
@@ -1332,7 +1542,7 @@ def main() -> int:
     ap.add_argument("--no-extras", action="store_true", help="skip the PyTorch baseline and the 1.5B-shape points")
     ap.add_argument("--prefill-only", action="store_true",
                     help="time only the 2,048-token prefill and print a short line (for profiling prefill)")
-    ap.add_argument("--design", default="", choices=["", "dafolorn", "zeluzen", "benarax", "radalix"],
+    ap.add_argument("--design", default="", choices=["", "dafolorn", "zeluzen", "benarax", "radalix", "vononex"],
                     help="instead of the headline numbers: this design at real layer sizes beside the Qwen2 shape of equal "
                          "size (decode and prefill tokens/s, and its kernels beside the like kernels); --shape picks one size")
     args = ap.parse_args()
@@ -1346,6 +1556,8 @@ def main() -> int:
         return run_design_benarax(args, pk)
     if args.design == "radalix":
         return run_design_radalix(args, pk)
+    if args.design == "vononex":
+        return run_design_vononex(args, pk)
     if args.design:
         return run_design(args, pk)
     if args.gpus != 1:

@@ -23,24 +23,40 @@ struct GatedScanArgs {
   int width;
 };
 
-__device__ __forceinline__ float sigmoid_f32(float v) { return 1.0f / (1.0f + expf(-v)); }
+// sigmoid(|v|) and sigmoid(-|v|); the divisor lies between 1 and 2, where the fast division is good to an ulp or two
+__device__ __forceinline__ void sigmoid_pair(float v, float& big, float& small) {
+  const float e = expf(-fabsf(v));
+  big = __fdividef(1.0f, 1.0f + e);
+  small = e * big;
+}
+__device__ __forceinline__ float sigmoid_f32(float v) {
+  float big, small;
+  sigmoid_pair(v, big, small);
+  return v >= 0.0f ? big : small;
+}
 
+// SLICED false: plain rows, so that a caller's loads are one straight run without a loop between them.
+template <bool SLICED>
 __device__ __forceinline__ float load_sliced(const GatedScanArgs& a, size_t at) {
-  float s = a.rows[at];
-  for (int k = 1; k < a.splits; k += 4) {                     // four slices in flight, added in split order
-    float part[4];
+  float s = __ldcg(a.rows + at);
+  if constexpr (SLICED) {
+    for (int k = 1; k < a.splits; k += 4) {                   // four slices in flight, added in split order
+      float part[4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) part[j] = k + j < a.splits ? a.rows[(size_t)(k + j) * a.split_stride + at] : 0.0f;
+      for (int j = 0; j < 4; ++j) part[j] = k + j < a.splits ? __ldcg(a.rows + (size_t)(k + j) * a.split_stride + at) : 0.0f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) s += part[j];
+      for (int j = 0; j < 4; ++j) s += part[j];
+    }
   }
   return s;
 }
 
 // what a token does to S: S <- keep S + take
 __device__ __forceinline__ void gate_of(float zr, float u, float& keep, float& take) {
-  keep = sigmoid_f32(-zr);
-  take = sigmoid_f32(zr) * (u >= 0.0f ? u + 0.5f : sigmoid_f32(u));
+  float big, small;
+  sigmoid_pair(zr, big, small);
+  keep = zr >= 0.0f ? small : big;
+  take = (zr >= 0.0f ? big : small) * (u >= 0.0f ? u + 0.5f : sigmoid_f32(u));
 }
 
 // One token a request: a thread per channel.
@@ -57,7 +73,8 @@ __global__ void __launch_bounds__(128) gated_step_kernel(const GatedScanArgs a) 
   float* st = a.state + (long long)slot * a.slot_stride + c;
   const float S0 = *st;
   const size_t at = t * 3 * a.width + c;
-  const float zr = load_sliced(a, at) + bz, u = load_sliced(a, at + a.width) + bu, g = load_sliced(a, at + 2 * (size_t)a.width);
+  const float zr = load_sliced<true>(a, at) + bz, u = load_sliced<true>(a, at + a.width) + bu;
+  const float g = load_sliced<true>(a, at + 2 * (size_t)a.width);
   float keep, take;
   gate_of(zr, u, keep, take);
   const float S = fmaf(keep, S0, take);
@@ -65,9 +82,9 @@ __global__ void __launch_bounds__(128) gated_step_kernel(const GatedScanArgs a) 
   static_cast<T*>(a.out)[t * a.width + c] = from_f32<T>(S * (g * sigmoid_f32(g)));
 }
 
-constexpr int kScanTokens = 64, kScanWorkers = 8, kScanPer = kScanTokens / kScanWorkers;     // tokens a worker warp holds
+constexpr int kScanTokens = 64, kScanWorkers = 16, kScanPer = kScanTokens / kScanWorkers;     // tokens a worker warp holds
 
-template <typename T>
+template <typename T, bool SLICED>
 __global__ void __launch_bounds__((kScanWorkers + 1) * 32) gated_scan_kernel(const GatedScanArgs a) {
   __shared__ float keep_s[2][kScanTokens][32], take_s[2][kScanTokens][32];     // take becomes S as the walk passes
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -85,15 +102,15 @@ __global__ void __launch_bounds__((kScanWorkers + 1) * 32) gated_scan_kernel(con
     for (int i = 0; i < tiles; ++i) {
       const int b = i & 1, m = min(kScanTokens, n - i * kScanTokens);
       int t = 0;
-      for (; t + 8 <= m; t += 8) {
-        float k[8], v[8];
+      for (; t + 16 <= m; t += 16) {
+        float k[16], v[16];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < 16; ++j) {
           k[j] = keep_s[b][t + j][lane];
           v[j] = take_s[b][t + j][lane];
         }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < 16; ++j) {
           S = fmaf(k[j], S, v[j]);
           take_s[b][t + j][lane] = S;
         }
@@ -107,7 +124,7 @@ __global__ void __launch_bounds__((kScanWorkers + 1) * 32) gated_scan_kernel(con
     if (live) *st = S;
     return;
   }
-  // ---- the others: a warp owns tokens warp, warp + 8, ... of every tile
+  // ---- the others: a warp owns tokens warp, warp + 16, ... of every tile
   float zr[kScanPer], ur[kScanPer], gr[kScanPer], gate[kScanPer];
   auto fetch = [&](int i) {
 #pragma unroll
@@ -116,9 +133,9 @@ __global__ void __launch_bounds__((kScanWorkers + 1) * 32) gated_scan_kernel(con
       zr[j] = ur[j] = gr[j] = 0.0f;
       if (live && t < n) {
         const size_t at = (size_t)(first + t) * 3 * a.width + c;
-        zr[j] = load_sliced(a, at);
-        ur[j] = load_sliced(a, at + a.width);
-        gr[j] = load_sliced(a, at + 2 * (size_t)a.width);
+        zr[j] = load_sliced<SLICED>(a, at);
+        ur[j] = load_sliced<SLICED>(a, at + a.width);
+        gr[j] = load_sliced<SLICED>(a, at + 2 * (size_t)a.width);
       }
     }
   };
@@ -178,5 +195,8 @@ extern "C" int ifx_gated_scan(const float* rows, int splits, const float* bias, 
     return launch_pdl(f32 ? gated_step_kernel<float> : gated_step_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, 1, a);
   }
   const dim3 grid((width + 31) / 32, num_requests);
-  return launch_pdl(f32 ? gated_scan_kernel<float> : gated_scan_kernel<__nv_bfloat16>, grid, dim3((kScanWorkers + 1) * 32), 0, stream, 1, a);
+  const dim3 block((kScanWorkers + 1) * 32);
+  if (splits > 1)
+    return launch_pdl(f32 ? gated_scan_kernel<float, true> : gated_scan_kernel<__nv_bfloat16, true>, grid, block, 0, stream, 1, a);
+  return launch_pdl(f32 ? gated_scan_kernel<float, false> : gated_scan_kernel<__nv_bfloat16, false>, grid, block, 0, stream, 1, a);
 }

@@ -7,7 +7,7 @@
 //                          and the cosines and sines of the values' angles, for whoever turns a sum of values back.
 //                          One block, or a cluster of blocks that share the heads, per token.
 //   rotate_rows            rows [heads of d | heads of d | rest] -> float32: both groups of heads turned, the second one
-//                          scaled behind it, the rest as it is.  A warp per (token, head).
+//                          scaled behind it, the rest as it is.
 //
 // Both read plain rows (wider ones than needed, from a column on) or the float32 partial sums of a K-split product.
 // Angles are position * frequency in float32 with precise sines; norms, rotations and factors are float32.
@@ -48,12 +48,19 @@ struct RowSource {
     }
     return s;
   }
+  // float32 only; SLICED false (plain rows): a caller's loads are one straight run without a branch between them
+  template <bool SLICED>
   __device__ __forceinline__ float load1(size_t token, int c) const {
     const size_t at = token * ld + col0 + c;
-    if (partial == nullptr)
-      return is_bf16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(rows)[at]) : static_cast<const float*>(rows)[at];
+    if (!SLICED) return static_cast<const float*>(rows)[at];
     float s = 0.0f;
-    for (int k = 0; k < splits; ++k) s += partial[(size_t)k * split_stride + at];
+    for (int k = 0; k < splits; k += 4) {                    // four slices in flight, added in split order
+      float part[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) part[j] = k + j < splits ? partial[(size_t)(k + j) * split_stride + at] : 0.0f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s += part[j];
+    }
     return s;
   }
 };
@@ -209,39 +216,155 @@ __global__ void __launch_bounds__(1024) row_norm_rope_append_kernel(const RowRop
   }
 }
 
+// The same work for many tokens in the common case: plain bfloat16 rows, whole heads turned in halves, sizes that are
+// multiples of 4 up to 128.  A lane holds elements (2l, 2l + 1) and their partners half a head away, all of a warp's UPW
+// heads in registers, fetched before anything is waited for.
+template <int UPW>
+__global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeArgs a) {
+  __shared__ __align__(16) float2 cs[128];                                 // [d / 2] then [dv / 2]
+  __shared__ float part_q[16], part_k[16];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+  const int units = a.nq + 2 * a.nkv;
+  const int half_rot = a.rot / 2, half_v = a.v_inv_freq ? a.dv / 2 : 0;
+  const __nv_bfloat16* row = static_cast<const __nv_bfloat16*>(a.src.rows) + (size_t)t * a.src.ld + a.src.col0;
+  const int pos = a.positions[t];
+  int page = -1;
+  if (a.write_cache) page = a.block_table[(size_t)a.req_slot[a.token_req[t]] * a.max_blocks + pos / a.page_size];
+  pdl_wait();
+  __nv_bfloat162 lo_raw[UPW], hi_raw[UPW];
+  float2 lo[UPW], hi[UPW];
+#pragma unroll
+  for (int k = 0; k < UPW; ++k) {
+    const int u = warp + k * nwarps;
+    const bool is_v = u >= a.nq + a.nkv;
+    const int half = (is_v ? a.dv : a.d) / 2;
+    const int col = is_v ? (a.nq + a.nkv) * a.d + (u - a.nq - a.nkv) * a.dv : u * a.d;
+    lo_raw[k] = hi_raw[k] = __floats2bfloat162_rn(0.0f, 0.0f);
+    lo[k] = hi[k] = make_float2(0.0f, 0.0f);
+    if (u < units && 2 * lane < half) {
+      lo_raw[k] = *reinterpret_cast<const __nv_bfloat162*>(row + col + 2 * lane);
+      hi_raw[k] = *reinterpret_cast<const __nv_bfloat162*>(row + col + half + 2 * lane);
+      if (a.bias) {
+        lo[k] = *reinterpret_cast<const float2*>(a.bias + col + 2 * lane);
+        hi[k] = *reinterpret_cast<const float2*>(a.bias + col + half + 2 * lane);
+      }
+    }
+  }
+  for (int j = threadIdx.x; j < half_rot + half_v; j += blockDim.x) {
+    float sn, c;
+    sincosf((float)pos * (j < half_rot ? a.inv_freq[j] : a.v_inv_freq[j - half_rot]), &sn, &c);
+    cs[j] = make_float2(c, sn);
+    if (j >= half_rot && a.turn_out) a.turn_out[(size_t)t * half_v + (j - half_rot)] = make_float2(c, sn);
+  }
+  float ss_q = 0.0f, ss_k = 0.0f;
+#pragma unroll
+  for (int k = 0; k < UPW; ++k) {
+    const int u = warp + k * nwarps;
+    const float2 l = __bfloat1622float2(lo_raw[k]), h = __bfloat1622float2(hi_raw[k]);
+    lo[k].x += l.x; lo[k].y += l.y; hi[k].x += h.x; hi[k].y += h.y;
+    const float ss = fmaf(lo[k].x, lo[k].x, fmaf(lo[k].y, lo[k].y, fmaf(hi[k].x, hi[k].x, hi[k].y * hi[k].y)));
+    if (u < a.nq) ss_q += ss;
+    else if (u < a.nq + a.nkv) ss_k += ss;
+  }
+  ss_q = warp_sum(ss_q);
+  ss_k = warp_sum(ss_k);
+  if (lane == 0) {
+    part_q[warp] = ss_q;
+    part_k[warp] = ss_k;
+  }
+  __syncthreads();
+  ss_q = warp_sum(lane < nwarps ? part_q[lane] : 0.0f);
+  ss_k = warp_sum(lane < nwarps ? part_k[lane] : 0.0f);
+  const float inv_q = 1.0f / sqrtf(ss_q / (float)(a.nq * a.d) + a.eps), inv_k = 1.0f / sqrtf(ss_k / (float)(a.nkv * a.d) + a.eps);
+#pragma unroll
+  for (int k = 0; k < UPW; ++k) {
+    const int u = warp + k * nwarps;
+    const bool is_q = u < a.nq, is_v = u >= a.nq + a.nkv;
+    const int half = (is_v ? a.dv : a.d) / 2;
+    if (u >= units || 2 * lane >= half) continue;
+    __nv_bfloat16* dst;
+    if (is_q) {
+      dst = static_cast<__nv_bfloat16*>(a.q_out) + ((size_t)t * a.nq + u) * a.d;
+    } else {
+      if (page < 0 || page >= a.num_pages) continue;         // never write outside the pool
+      const int g = u - a.nq - (is_v ? a.nkv : 0);
+      dst = static_cast<__nv_bfloat16*>(a.kv_pool) +
+            ((((size_t)page * 2 + (is_v ? 1 : 0)) * a.nkv + g) * a.page_size + (pos % a.page_size)) * a.d_row;
+    }
+    float2 x = lo[k], y = hi[k];
+    const float* nw = is_q ? a.q_norm : (is_v ? nullptr : a.k_norm);
+    if (nw) {
+      const float inv = is_q ? inv_q : inv_k;
+      nw += (size_t)(is_q ? u : u - a.nq) * a.d + 2 * lane;
+      const float2 wl = *reinterpret_cast<const float2*>(nw), wh = *reinterpret_cast<const float2*>(nw + half);
+      x.x *= inv * wl.x; x.y *= inv * wl.y; y.x *= inv * wh.x; y.y *= inv * wh.y;
+    }
+    if (!is_v || half_v) {
+      const float4 c = *reinterpret_cast<const float4*>(&cs[(is_v ? half_rot : 0) + 2 * lane]);      // cos, sin of two pairs
+      const float2 rx = make_float2(x.x * c.x - y.x * c.y, x.y * c.z - y.y * c.w);
+      y = make_float2(y.x * c.x + x.x * c.y, y.y * c.z + x.y * c.w);
+      x = rx;
+    }
+    if (is_q) {
+      const float f = a.temp ? a.temp[u] : 1.0f;
+      x.x *= f; x.y *= f; y.x *= f; y.y *= f;
+    } else {                                                 // the cache only ever holds finite values
+      x.x = isfinite(x.x) ? x.x : 0.0f;
+      x.y = isfinite(x.y) ? x.y : 0.0f;
+      y.x = isfinite(y.x) ? y.x : 0.0f;
+      y.y = isfinite(y.y) ? y.y : 0.0f;
+    }
+    *reinterpret_cast<__nv_bfloat162*>(dst + 2 * lane) = __floats2bfloat162_rn(x.x, x.y);
+    *reinterpret_cast<__nv_bfloat162*>(dst + half + 2 * lane) = __floats2bfloat162_rn(y.x, y.y);
+  }
+}
+
+// A warp goes over the heads u, u + step, ... of one token: its lanes' angles are the same for all of them.  Four heads'
+// elements are fetched before the first is stored (the rows may be turned where they lie).
+template <bool SLICED>
 __global__ void __launch_bounds__(128) rotate_rows_kernel(const RowSource src, const float* __restrict__ inv_freq, int rot,
                                                           int interleaved, const int* __restrict__ positions,
                                                           float* __restrict__ out, int width, int heads, int d, float k_scale,
                                                           int in_place) {
   pdl_launch_dependents();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int u = blockIdx.y * 4 + warp;                       // [0, heads) first group, [heads, 2 heads) second, then the rest
+  const int u0 = blockIdx.y * 4 + warp, step = gridDim.y * 4;
   const float pos = (float)positions[t];
   float* o = out + (size_t)t * width;
-  float2 first = make_float2(1.0f, 0.0f);                    // the lane's first pair's angle, before the rows are known to be there
-  if (u < 2 * heads && lane < rot / 2) sincosf(pos * inv_freq[lane], &first.y, &first.x);
-  pdl_wait();
-  if (u < 2 * heads) {
-    const float scale = u >= heads ? k_scale : 1.0f;
-    for (int j = lane; j < (d + 1) / 2; j += 32) {
-      int e0, e1;
-      pair_of(j, rot, interleaved, e0, e1);
-      const bool both = e1 < d;
-      float x = src.load1(t, u * d + e0), y = both ? src.load1(t, u * d + e1) : 0.0f;
-      if (j < rot / 2) {
-        float2 c = first;
-        if (j != lane) sincosf(pos * inv_freq[j], &c.y, &c.x);
-        const float rx = x * c.x - y * c.y, ry = y * c.x + x * c.y;
-        x = rx;
-        y = ry;
+  bool arrived = false;
+  for (int j = lane; j - lane < (d + 1) / 2; j += 32) {       // whole warps: a lane beyond the head does nothing
+    const bool live = j < (d + 1) / 2;
+    int e0, e1;
+    pair_of(live ? j : 0, rot, interleaved, e0, e1);
+    const bool both = e1 < d, turns = live && j < rot / 2;
+    float2 c = make_float2(1.0f, 0.0f);
+    if (turns) sincosf(pos * inv_freq[j], &c.y, &c.x);
+    if (!arrived) pdl_wait();                                // angles do not come from the kernel in front
+    arrived = true;
+    for (int u = u0; u < 2 * heads; u += 4 * step) {
+      float x[4], y[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int h = u + k * step;
+        const bool in = live && h < 2 * heads;
+        x[k] = in ? src.load1<SLICED>(t, h * d + e0) : 0.0f;
+        y[k] = in && both ? src.load1<SLICED>(t, h * d + e1) : 0.0f;
       }
-      o[u * d + e0] = x * scale;
-      if (both) o[u * d + e1] = y * scale;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int h = u + k * step;
+        if (!live || h >= 2 * heads) continue;
+        const float scale = h >= heads ? k_scale : 1.0f;
+        const float rx = turns ? x[k] * c.x - y[k] * c.y : x[k], ry = turns ? y[k] * c.x + x[k] * c.y : y[k];
+        o[h * d + e0] = rx * scale;
+        if (both) o[h * d + e1] = ry * scale;
+      }
     }
-  } else if (!in_place) {
-    const int c0 = 2 * heads * d + (u - 2 * heads) * 128;
-    for (int c = c0 + lane; c < min(c0 + 128, width); c += 32) o[c] = src.load1(t, c);
   }
+  if (!arrived) pdl_wait();
+  if (in_place) return;
+  for (int c0 = 2 * heads * d + u0 * 128; c0 < width; c0 += step * 128)
+    for (int c = c0 + lane; c < min(c0 + 128, width); c += 32) o[c] = src.load1<SLICED>(t, c);
 }
 
 static int make_source(RowSource* s, const void* rows, int dtype, const float* partial, int splits, int tokens, long long ld, int col0) {
@@ -286,6 +409,19 @@ int ifx_row_norm_rope_append(const void* rows, int src_dtype, const float* parti
   a.kv_pool = kv_pool; a.q_out = q_out; a.turn_out = reinterpret_cast<float2*>(turn_out); a.nq = nq; a.nkv = nkv; a.d = d; a.dv = dv;
   a.d_row = d_row; a.write_cache = write_cache;
   const int units = nq + 2 * nkv, dmax = d > dv ? d : dv;
+  auto aligned = [](const void* p, int n) { return reinterpret_cast<uintptr_t>(p) % n == 0; };
+  if (dtype == IFX_DT_BF16 && rows != nullptr && src_dtype == IFX_DT_BF16 && num_tokens > 32 && rot == d && !interleaved &&
+      (v_inv_freq == nullptr || !v_interleaved) && d % 4 == 0 && dv % 4 == 0 && dmax <= 128 && units <= 64 && d_row % 2 == 0 &&
+      aligned(bias, 8) && aligned(q_norm, 8) && aligned(k_norm, 8) && aligned(q_out, 4) && aligned(kv_pool, 4)) {
+    const int per_warp = (units + 15) / 16, warps = (units + per_warp - 1) / per_warp;
+    const dim3 grid(num_tokens), block(32 * warps);
+    switch (per_warp) {
+      case 1: return launch_pdl(row_norm_rope_rows_kernel<1>, grid, block, 0, stream, 1, a);
+      case 2: return launch_pdl(row_norm_rope_rows_kernel<2>, grid, block, 0, stream, 1, a);
+      case 3: return launch_pdl(row_norm_rope_rows_kernel<3>, grid, block, 0, stream, 1, a);
+      default: return launch_pdl(row_norm_rope_rows_kernel<4>, grid, block, 0, stream, 1, a);
+    }
+  }
   // Few bfloat16 tokens: a cluster of blocks shares a token's heads, so that more than one SM fetches its slices.  Float32
   // runs keep one block a token, so that the order of a row's additions never depends on the step.
   int C = 1;
@@ -318,9 +454,11 @@ int ifx_rotate_rows(const float* rows, const float* partial, int splits, long lo
   RowSource src;
   const int rc = make_source(&src, rows, IFX_DT_F32, partial, splits, num_tokens, ld, col0);
   if (rc) return rc;
-  const int units = 2 * heads + (in_place ? 0 : (width - 2 * heads * d + 127) / 128);
-  if ((units + 3) / 4 > 65535) return IFX_E_TOOBIG;
-  return launch_pdl(rotate_rows_kernel, dim3(num_tokens, (units + 3) / 4), dim3(128), 0, stream, 1, src, inv_freq, rot, interleaved,
+  // few tokens: a head (or 128 columns of the rest) a warp; many: one block a token
+  const int rest = in_place ? 0 : (width - 2 * heads * d + 127) / 128, most = 2 * heads > rest ? 2 * heads : rest;
+  int blocks = num_tokens >= 128 ? 1 : (most + 3) / 4;
+  if (blocks > 1024) blocks = 1024;
+  return launch_pdl(partial ? rotate_rows_kernel<true> : rotate_rows_kernel<false>, dim3(num_tokens, blocks), dim3(128), 0, stream, 1, src, inv_freq, rot, interleaved,
                     positions, out, width, heads, d, k_scale, in_place);
 }
 
