@@ -9,12 +9,13 @@ sequence slots are leased with a generation stamp so that a stale free is refuse
 storage itself.
 
 Caches (one per schedule entry that writes) with the same needs - same heads, head
-size and window - form a group.  A group has its own pool
+size, window and kept first tokens - form a group.  A group has its own pool
 [caches_in_group, pages, planes (K, V; or one latent), kv_heads, page_size, head_dim], its own page
 allocator and its own block table [max_seqs, max_blocks] on the device, indexed by
 the request's slot: one page id serves every cache of the group.  A request's
 pages are given back when it ends, and, in a group with a window, as soon as
-the window has moved past them.  Entries of the device block table change only
+the window has moved past them (all but the pages of the first tokens that stay
+visible).  Entries of the device block table change only
 through the updates a step drains with `drain_table_updates`.
 """
 from __future__ import annotations
@@ -240,7 +241,7 @@ class CacheManager:
 
     def commit(self, rid, new_len: int) -> None:
         """The step has stored positions up to new_len - 1; pages that a window has
-        moved past are given back."""
+        moved past are given back, all but those of the first tokens that stay visible."""
         req = self._requests[rid]
         req.length = new_len
         for gi, (g, held) in enumerate(zip(self.groups, req.blocks)):
@@ -248,7 +249,8 @@ class CacheManager:
                 continue
             first = min(self._first_needed_block(g, new_len), req.hi[gi])
             if req.lo[gi] < first:
-                dead = [b for b in range(req.lo[gi], first) if b in held]
+                stay = -(-g.spec.keep_first // self.page_size)         # blocks of first tokens that stay visible
+                dead = [b for b in range(max(req.lo[gi], stay), first) if b in held]
                 if dead:
                     g.alloc.release([held[b] for b in dead], owner=rid)
                     for b in dead:

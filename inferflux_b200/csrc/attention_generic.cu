@@ -20,7 +20,9 @@
 //   d_v, d_row   values of another size than the keys; both lie in cache rows of d_row elements
 //                (a multiple of 8 that holds either; what lies behind a row's d or d_v elements is zero)
 //   chunk        > 0: a query at position p sees the keys from (p / chunk) * chunk on, not from 0
-//   turn_back    float2 [tokens, d_v / 2]: a head's output is turned back by the token's angles (see TurnBack)
+//   keep_first   the first keys of a sequence that every query sees besides (they are visited first)
+//   head_gate    float [tokens, nq]: a head's output is multiplied by it
+//   turn_back    float2 [tokens, d_v / 2]: a head's output is turned back by the token's angles (see HeadOutput)
 //   sink         1: the softmax's denominator holds one more unit, a key of score 0 without a value
 #include "common.cuh"
 
@@ -68,8 +70,8 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
                                          const int* __restrict__ token_req, const int* __restrict__ req_slot,
                                          const int* __restrict__ rows, T* __restrict__ out, int num_tokens, int nq,
                                          int nkv, int d, int d_v, int d_row,
-                                         int page_size, int max_blocks, int num_pages, int window, int chunk,
-                                         int sink, const float* __restrict__ sink_values, float scale, TurnBack turn) {
+                                         int page_size, int max_blocks, int num_pages, KeyMask mask,
+                                         float scale, HeadOutput post) {
   __shared__ __align__(16) float q_s[kWarpsPerBlock][kMaxHeadDim];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * kWarpsPerBlock + warp;
@@ -87,19 +89,18 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
   for (int e = lane; e < d_row; e += 32) q_s[warp][e] = e < d ? to_f32(qrow[e]) : 0.0f;
   __syncwarp();
 
-  int first = window > 0 ? max(0, pos - window + 1) : 0;
-  if (chunk > 0) first = max(first, (pos / chunk) * chunk);
-  const int end = pos + 1;
+  const int first = mask.first(pos), kept = mask.kept(first), end = pos + 1;
   // the sink is a key of score 0 that comes first and brings no value: maximum 0, sum 1
   // (with sink_values the score is the head's learned number instead of 0)
-  float m = sink ? (sink_values ? sink_values[h] : 0.0f) : -INFINITY, l = sink ? 1.0f : 0.0f;
+  float m = mask.sink ? (mask.sink_values ? mask.sink_values[h] : 0.0f) : -INFINITY, l = mask.sink ? 1.0f : 0.0f;
   float acc[kMaxHeadDim / 32];
 #pragma unroll
   for (int i = 0; i < kMaxHeadDim / 32; ++i) acc[i] = 0.0f;
 
-  for (int base = first; base < end; base += 32) {
+  for (int part = kept > 0 ? 0 : 1; part < 2; ++part)      // keys [0, kept), then [first, end)
+  for (int base = part ? first : 0, stop = part ? end : kept; base < stop; base += 32) {
     const int j = base + lane;
-    const bool valid = j < end;
+    const bool valid = j < stop;
     float s = -INFINITY;
     size_t row_off = 0;                                  // element offset of key row j inside its page's K part
     int page = 0;
@@ -116,7 +117,7 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
     m = m_new;
 #pragma unroll
     for (int i = 0; i < kMaxHeadDim / 32; ++i) acc[i] *= corr;
-    const int count = min(32, end - base);
+    const int count = min(32, stop - base);
     for (int jj = 0; jj < count; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const int pg = __shfl_sync(0xffffffffu, page, jj);
@@ -129,9 +130,9 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
       }
     }
   }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * post.factor(t, h);
   T* orow = out + ((size_t)t * nq + h) * d_v;
-  if (turn.table != nullptr) {                             // the head's row through shared memory: pairs meet there
+  if (post.table != nullptr) {                             // the head's row through shared memory: pairs meet there
     __syncwarp();
 #pragma unroll
     for (int i = 0; i < kMaxHeadDim / 32; ++i) {
@@ -140,9 +141,9 @@ __global__ void attention_generic_kernel(const T* __restrict__ q, const T* __res
     }
     __syncwarp();
     for (int m = lane; m < d_v / 2; m += 32) {
-      const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + d_v / 2;
+      const int e0 = post.interleaved ? 2 * m : m, e1 = post.interleaved ? 2 * m + 1 : m + d_v / 2;
       float u = q_s[warp][e0], v = q_s[warp][e1];
-      TurnBack::apply(turn.table[(size_t)t * (d_v / 2) + m], u, v);
+      HeadOutput::apply(post.table[(size_t)t * (d_v / 2) + m], u, v);
       orow[e0] = from_f32<T>(u);
       orow[e1] = from_f32<T>(v);
     }
@@ -164,24 +165,26 @@ extern "C" int ifx_attention_generic_sink(const void* q, const void* kv_pool, co
                                           const int* rows, void* out, int num_tokens, int nq, int nkv, int d, int d_v,
                                           int d_row, int page_size, int max_blocks, int num_pages, int window, int chunk,
                                           int sink, const float* sink_values, float scale, const float* turn_back,
-                                          int turn_interleaved, int dtype, cudaStream_t stream) {
+                                          int turn_interleaved, int keep_first, const float* head_gate, int dtype,
+                                          cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  const KeyMask mask{window, chunk, sink, sink_values, keep_first};
   if (turn_back != nullptr && d_v % 2) return IFX_E_BADARG;
-  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
+  const HeadOutput post{reinterpret_cast<const float2*>(turn_back), turn_interleaved, head_gate, nq};
   if (nq <= 0 || nkv <= 0 || nq % nkv || d <= 0 || d_v <= 0 || d_row % 8 || d_row > kMaxHeadDim || d > d_row ||
-      d_v > d_row || page_size <= 0 || max_blocks <= 0 || chunk < 0)
+      d_v > d_row || page_size <= 0 || max_blocks <= 0 || chunk < 0 || keep_first < 0)
     return IFX_E_BADARG;
   const long long items = (long long)num_tokens * nq;
   const unsigned blocks = (unsigned)((items + kWarpsPerBlock - 1) / kWarpsPerBlock);
   if (dtype == IFX_DT_F32)
     attention_generic_kernel<float><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
         (const float*)q, (const float*)kv_pool, block_table, positions, token_req, req_slot, rows, (float*)out,
-        num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, window, chunk, sink, sink_values, scale, turn);
+        num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, mask, scale, post);
   else if (dtype == IFX_DT_BF16)
     attention_generic_kernel<__nv_bfloat16><<<blocks, kWarpsPerBlock * 32, 0, stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv_pool, block_table, positions, token_req, req_slot,
-        rows, (__nv_bfloat16*)out, num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, window,
-        chunk, sink, sink_values, scale, turn);
+        rows, (__nv_bfloat16*)out, num_tokens, nq, nkv, d, d_v, d_row, page_size, max_blocks, num_pages, mask,
+        scale, post);
   else
     return IFX_E_DTYPE;
   IFX_CHECK_LAUNCH();
@@ -195,7 +198,7 @@ extern "C" int ifx_attention_generic_ex(const void* q, const void* kv_pool, cons
                                         int sink, float scale, int dtype, cudaStream_t stream) {
   return ifx_attention_generic_sink(q, kv_pool, block_table, positions, token_req, req_slot, rows, out, num_tokens, nq, nkv,
                                     d, d_v, d_row, page_size, max_blocks, num_pages, window, chunk, sink, nullptr, scale, nullptr,
-                                    0, dtype, stream);
+                                    0, 0, nullptr, dtype, stream);
 }
 
 extern "C" int ifx_attention_generic(const void* q, const void* kv_pool, const int* block_table,

@@ -80,6 +80,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 struct PageMap {
   const int* table;      // this request's row of the block table, or a shared-memory copy of a part of it
   int blk_base;          // the logical block that table[0] stands for
+  const int* table_all;  // the whole row: blocks below blk_base (keys that stay visible in front of a window) are read from it
   int page_size, page_shift, num_pages, nkv, g;
   // Element offset of key `k`'s row (head g) in the pool; the value row lies v_off further.
   __device__ __forceinline__ size_t key_row(int k, int d) const {
@@ -91,7 +92,7 @@ struct PageMap {
       blk = k / page_size;
       off = k - blk * page_size;
     }
-    int page = table[blk - blk_base];
+    int page = blk >= blk_base ? table[blk - blk_base] : table_all[blk];
     if (page < 0 || page >= num_pages) page = 0;          // a broken table must not leave the pool
     return ((((size_t)page * 2) * nkv + g) * page_size + off) * d;
   }
@@ -100,12 +101,12 @@ struct PageMap {
 // ------------------------------------------------------------- prompt portions
 // The finished rows of a key head's G query heads ([G][D] in shared memory), turned back and stored.
 template <int D>
-__device__ __forceinline__ void store_turned(const float* rows_s, bf16* out, const TurnBack& turn, int t, int G, int tid, int threads) {
+__device__ __forceinline__ void store_turned(const float* rows_s, bf16* out, const HeadOutput& post, int t, int G, int tid, int threads) {
   for (int idx = tid; idx < G * (D / 2); idx += threads) {
     const int row = idx / (D / 2), m = idx % (D / 2);
-    const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + D / 2;
+    const int e0 = post.interleaved ? 2 * m : m, e1 = post.interleaved ? 2 * m + 1 : m + D / 2;
     float u = rows_s[row * D + e0], v = rows_s[row * D + e1];
-    TurnBack::apply(turn.table[(size_t)t * (D / 2) + m], u, v);
+    HeadOutput::apply(post.table[(size_t)t * (D / 2) + m], u, v);
     out[row * D + e0] = __float2bfloat16_rn(u);
     out[row * D + e1] = __float2bfloat16_rn(v);
   }
@@ -115,7 +116,7 @@ template <int D, int KT>
 __global__ void __launch_bounds__(128)
 attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool, const int* __restrict__ block_table,
                     const int* __restrict__ tiles, const int* __restrict__ req_slot, bf16* __restrict__ out, int nq,
-                    int nkv, int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn,
+                    int nkv, int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, HeadOutput post,
                     float scale_log2, int tbl_cap) {
   constexpr int LDS = D + 8;            // shared-memory row stride in elements
   constexpr int CPR = D / 8;            // 16-byte chunks per row
@@ -132,12 +133,15 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
   const int r = tile[0], row0 = tile[1] + half, rows = min(64, tile[2] - half), pos0 = tile[3] + half;
   const int h = blockIdx.y;
   const int* table_g = block_table + (size_t)req_slot[r] * max_blocks;
-  PageMap pm{table_g, 0, page_size, page_shift, num_pages, nkv, h / (nq / nkv)};
+  PageMap pm{table_g, 0, table_g, page_size, page_shift, num_pages, nkv, h / (nq / nkv)};
   const size_t v_off = (size_t)nkv * page_size * D;
 
   const int kfirst = window.first(pos0);
   const int kend = pos0 + rows;
+  // key tiles in the order they are visited: [0, kept_tiles) with the keys that stay visible, then [tile_begin, tile_end)
   const int tile_begin = kfirst / KT, tile_end = (kend + KT - 1) / KT;
+  const int kept_tiles = min((window.keep + KT - 1) / KT, tile_begin);
+  const int num_tiles = kept_tiles + tile_end - tile_begin;
   {   // the block-table entries of keys [kfirst, kend) go to shared memory once
     const int b0 = kfirst / page_size, b1 = (kend - 1) / page_size;
     if (b1 - b0 + 1 <= tbl_cap) {
@@ -162,7 +166,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
       const int k = t * KT + row;
       bf16* kd = k_s + (stage * KT + row) * LDS + c * 8;
       bf16* vd = v_s + (stage * KT + row) * LDS + c * 8;
-      if (k >= kfirst && k < kend) {
+      if (window.sees(k, kfirst) && k < kend) {
         const bf16* src = kv_pool + pm.key_row(k, D) + c * 8;
         cp_async16(smem_u32(kd), src);
         cp_async16(smem_u32(vd), src + v_off);
@@ -172,7 +176,8 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
       }
     }
   };
-  load_tile(tile_begin, 0);
+  auto tile_at = [&](int i) { return i < kept_tiles ? i : i - kept_tiles + tile_begin; };
+  load_tile(tile_at(0), 0);
   cp_async_commit();
 
   uint32_t qf[D / 16][4];
@@ -183,13 +188,13 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
   const int p_lo = pos0 + warp * 16 + (lane >> 2), p_hi = p_lo + 8;
   const int w_lo = window.first(p_lo), w_hi = window.first(p_hi);
 
-  for (int t = tile_begin; t < tile_end; ++t) {
-    const int stage = (t - tile_begin) & 1;
-    if (t + 1 < tile_end) load_tile(t + 1, stage ^ 1);
+  for (int i = 0; i < num_tiles; ++i) {
+    const int stage = i & 1, t = tile_at(i);
+    if (i + 1 < num_tiles) load_tile(tile_at(i + 1), stage ^ 1);
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    if (t == tile_begin) {
+    if (i == 0) {
 #pragma unroll
       for (int kk = 0; kk < D / 16; ++kk) {
         const int row = warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, col = kk * 16 + (lane >> 4) * 8;
@@ -215,15 +220,16 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
     // Masking only where a key of the tile can be invisible to a row of this warp: a tile that lies
     // wholly inside every row's range (most tiles of a long prompt) skips the compares.
     const int key0 = t * KT;
-    const bool inside = key0 + KT - 1 <= pos0 + warp * 16 && key0 >= kfirst &&
-                        (!window.any() || key0 >= window.first(pos0 + warp * 16 + 15));
+    const bool inside = key0 + KT - 1 <= pos0 + warp * 16 &&
+                        ((key0 >= kfirst && (!window.any() || key0 >= window.first(pos0 + warp * 16 + 15))) ||
+                         key0 + KT <= window.keep);
     if (!inside) {
 #pragma unroll
       for (int n = 0; n < KT / 8; ++n) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + n * 8 + 2 * (lane & 3) + (e & 1);
-          const bool ok = e < 2 ? (key <= p_lo && key >= w_lo) : (key <= p_hi && key >= w_hi);
+          const bool ok = e < 2 ? (key <= p_lo && window.sees(key, w_lo)) : (key <= p_hi && window.sees(key, w_hi));
           if (!ok) s[n][e] = -INFINITY;
         }
       }
@@ -285,26 +291,27 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool
     l_lo += exp2f(window.sink_log2(h) - m_lo * scale_log2);
     l_hi += exp2f(window.sink_log2(h) - m_hi * scale_log2);
   }
-  const float i_lo = l_lo > 0.0f ? 1.0f / l_lo : 0.0f, i_hi = l_hi > 0.0f ? 1.0f / l_hi : 0.0f;
   const int r_lo = warp * 16 + (lane >> 2), r_hi = r_lo + 8;
-  if (turn.table != nullptr) {                          // both elements of a pair lie in this thread
-    const float2* cs_lo = turn.table + (size_t)(row0 + min(r_lo, rows - 1)) * (D / 2);
-    const float2* cs_hi = turn.table + (size_t)(row0 + min(r_hi, rows - 1)) * (D / 2);
-    if (turn.interleaved) {
+  const float i_lo = (l_lo > 0.0f ? 1.0f / l_lo : 0.0f) * post.factor(row0 + min(r_lo, rows - 1), h);
+  const float i_hi = (l_hi > 0.0f ? 1.0f / l_hi : 0.0f) * post.factor(row0 + min(r_hi, rows - 1), h);
+  if (post.table != nullptr) {                          // both elements of a pair lie in this thread
+    const float2* cs_lo = post.table + (size_t)(row0 + min(r_lo, rows - 1)) * (D / 2);
+    const float2* cs_hi = post.table + (size_t)(row0 + min(r_hi, rows - 1)) * (D / 2);
+    if (post.interleaved) {
 #pragma unroll
       for (int n = 0; n < D / 8; ++n) {
         const int m = n * 4 + (lane & 3);
-        TurnBack::apply(cs_lo[m], o[n][0], o[n][1]);
-        TurnBack::apply(cs_hi[m], o[n][2], o[n][3]);
+        HeadOutput::apply(cs_lo[m], o[n][0], o[n][1]);
+        HeadOutput::apply(cs_hi[m], o[n][2], o[n][3]);
       }
     } else {
 #pragma unroll
       for (int n = 0; n < D / 16; ++n) {
         const int m = n * 8 + 2 * (lane & 3);
-        TurnBack::apply(cs_lo[m], o[n][0], o[n + D / 16][0]);
-        TurnBack::apply(cs_lo[m + 1], o[n][1], o[n + D / 16][1]);
-        TurnBack::apply(cs_hi[m], o[n][2], o[n + D / 16][2]);
-        TurnBack::apply(cs_hi[m + 1], o[n][3], o[n + D / 16][3]);
+        HeadOutput::apply(cs_lo[m], o[n][0], o[n + D / 16][0]);
+        HeadOutput::apply(cs_lo[m + 1], o[n][1], o[n + D / 16][1]);
+        HeadOutput::apply(cs_hi[m], o[n][2], o[n + D / 16][2]);
+        HeadOutput::apply(cs_hi[m + 1], o[n][3], o[n + D / 16][3]);
       }
     }
   }
@@ -325,7 +332,7 @@ template <int D, int STAGES>
 __global__ void __launch_bounds__(128)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool, const int* __restrict__ block_table,
                    const int4* __restrict__ decode_meta, bf16* __restrict__ out, int nq, int nkv, int page_size,
-                   int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn, float scale_log2, int tbl_cap) {
+                   int page_shift, int max_blocks, int num_pages, KeyMask window, HeadOutput post, float scale_log2, int tbl_cap) {
   constexpr int LDS = D + 8;
   constexpr int CPR = D / 8;
   constexpr int STAGE_ELEMS = 2 * 16 * LDS;             // K tile then V tile
@@ -349,16 +356,17 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
   const int t = meta.x;
   const int pos = meta.y;
   const int* table_g = block_table + (size_t)meta.z * max_blocks;
-  PageMap pm{table_g, 0, page_size, page_shift, num_pages, nkv, g};
+  PageMap pm{table_g, 0, table_g, page_size, page_shift, num_pages, nkv, g};
   const size_t v_off = (size_t)nkv * page_size * D;
 
-  const int kfirst = window.first(pos);
-  const int kend = pos + 1;
-  const int per_split = (((kend - kfirst + num_splits - 1) / num_splits) + 63) / 64 * 64;
-  const int k0 = kfirst + split * per_split;
+  // The token's keys are counted without the gap: index i is key i for i < kept, else key i + gap.
+  const int kfirst = window.first(pos), kept = window.kept(kfirst), gap = kfirst - kept;
+  const int kend = pos + 1 - gap;
+  const int per_split = (((kend + num_splits - 1) / num_splits) + 63) / 64 * 64;
+  const int k0 = split * per_split;
   const int k1 = min(kend, k0 + per_split);
-  if (k0 < k1) {   // the block-table entries of keys [k0, k1) go to shared memory once
-    const int b0 = k0 / page_size, b1 = (k1 - 1) / page_size;
+  if (k0 < k1 && k1 > kept) {   // the block-table entries of this split's keys behind the gap go to shared memory once
+    const int b0 = (max(k0, kept) + gap) / page_size, b1 = (k1 - 1 + gap) / page_size;
     if (b1 - b0 + 1 <= tbl_cap) {
       for (int i = tid; i <= b1 - b0; i += 128) tbl_s[i] = table_g[b0 + i];
       pm.table = tbl_s;
@@ -389,7 +397,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
       bf16* kd = kd0 + row * LDS + c * 8;
       bf16* vd = kd + 16 * LDS;
       if (k < k1) {
-        const bf16* src = kv_pool + pm.key_row(k, D) + c * 8;
+        const bf16* src = kv_pool + pm.key_row(k < kept ? k : k + gap, D) + c * 8;
         cp_async16(smem_u32(kd), src);
         cp_async16(smem_u32(vd), src + v_off);
       } else {
@@ -527,8 +535,8 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
     }
     if (num_splits == 1) {
       if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-      const float v = L > 0.0f ? O / L : 0.0f;
-      if (turn.table != nullptr) fin_o[row * D + dim] = v;      // turned back below, where the pairs meet
+      const float v = (L > 0.0f ? O / L : 0.0f) * post.factor(t, g * G + row);
+      if (post.table != nullptr) fin_o[row * D + dim] = v;      // turned back below, where the pairs meet
       else out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(v);
     } else {
       fin_o[row * D + dim] = O;
@@ -539,9 +547,9 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
     }
   }
   if (num_splits == 1) {
-    if (turn.table != nullptr) {
+    if (post.table != nullptr) {
       __syncthreads();
-      store_turned<D>(fin_o, out + ((size_t)t * nq + g * G) * D, turn, t, G, tid, 128);
+      store_turned<D>(fin_o, out + ((size_t)t * nq + g * G) * D, post, t, G, tid, 128);
     }
     return;
   }
@@ -576,15 +584,15 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
       }
     }
     if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-    return L > 0.0f ? O / L : 0.0f;
+    return (L > 0.0f ? O / L : 0.0f) * post.factor(t, g * G + row);
   };
-  if (turn.table != nullptr) {                          // a block takes pairs: both elements and the query's angle
+  if (post.table != nullptr) {                          // a block takes pairs: both elements and the query's angle
     const int PS = D / 2 / num_splits;
     for (int idx = tid; idx < G * PS; idx += 128) {
       const int row = idx / PS, m = split * PS + idx % PS;
-      const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + D / 2;
+      const int e0 = post.interleaved ? 2 * m : m, e1 = post.interleaved ? 2 * m + 1 : m + D / 2;
       float u = merged(row, e0), v = merged(row, e1);
-      TurnBack::apply(turn.table[(size_t)t * (D / 2) + m], u, v);
+      HeadOutput::apply(post.table[(size_t)t * (D / 2) + m], u, v);
       bf16* o_row = out + ((size_t)t * nq + g * G + row) * D;
       o_row[e0] = __float2bfloat16_rn(u);
       o_row[e1] = __float2bfloat16_rn(v);
@@ -613,7 +621,7 @@ __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16* __restrict__ q,
                        const int* __restrict__ block_table, const int4* __restrict__ decode_meta,
                        bf16* __restrict__ out, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                       int num_pages, KeyMask window, TurnBack turn, float scale_log2, int tbl_cap, int* __restrict__ error_flag) {
+                       int num_pages, KeyMask window, HeadOutput post, float scale_log2, int tbl_cap, int* __restrict__ error_flag) {
   constexpr int LDS = D + 8;
   constexpr int CPR = D / 8;
   constexpr int HALVES = D / 64;
@@ -651,14 +659,17 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
   const int* table = table_g;
   int blk_base = 0;
 
+  // Tiles start on multiples of 16 so that one lies in one page.  They are counted without the gap between the keys that
+  // stay visible and the window: index i is key i for i < kept, else key i + gap (kept and gap are multiples of 16).
   const int kfirst = window.first(pos);
-  const int kstart = kfirst & ~15;                      // tiles start on multiples of 16 so that one lies in one page
-  const int kend = pos + 1;
-  const int per_split = (((kend - kstart + num_splits - 1) / num_splits) + WARPS * 16 - 1) / (WARPS * 16) * (WARPS * 16);
-  const int k0 = kstart + split * per_split;
+  const int kstart = kfirst & ~15;
+  const int kept = min((window.keep + 15) & ~15, kstart), gap = kstart - kept;
+  const int kend = pos + 1 - gap;
+  const int per_split = (((kend + num_splits - 1) / num_splits) + WARPS * 16 - 1) / (WARPS * 16) * (WARPS * 16);
+  const int k0 = split * per_split;
   const int k1 = min(kend, k0 + per_split);
-  if (k0 < k1) {
-    const int b0 = k0 >> page_shift, b1 = (k1 - 1) >> page_shift;
+  if (k0 < k1 && k1 > kept) {
+    const int b0 = (max(k0, kept) + gap) >> page_shift, b1 = (k1 - 1 + gap) >> page_shift;
     if (b1 - b0 + 1 <= tbl_cap) {
       for (int i = tid; i <= b1 - b0; i += THREADS) tbl_s[i] = table_g[b0 + i];
       table = tbl_s;
@@ -669,10 +680,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
 
   const uint32_t my_stage0 = smem_addr(stage_base) + warp * STAGES * STAGE_BYTES;
   const uint32_t my_bar0 = smem_addr(bars + warp * STAGES);
-  auto issue_tile = [&](int base, int stage) {           // lane 0 only: keys base .. base + 15
-    int page = table[(base >> page_shift) - blk_base];
+  auto issue_tile = [&](int base, int stage) {           // lane 0 only: the 16 keys from index `base` on
+    const int key0 = base < kept ? base : base + gap, blk = key0 >> page_shift;
+    int page = blk >= blk_base ? table[blk - blk_base] : table_g[blk];
     if (page < 0 || page >= num_pages) page = 0;
-    const int off = base & (page_size - 1);
+    const int off = key0 & (page_size - 1);
     const int yk = ((page * 2) * nkv + g) * page_size + off;
     const int yv = ((page * 2 + 1) * nkv + g) * page_size + off;
     const uint32_t dst = my_stage0 + stage * STAGE_BYTES, bar = my_bar0 + 8 * stage;
@@ -694,7 +706,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s) {
       const int base = first_base + s * stride;
-      if (base < k1 && base + 16 <= pos) issue_tile(base, s);       // the tile with the token's own key waits
+      if (base < k1 && base + 16 < kend) issue_tile(base, s);       // the tile with the token's own key waits
     }
   }
   pdl_wait();
@@ -702,7 +714,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s) {
       const int base = first_base + s * stride;
-      if (base < k1 && base + 16 > pos) issue_tile(base, s);
+      if (base < k1 && base + 16 >= kend) issue_tile(base, s);
     }
   }
   for (int i = tid; i < 16 * CPR; i += THREADS) {
@@ -752,8 +764,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
     for (int n = 0; n < 2; ++n) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int key = base + n * 8 + 2 * (lane & 3) + (e & 1);
-        s[n][e] = (key < k1 && key >= kfirst) ? s[n][e] * scale_log2 : -INFINITY;
+        const int idx = base + n * 8 + 2 * (lane & 3) + (e & 1), key = idx < kept ? idx : idx + gap;
+        s[n][e] = (idx < k1 && window.sees(key, kfirst)) ? s[n][e] * scale_log2 : -INFINITY;
       }
       mx_lo = fmaxf(mx_lo, fmaxf(s[n][0], s[n][1]));
       mx_hi = fmaxf(mx_hi, fmaxf(s[n][2], s[n][3]));
@@ -851,8 +863,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
     }
     if (num_splits == 1) {
       if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-      const float v = L > 0.0f ? O / L : 0.0f;
-      if (turn.table != nullptr) fin_o[row * D + dim] = v;      // turned back below, where the pairs meet
+      const float v = (L > 0.0f ? O / L : 0.0f) * post.factor(t, g * G + row);
+      if (post.table != nullptr) fin_o[row * D + dim] = v;      // turned back below, where the pairs meet
       else out[((size_t)t * nq + g * G + row) * D + dim] = __float2bfloat16_rn(v);
     } else {
       fin_o[row * D + dim] = O;
@@ -863,9 +875,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
     }
   }
   if (num_splits == 1) {
-    if (turn.table != nullptr) {
+    if (post.table != nullptr) {
       __syncthreads();
-      store_turned<D>(fin_o, out + ((size_t)t * nq + g * G) * D, turn, t, G, tid, THREADS);
+      store_turned<D>(fin_o, out + ((size_t)t * nq + g * G) * D, post, t, G, tid, THREADS);
     }
     return;
   }
@@ -898,15 +910,15 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
       }
     }
     if (window.sink && M != -INFINITY) L += exp2f(window.sink_log2(g * G + row) - M);
-    return L > 0.0f ? O / L : 0.0f;
+    return (L > 0.0f ? O / L : 0.0f) * post.factor(t, g * G + row);
   };
-  if (turn.table != nullptr) {                          // a block takes pairs: both elements and the query's angle
+  if (post.table != nullptr) {                          // a block takes pairs: both elements and the query's angle
     const int PS = D / 2 / num_splits;
     for (int idx = tid; idx < G * PS; idx += THREADS) {
       const int row = idx / PS, m = split * PS + idx % PS;
-      const int e0 = turn.interleaved ? 2 * m : m, e1 = turn.interleaved ? 2 * m + 1 : m + D / 2;
+      const int e0 = post.interleaved ? 2 * m : m, e1 = post.interleaved ? 2 * m + 1 : m + D / 2;
       float u = merged(row, e0), v = merged(row, e1);
-      TurnBack::apply(turn.table[(size_t)t * (D / 2) + m], u, v);
+      HeadOutput::apply(post.table[(size_t)t * (D / 2) + m], u, v);
       bf16* o_row = out + ((size_t)t * nq + g * G + row) * D;
       o_row[e0] = __float2bfloat16_rn(u);
       o_row[e1] = __float2bfloat16_rn(v);
@@ -924,7 +936,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
 template <int D, int STAGES, int WARPS>
 int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const int* block_table, const int4* decode_meta,
                              bf16* out, int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                             int num_pages, KeyMask window, TurnBack turn, float scale_log2, int num_splits, int max_keys, int* error_flag,
+                             int num_pages, KeyMask window, HeadOutput post, float scale_log2, int num_splits, int max_keys, int* error_flag,
                              cudaStream_t stream) {
   constexpr int stage_bytes = WARPS * STAGES * 2 * 16 * D * 2;
   constexpr int merge_bytes = (WARPS * 16 * D + 2 * WARPS * 16) * 4;
@@ -953,7 +965,7 @@ int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const i
   }
   return launch_pdl(attn_decode_tma_kernel<D, STAGES, WARPS>, dim3(num_items, nkv, num_splits), dim3(WARPS * 32),
                     (size_t)smem, stream, num_splits, pool_map, q, block_table, decode_meta, out, nq, nkv, page_size,
-                    page_shift, max_blocks, num_pages, window, turn, scale_log2, tbl_cap, error_flag);
+                    page_shift, max_blocks, num_pages, window, post, scale_log2, tbl_cap, error_flag);
 }
 
 // Four warps with three 16-key tiles in flight each (96 KB a block at head size 128) feed the HBM when two blocks
@@ -965,13 +977,13 @@ int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const i
 template <int D>
 int launch_decode_tma(const CUtensorMap& pool_map, const bf16* q, const int* block_table, const int4* decode_meta,
                       bf16* out, int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                      int num_pages, KeyMask window, TurnBack turn, float scale_log2, int num_splits, int max_keys, int* error_flag,
+                      int num_pages, KeyMask window, HeadOutput post, float scale_log2, int num_splits, int max_keys, int* error_flag,
                       cudaStream_t stream) {
   constexpr int STAGES = D <= 128 ? 3 : 2;
   const long long blocks = (long long)num_items * nkv * num_splits;
   const int keys_per_block = max_keys / (num_splits > 0 ? num_splits : 1);
 #define ARGS pool_map, q, block_table, decode_meta, out, num_items, nq, nkv, page_size, page_shift, max_blocks, num_pages, \
-             window, turn, scale_log2, num_splits, max_keys, error_flag, stream
+             window, post, scale_log2, num_splits, max_keys, error_flag, stream
   if (D <= 128 && blocks <= 104 && keys_per_block >= 8 * 16) return launch_decode_tma_stages<D, STAGES, 8>(ARGS);
   return launch_decode_tma_stages<D, STAGES, 4>(ARGS);
 #undef ARGS
@@ -980,7 +992,7 @@ int launch_decode_tma(const CUtensorMap& pool_map, const bf16* q, const int* blo
 template <int D>
 int launch_prefill(const bf16* q, const bf16* kv_pool, const int* block_table, const int* tiles, const int* req_slot,
                    bf16* out, int num_tiles, int nq, int nkv, int page_size, int page_shift, int max_blocks,
-                   int num_pages, KeyMask window, TurnBack turn, float scale_log2, int max_keys, cudaStream_t stream) {
+                   int num_pages, KeyMask window, HeadOutput post, float scale_log2, int max_keys, cudaStream_t stream) {
   constexpr int KT = 64;                                // keys per tile
   constexpr int tile_bytes = (64 + 4 * KT) * (D + 8) * 2;
   int tbl_cap = max_keys / page_size + 2;               // entries a tile can need
@@ -994,7 +1006,7 @@ int launch_prefill(const bf16* q, const bf16* kv_pool, const int* block_table, c
   }
   dim3 grid(num_tiles * 4, nq);
   attn_prefill_kernel<D, KT><<<grid, 128, smem, stream>>>(q, kv_pool, block_table, tiles, req_slot, out, nq, nkv, page_size,
-                                                      page_shift, max_blocks, num_pages, window, turn, scale_log2, tbl_cap);
+                                                      page_shift, max_blocks, num_pages, window, post, scale_log2, tbl_cap);
   IFX_CHECK_LAUNCH();
   return 0;
 }
@@ -1002,7 +1014,7 @@ int launch_prefill(const bf16* q, const bf16* kv_pool, const int* block_table, c
 template <int D>
 int launch_decode(const bf16* q, const bf16* kv_pool, const int* block_table, const int4* decode_meta, bf16* out,
                   int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks, int num_pages,
-                  KeyMask window, TurnBack turn, float scale_log2, int num_splits, int max_keys, cudaStream_t stream) {
+                  KeyMask window, HeadOutput post, float scale_log2, int num_splits, int max_keys, cudaStream_t stream) {
   constexpr int STAGES = D <= 128 ? 3 : 2;
   constexpr int stage_bytes = 4 * STAGES * 2 * 16 * (D + 8) * 2;
   constexpr int merge_bytes = (4 * 16 * D + 2 * 4 * 16) * 4;
@@ -1032,7 +1044,7 @@ int launch_decode(const bf16* q, const bf16* kv_pool, const int* block_table, co
   cfg.attrs = attr;
   cfg.numAttrs = num_splits > 1 ? 1 : 0;
   cudaError_t e = cudaLaunchKernelEx(&cfg, attn_decode_kernel<D, STAGES>, q, kv_pool, block_table, decode_meta, out, nq,
-                                     nkv, page_size, page_shift, max_blocks, num_pages, window, turn, scale_log2, tbl_cap);
+                                     nkv, page_size, page_shift, max_blocks, num_pages, window, post, scale_log2, tbl_cap);
   if (e != cudaSuccess) return (int)e;
   return 0;
 }
@@ -1071,17 +1083,17 @@ int ifx_attention_mma_supports(int d) {
 
 // tiles: int32 [num_tiles, 4] = (request index, first flat row, rows <= 256, first position).
 // max_keys: no request of the step holds more keys than this (sizes the shared-memory copy of the block table).
-// chunk, sink: see KeyMask.
+// chunk, sink, keep_first: see KeyMask.  head_gate: null, or float32 [tokens, nq], see HeadOutput.
 // sink_values: null, or one learned number per query head (float32 [nq]) that takes the place of the sink's score 0.
-// turn_back: null, or float2 [tokens, d / 2], see TurnBack.
+// turn_back: null, or float2 [tokens, d / 2], see HeadOutput.
 int ifx_attention_prefill_bf16_sink(const void* q, const void* kv_pool, const int* block_table, const int* tiles,
                                     const int* req_slot, void* out, int num_tiles, int nq, int nkv, int d, int page_size,
                                     int max_blocks, int num_pages, int window_size, int chunk, int sink,
                                     const float* sink_values, float scale, const float* turn_back,
-                                   int turn_interleaved, int max_keys, int* error_flag,
+                                   int turn_interleaved, int keep_first, const float* head_gate, int max_keys, int* error_flag,
                                     cudaStream_t stream) {
-  const KeyMask window{window_size, chunk, sink, sink_values};
-  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
+  const KeyMask window{window_size, chunk, sink, sink_values, keep_first};
+  const HeadOutput post{reinterpret_cast<const float2*>(turn_back), turn_interleaved, head_gate, nq};
   if (num_tiles <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || max_blocks <= 0 || nq > 65535 || !(scale > 0.0f))
     return IFX_E_BADARG;                                  // the kernels take the maximum before scaling
@@ -1089,7 +1101,7 @@ int ifx_attention_prefill_bf16_sink(const void* q, const void* kv_pool, const in
   const int ps = shift_of(page_size);
 #define CALL(DD)                                                                                                   \
   launch_prefill<DD>((const bf16*)q, (const bf16*)kv_pool, block_table, tiles, req_slot, (bf16*)out, num_tiles, nq, \
-                     nkv, page_size, ps, max_blocks, num_pages, window, turn, scale_log2, max_keys, stream)
+                     nkv, page_size, ps, max_blocks, num_pages, window, post, scale_log2, max_keys, stream)
   IFX_DISPATCH_D(d, CALL)
 #undef CALL
 }
@@ -1099,7 +1111,7 @@ int ifx_attention_prefill_bf16_ex(const void* q, const void* kv_pool, const int*
                                   int max_blocks, int num_pages, int window_size, int chunk, int sink, float scale,
                                   int max_keys, int* error_flag, cudaStream_t stream) {
   return ifx_attention_prefill_bf16_sink(q, kv_pool, block_table, tiles, req_slot, out, num_tiles, nq, nkv, d, page_size,
-                                         max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, max_keys, error_flag,
+                                         max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, 0, nullptr, max_keys, error_flag,
                                          stream);
 }
 
@@ -1121,13 +1133,13 @@ int ifx_attention_decode_max_splits(int d, int page_size) {
 // error_flag: device int that the TMA variant sets if a bounded wait runs out (nullptr: cp.async variant only).
 // num_splits: 1, 2, 4 or 8 blocks (one cluster) share a token's key range; it must divide d.  16 where
 // ifx_attention_decode_max_splits says so (the TMA variant, a cluster size beyond the portable 8).
-// max_keys: no token of the step sees more keys than this.
+// max_keys: no token of the step sees more keys than this (keys kept in front of a window included).
 int ifx_attention_decode_bf16_sink(const void* q, const void* kv_pool, const int* block_table, const int* decode_meta,
                                    void* out, int num_items, int nq, int nkv, int d, int page_size, int max_blocks,
                                    int num_pages, int window_size, int chunk, int sink, const float* sink_values, float scale, const float* turn_back,
-                                   int turn_interleaved, int num_splits, int max_keys, int* error_flag, cudaStream_t stream) {
-  const KeyMask window{window_size, chunk, sink, sink_values};
-  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
+                                   int turn_interleaved, int keep_first, const float* head_gate, int num_splits, int max_keys, int* error_flag, cudaStream_t stream) {
+  const KeyMask window{window_size, chunk, sink, sink_values, keep_first};
+  const HeadOutput post{reinterpret_cast<const float2*>(turn_back), turn_interleaved, head_gate, nq};
   if (num_items <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv || nq / nkv > 16 || page_size <= 0 || max_blocks <= 0 || nkv > 65535 ||
       nq > 65535)
@@ -1145,7 +1157,7 @@ int ifx_attention_decode_bf16_sink(const void* q, const void* kv_pool, const int
     if (rc) return rc;
 #define CALL_TMA(DD)                                                                                              \
   return launch_decode_tma<DD>(pool_map, (const bf16*)q, block_table, (const int4*)decode_meta, (bf16*)out,       \
-                               num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn, scale_log2,      \
+                               num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, post, scale_log2,      \
                                num_splits, max_keys, error_flag, stream)
     if (d == 64) CALL_TMA(64);
     if (d == 128) CALL_TMA(128);
@@ -1154,7 +1166,7 @@ int ifx_attention_decode_bf16_sink(const void* q, const void* kv_pool, const int
   }
 #define CALL(DD)                                                                                                  \
   launch_decode<DD>((const bf16*)q, (const bf16*)kv_pool, block_table, (const int4*)decode_meta, (bf16*)out,     \
-                    num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn, scale_log2, num_splits,     \
+                    num_items, nq, nkv, page_size, ps, max_blocks, num_pages, window, post, scale_log2, num_splits,     \
                     max_keys, stream)
   IFX_DISPATCH_D(d, CALL)
 #undef CALL
@@ -1165,7 +1177,7 @@ int ifx_attention_decode_bf16_ex(const void* q, const void* kv_pool, const int* 
                                  int num_pages, int window_size, int chunk, int sink, float scale, int num_splits,
                                  int max_keys, int* error_flag, cudaStream_t stream) {
   return ifx_attention_decode_bf16_sink(q, kv_pool, block_table, decode_meta, out, num_items, nq, nkv, d, page_size,
-                                        max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, num_splits, max_keys,
+                                        max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, 0, nullptr, num_splits, max_keys,
                                         error_flag, stream);
 }
 

@@ -133,7 +133,7 @@ __global__ void __launch_bounds__(kThreads)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap pool_map,
                             const int* __restrict__ block_table, const int* __restrict__ tiles,
                             const int* __restrict__ req_slot, bf16* __restrict__ out, int nq, int nkv, int page_size,
-                            int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn, float scale_log2,
+                            int page_shift, int max_blocks, int num_pages, KeyMask window, HeadOutput post, float scale_log2,
                             int* __restrict__ error_flag) {
   using L = PrefillLayout<D>;
   constexpr int HALVES = L::HALVES, SLOTS = L::SLOTS;
@@ -185,8 +185,17 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
   const int tb_0 = window.first(pos0) / kBN;
   const int te_0 = (pos0 + min(rows, kBM) + kBN - 1) / kBN;
   const int tb_1 = window.first(pos0 + kBM) / kBN;
-  const int te_1 = rows_1 > 0 ? (pos0 + rows + kBN - 1) / kBN : tb_1;
-  const int tb = tb_0, te = max(te_0, te_1);
+  const int te_1 = rows_1 > 0 ? (pos0 + rows + kBN - 1) / kBN : 0;
+  const int te = max(te_0, te_1);
+  // Key tiles in the order they are visited, counted without a gap: [0, nk) with the keys that stay visible in front of the
+  // windows, then [tb_0, te).  Query tile q uses those that hold kept keys and those of its own window.
+  const int keep_tiles = (window.keep + kBN - 1) / kBN, nk = min(keep_tiles, tb_0), tile_gap = tb_0 - nk;
+  const int num_kt = te - tile_gap;
+  auto tile_at = [&](int i) { return i < nk ? i : i + tile_gap; };
+  auto active = [&](int q, int i) {
+    const int kt = tile_at(i);
+    return kt < (q == 0 ? te_0 : te_1) && (kt < keep_tiles || kt >= (q == 0 ? tb_0 : tb_1));
+  };
   const int kfirst = window.first(pos0), kend = pos0 + rows;
 
   if (warp == 0) {
@@ -201,18 +210,20 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     }
     bool ok = true;
     int issued = 0;                                       // slots filled so far
-    for (int kt = tb; kt < te && ok; ++kt) {
+    for (int i = 0; i < num_kt && ok; ++i) {
+      const int kt = tile_at(i);
       // lanes 0-7 take one 16-key block each; its page is looked up before the wait for a free slot
       const int key = kt * kBN + lane * 16;
       int page = 0, off = 0;
-      if (lane < kBN / 16 && key < kend && key + 16 > kfirst) {      // else: any valid page, its keys get weight zero
+      // no visible key among the 16: any valid page, its keys get weight zero
+      if (lane < kBN / 16 && key < kend && (key + 16 > kfirst || key < window.keep)) {
         page = table[key >> page_shift];
         if (page < 0 || page >= num_pages) page = 0;
         off = key & (page_size - 1);
       }
 #pragma unroll 1
       for (int kv = 0; kv < 2; ++kv) {                     // the keys, then the values
-        const int j = 2 * (kt - tb) + kv, s = j % SLOTS;
+        const int j = 2 * i + kv, s = j % SLOTS;
         ok = __all_sync(0xffffffffu, mbar_wait(bar(L::B_EMPTY + s), ((j / SLOTS) & 1) ^ 1));
         if (!ok) break;
         const uint32_t fb = bar(L::B_FULL + s);
@@ -239,11 +250,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                                ((uint32_t)(kBM >> 4) << 24);                       // both operands K-major
       const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(D >> 3) << 17) |
                                ((uint32_t)(kBM >> 4) << 24);                       // B (values) MN-major
-      auto active = [&](int q, int kt) { return q == 0 ? (kt >= tb_0 && kt < te_0) : (kt >= tb_1 && kt < te_1); };
-      auto last_q = [&](int kt) { return active(1, kt) ? 1 : 0; };    // the query tile that uses a key tile last
+      auto last_q = [&](int i) { return active(1, i) ? 1 : 0; };      // the query tile that uses a key tile last
       bool ok = mbar_wait(bar(L::B_Q), 0);
-      auto issue_s = [&](int q, int kt) -> bool {         // S_q = Q_q . K(kt)^T
-        const int j = 2 * (kt - tb), s = j % SLOTS;
+      auto issue_s = [&](int q, int i) -> bool {          // S_q = Q_q . K^T with the i-th key tile
+        const int j = 2 * i, s = j % SLOTS;
         if (!mbar_wait(bar(L::B_FULL + s), (j / SLOTS) & 1)) return false;
         tc_fence_after();
         const uint32_t k_src = kv_s + s * SLOT_BYTES, q_src = q_s + q * Q_BYTES;
@@ -254,12 +264,12 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     desc_kmajor_sw128(k_src + half * kBN * 128) + (inner >> 4), idesc_s, k > 0 ? 1u : 0u);
         }
         umma_commit(bar(L::B_S_FULL + q));
-        if (q == last_q(kt)) umma_commit(bar(L::B_EMPTY + s));      // the keys have been read
+        if (q == last_q(i)) umma_commit(bar(L::B_EMPTY + s));       // the keys have been read
         return true;
       };
       int done[2] = {0, 0};                                // key tiles of each query tile so far
-      auto issue_pv = [&](int q, int kt) -> bool {        // O_q += P_q . V(kt)
-        const int j = 2 * (kt - tb) + 1, s = j % SLOTS;
+      auto issue_pv = [&](int q, int i) -> bool {         // O_q += P_q . V with the i-th key tile
+        const int j = 2 * i + 1, s = j % SLOTS;
         if (!mbar_wait(bar(L::B_P_FULL + q), done[q] & 1) || !mbar_wait(bar(L::B_FULL + s), (j / SLOTS) & 1))
           return false;
         tc_fence_after();
@@ -269,20 +279,20 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
           umma_bf16_ts(tmem_o + q * D, tmem_s + q * kBN + k * 8, desc_mnmajor_sw128(v_src + k * 2048, kBN * 128),
                        idesc_o, (done[q] > 0 || k > 0) ? 1u : 0u);
         umma_commit(bar(L::B_O_FULL + q));
-        if (q == last_q(kt)) umma_commit(bar(L::B_EMPTY + s));      // the values have been read
+        if (q == last_q(i)) umma_commit(bar(L::B_EMPTY + s));       // the values have been read
         ++done[q];
         return true;
       };
       for (int q = 0; q < 2 && ok; ++q)
-        if (active(q, tb)) ok = issue_s(q, tb);
-      for (int kt = tb; kt < te && ok; ++kt) {
+        if (active(q, 0)) ok = issue_s(q, 0);
+      for (int i = 0; i < num_kt && ok; ++i) {
         for (int q = 0; q < 2 && ok; ++q) {
-          if (!active(q, kt)) continue;
-          if (kt != tb && kt == (q == 0 ? tb_0 : tb_1)) ok = issue_s(q, kt);   // a tile that starts later (window)
-          if (ok) ok = issue_pv(q, kt);
+          if (!active(q, i)) continue;
+          if (i > 0 && !active(q, i - 1)) ok = issue_s(q, i);         // a query tile that starts, or goes on, later (window)
+          if (ok) ok = issue_pv(q, i);
           // the next scores of this query tile go over its probabilities: the product that reads them
           // was issued just before and runs first; meanwhile the other tile's softmax is at work
-          if (ok && active(q, kt + 1)) ok = issue_s(q, kt + 1);
+          if (ok && i + 1 < num_kt && active(q, i + 1)) ok = issue_s(q, i + 1);
         }
       }
       if (!ok) atomicExch(error_flag, 8);
@@ -297,18 +307,19 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     const int pos0_q = pos0 + q * kBM;
     const int pos = pos0_q + row;
     const int wfirst = window.first(pos);
-    const int tb_q = q == 0 ? tb_0 : tb_1, te_q = q == 0 ? te_0 : te_1;
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const uint32_t s_addr = tmem_s + q * kBN + lane_addr, o_addr = tmem_o + q * D + lane_addr;
     float m_ref = -INFINITY, l_run = 0.0f;
     bool ok = true;
-    int i = 0;
-    for (int kt = tb_q; kt < te_q; ++kt, ++i) {
-      const int key0 = kt * kBN;
+    int i = 0;                                            // key tiles of this query tile so far
+    for (int n = 0; n < num_kt; ++n) {
+      if (!active(q, n)) continue;
+      const int key0 = tile_at(n) * kBN;
       ok = __all_sync(0xffffffffu, mbar_wait(bar(L::B_S_FULL + q), i & 1));
       if (!ok) break;
       tc_fence_after();
-      const bool edge = key0 + kBN - 1 > pos0_q || (window.any() && key0 < window.first(pos0_q + kBM - 1));
+      const bool edge = key0 + kBN - 1 > pos0_q ||
+                        (window.any() && key0 < window.first(pos0_q + kBM - 1) && key0 + kBN > window.keep);
       // pass 1: the row's maximum
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -321,7 +332,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 #pragma unroll
           for (int j = 0; j < 64; ++j) {
             const int key = key0 + c + j;
-            if (key > pos || key < wfirst) s[j] = -INFINITY;
+            if (key > pos || !window.sees(key, wfirst)) s[j] = -INFINITY;
           }
         }
 #pragma unroll
@@ -367,7 +378,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 #pragma unroll
           for (int j = 0; j < 64; ++j) {
             const int key = key0 + c + j;
-            if (key > pos || key < wfirst) s[j] = -INFINITY;
+            if (key > pos || !window.sees(key, wfirst)) s[j] = -INFINITY;
           }
         }
         uint32_t packed[32];
@@ -386,39 +397,40 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(bar(L::B_P_FULL + q));
+      ++i;
     }
     if (ok && i > 0) ok = __all_sync(0xffffffffu, mbar_wait(bar(L::B_O_FULL + q), (i - 1) & 1));
     if (!ok && lane == 0) atomicExch(error_flag, 9);
     if (ok && i > 0) {
       tc_fence_after();
       if (window.sink && m_ref > -INFINITY) l_run += exp2f(window.sink_log2(h) - m_ref * scale_log2);     // the sink's share
-      const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+      const float inv = (l_run > 0.0f ? 1.0f / l_run : 0.0f) * post.factor(row0 + q * kBM + min(row, max(rows_q - 1, 0)), h);
       bf16* dst = out + ((size_t)(row0 + q * kBM + row) * nq + h) * D;
-      if (turn.table != nullptr) {                         // 16 pairs at a time: 32 columns, or 16 and their 16 partners
-        const float4* cs4 = reinterpret_cast<const float4*>(turn.table + (size_t)(row0 + q * kBM + min(row, max(rows_q - 1, 0))) * (D / 2));
-        const int apart = turn.interleaved ? 16 : D / 2;
+      if (post.table != nullptr) {                         // 16 pairs at a time: 32 columns, or 16 and their 16 partners
+        const float4* cs4 = reinterpret_cast<const float4*>(post.table + (size_t)(row0 + q * kBM + min(row, max(rows_q - 1, 0))) * (D / 2));
+        const int apart = post.interleaved ? 16 : D / 2;
 #pragma unroll 1
         for (int m0 = 0; m0 < D / 2; m0 += 16) {
-          const int c = turn.interleaved ? 2 * m0 : m0;
+          const int c = post.interleaved ? 2 * m0 : m0;
           float lo[16], hi[16];
           tmem_ld16f(o_addr + c, lo);
           tmem_ld16f(o_addr + c + apart, hi);
           tmem_wait_ld();
-          if (turn.interleaved) {
+          if (post.interleaved) {
 #pragma unroll
             for (int j = 0; j < 8; j += 2) {
               const float4 a = cs4[(m0 + j) >> 1], b = cs4[(m0 + 8 + j) >> 1];
-              TurnBack::apply(make_float2(a.x, a.y), lo[2 * j], lo[2 * j + 1]);
-              TurnBack::apply(make_float2(a.z, a.w), lo[2 * j + 2], lo[2 * j + 3]);
-              TurnBack::apply(make_float2(b.x, b.y), hi[2 * j], hi[2 * j + 1]);
-              TurnBack::apply(make_float2(b.z, b.w), hi[2 * j + 2], hi[2 * j + 3]);
+              HeadOutput::apply(make_float2(a.x, a.y), lo[2 * j], lo[2 * j + 1]);
+              HeadOutput::apply(make_float2(a.z, a.w), lo[2 * j + 2], lo[2 * j + 3]);
+              HeadOutput::apply(make_float2(b.x, b.y), hi[2 * j], hi[2 * j + 1]);
+              HeadOutput::apply(make_float2(b.z, b.w), hi[2 * j + 2], hi[2 * j + 3]);
             }
           } else {
 #pragma unroll
             for (int j = 0; j < 16; j += 2) {
               const float4 a = cs4[(m0 + j) >> 1];
-              TurnBack::apply(make_float2(a.x, a.y), lo[j], hi[j]);
-              TurnBack::apply(make_float2(a.z, a.w), lo[j + 1], hi[j + 1]);
+              HeadOutput::apply(make_float2(a.x, a.y), lo[j], hi[j]);
+              HeadOutput::apply(make_float2(a.z, a.w), lo[j + 1], hi[j + 1]);
             }
           }
           if (row < rows_q) {
@@ -467,7 +479,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 template <int D>
 static int launch_prefill_tcgen05(const bf16* q, int num_tokens, const bf16* kv_pool, const int* block_table,
                                   const int* tiles, const int* req_slot, bf16* out, int num_tiles, int nq, int nkv,
-                                  int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, TurnBack turn,
+                                  int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, HeadOutput post,
                                   float scale_log2, int* error_flag, cudaStream_t stream) {
   CUtensorMap q_map, pool_map;
   int rc = make_tensor_map_bf16(&q_map, q, num_tokens, nq * D, kBM);
@@ -484,7 +496,7 @@ static int launch_prefill_tcgen05(const bf16* q, int num_tokens, const bf16* kv_
   }
   return launch_pdl(attn_prefill_tcgen05_kernel<D>, dim3(nq, num_tiles), dim3(kThreads), smem, stream, 1, q_map,
                     pool_map, block_table, tiles, req_slot, out, nq, nkv, page_size, page_shift, max_blocks,
-                    num_pages, window, turn, scale_log2, error_flag);
+                    num_pages, window, post, scale_log2, error_flag);
 }
 
 }  // namespace ifx
@@ -500,16 +512,17 @@ int ifx_attention_prefill_tcgen05_supports(int d, int page_size) {
 
 // q [num_tokens, nq * d] bfloat16, 16-byte aligned.  tiles: int32 [num_tiles, 4] = (request index, first
 // flat row, rows <= 256, first position).
-// chunk, sink: see KeyMask (common.cuh).
+// chunk, sink, keep_first: see KeyMask; head_gate: null, or float32 [tokens, nq], see HeadOutput (common.cuh).
 // sink_values: null, or one learned number per query head (float32 [nq]) that takes the place of the sink's score 0.
-// turn_back: null, or float2 [tokens, d / 2], see TurnBack.
+// turn_back: null, or float2 [tokens, d / 2], see HeadOutput.
 int ifx_attention_prefill_tcgen05_sink(const void* q, int num_tokens, const void* kv_pool, const int* block_table,
                                        const int* tiles, const int* req_slot, void* out, int num_tiles, int nq, int nkv,
                                        int d, int page_size, int max_blocks, int num_pages, int window_size, int chunk,
                                        int sink, const float* sink_values, float scale, const float* turn_back,
-                                   int turn_interleaved, int* error_flag, cudaStream_t stream) {
-  const KeyMask window{window_size, chunk, sink, sink_values};
-  const TurnBack turn{reinterpret_cast<const float2*>(turn_back), turn_interleaved};
+                                   int turn_interleaved, int keep_first, const float* head_gate, int* error_flag,
+                                       cudaStream_t stream) {
+  const KeyMask window{window_size, chunk, sink, sink_values, keep_first};
+  const HeadOutput post{reinterpret_cast<const float2*>(turn_back), turn_interleaved, head_gate, nq};
   if (num_tiles <= 0) return 0;
   if (!ifx_attention_prefill_tcgen05_supports(d, page_size) || nq <= 0 || nkv <= 0 || nq % nkv || max_blocks <= 0 ||
       num_tiles > 65535 || !(scale > 0.0f) || error_flag == nullptr)
@@ -519,10 +532,10 @@ int ifx_attention_prefill_tcgen05_sink(const void* q, int num_tokens, const void
   const float scale_log2 = scale * 1.4426950408889634f;
   if (d == 64)
     return launch_prefill_tcgen05<64>((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot,
-                                      (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn,
+                                      (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, post,
                                       scale_log2, error_flag, stream);
   return launch_prefill_tcgen05<128>((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot,
-                                     (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, turn,
+                                     (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, post,
                                      scale_log2, error_flag, stream);
 }
 
@@ -531,7 +544,7 @@ int ifx_attention_prefill_tcgen05_ex(const void* q, int num_tokens, const void* 
                                      int d, int page_size, int max_blocks, int num_pages, int window_size, int chunk,
                                      int sink, float scale, int* error_flag, cudaStream_t stream) {
   return ifx_attention_prefill_tcgen05_sink(q, num_tokens, kv_pool, block_table, tiles, req_slot, out, num_tiles, nq, nkv, d,
-                                            page_size, max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, error_flag,
+                                            page_size, max_blocks, num_pages, window_size, chunk, sink, nullptr, scale, nullptr, 0, 0, nullptr, error_flag,
                                             stream);
 }
 

@@ -79,11 +79,13 @@ inline int launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t sm
 }
 
 // Which keys a query sees besides "not later than itself": the last `window` of them (> 0), only those of its own
-// stretch of `chunk` positions (> 0), or both; `sink`: the softmax's denominator holds one more unit, a key of score 0
+// stretch of `chunk` positions (> 0), or both; the first `keep` keys of a sequence stay visible whatever the window or the
+// stretch.  A query's keys are therefore [0, kept(first)) and [first, pos].  `sink`: the softmax's denominator holds one more unit, a key of score 0
 // that brings no value; with `sink_values` (one learned number per query head) the unit is exp(that number) instead.
 struct KeyMask {
   int window, chunk, sink;
   const float* sink_values;
+  int keep;
   // the sink's score in units of log2, for kernels that keep maxima and sums as powers of two
   __device__ __forceinline__ float sink_log2(int head) const {
     return sink_values ? sink_values[head] * 1.4426950408889634f : 0.0f;
@@ -94,14 +96,23 @@ struct KeyMask {
     return f;
   }
   __device__ __forceinline__ bool any() const { return window > 0 || chunk > 0; }
+  __device__ __forceinline__ int kept(int first) const { return min(keep, first); }      // keys in front of `first` that stay
+  __device__ __forceinline__ bool sees(int key, int first) const { return key >= first || key < keep; }
 };
 
+// What happens to a head's finished sum of values before it is rounded and stored.
 // Values that were turned by their own position before they were summed: the sum is turned back by the query's.  `table`
 // [tokens, size / 2] holds cos and sin of the query's angles (null: nothing is turned); pairs are (m, m + size / 2), or
 // neighbours with `interleaved`.
-struct TurnBack {
+// A gate per token and head: the sum is multiplied by gate[token, head] of `heads` a row (null: 1).
+struct HeadOutput {
   const float2* table;
   int interleaved;
+  const float* gate;
+  int heads;
+  __device__ __forceinline__ float factor(int token, int head) const {
+    return gate ? gate[(size_t)token * heads + head] : 1.0f;
+  }
   __device__ __forceinline__ static void apply(float2 cs, float& u, float& v) {
     const float a = u * cs.x + v * cs.y, b = v * cs.x - u * cs.y;
     u = a;

@@ -43,7 +43,7 @@ constexpr int kTileK = 64;        // bf16 elements per k-block = one 128-byte sw
 
 enum { MODE_STORE = 0, MODE_PARTIAL = 1, MODE_SWIGLU = 2, MODE_SWIGLU64 = 3 };
 // an activation on the stored result of MODE_STORE, or (GEGLU) in place of SiLU on the gate of MODE_SWIGLU / SWIGLU64
-enum { ACT_NONE = 0, ACT_XIELU = 1, ACT_GEGLU = 2 };
+enum { ACT_NONE = 0, ACT_XIELU = 1, ACT_GEGLU = 2, ACT_RELU2 = 3 };
 
 __device__ __forceinline__ uint64_t make_smem_desc(uint32_t addr) {
   // K-major tile of 128-byte rows, 128-byte swizzle: 8-row groups 1024 bytes apart.
@@ -264,6 +264,7 @@ gemm_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             float r = GLU ? v : v + b;
             if (MODE == MODE_STORE && act_kind == ACT_XIELU)     // a z^2 + z/2 above zero, b (e^z - 1 - z) + z/2 below
               r = r > 0.0f ? fmaf(act_a * r, r, 0.5f * r) : fmaf(act_b, (__expf(r) - 1.0f) - r, 0.5f * r);
+            if (MODE == MODE_STORE && act_kind == ACT_RELU2) r = fmaxf(r, 0.0f) * fmaxf(r, 0.0f);
             if (out_is_f32) reinterpret_cast<float*>(out)[(size_t)m * N + n] = r;
             else reinterpret_cast<__nv_bfloat16*>(out)[(size_t)m * N + n] = __float2bfloat16_rn(r);
           }
@@ -371,7 +372,7 @@ static int gemm_skinny_any(const void* act, const void* W, const float* bias, vo
                           const float* row_sumsq, int sumsq_chunks, float eps, int* error_flag, cudaStream_t stream,
                           int act_kind, float act_a, float act_b) {
   if (M <= 0 || N <= 0) return 0;
-  if (act_kind != ACT_NONE && !(act_kind == ACT_XIELU && mode == MODE_STORE) && !(act_kind == ACT_GEGLU && mode == MODE_SWIGLU))
+  if (act_kind != ACT_NONE && !((act_kind == ACT_XIELU || act_kind == ACT_RELU2) && mode == MODE_STORE) && !(act_kind == ACT_GEGLU && mode == MODE_SWIGLU))
     return IFX_E_BADARG;
   if (K <= 0 || M > 256 || splits <= 0 || splits > 65535 || error_flag == nullptr) return IFX_E_BADARG;
   if (mode == MODE_STORE && splits != 1) return IFX_E_BADARG;
@@ -414,7 +415,7 @@ extern "C" int ifx_gemm_skinny(const void* act, const void* W, const float* bias
 }
 
 // mode 0 with an activation on the result before it is stored: act_kind 1 = xIELU with its two factors
-// (act_a z^2 + z/2 for z > 0, act_b (e^z - 1 - z) + z/2 otherwise).
+// (act_a z^2 + z/2 for z > 0, act_b (e^z - 1 - z) + z/2 otherwise), 3 = max(z, 0)^2.
 extern "C" int ifx_gemm_skinny_act(const void* act, const void* W, const float* bias, void* out, int M, int N, int K,
                                    int w_rows, int out_is_f32, const float* row_sumsq, int sumsq_chunks, float eps,
                                    int act_kind, float act_a, float act_b, int* error_flag, cudaStream_t stream) {

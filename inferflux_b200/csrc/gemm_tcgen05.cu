@@ -7,6 +7,7 @@
 //            out[m, n] = silu(acc_gate) * acc_up               (bfloat16; no [M, 2N] round trip,
 //                                                               no separate activation kernel)
 //   GEGLU    the same with gelu(acc_gate + bias) * (acc_up + bias), the tanh form
+//   RELU2    out[m, n] = max(acc, 0)^2                         (bfloat16)
 //   GROUP_RELU2  rows are sorted into groups of whole 128-row tiles; tile mt multiplies with the weight rows
 //            [tile_group[mt] * group_rows, + N) of a stack of matrices (a negative entry: the tile is unused and
 //            skipped);  out[m, n] = relu(acc)^2                 (bfloat16)
@@ -35,7 +36,7 @@ namespace ifx {
 constexpr int kBM = 128, kBN = 256, kBK = 64, kGemmStages = 4;
 constexpr uint32_t kABytes = kBM * kBK * 2, kBBytes = kBN * kBK * 2, kStageBytes = kABytes + kBBytes;
 
-enum { GEMM_STORE = 0, GEMM_SWIGLU = 1, GEMM_GROUP_RELU2 = 2, GEMM_GROUP_SCALE = 3, GEMM_GROUP_GLU = 4, GEMM_GEGLU = 5 };
+enum { GEMM_STORE = 0, GEMM_SWIGLU = 1, GEMM_GROUP_RELU2 = 2, GEMM_GROUP_SCALE = 3, GEMM_GROUP_GLU = 4, GEMM_GEGLU = 5, GEMM_RELU2 = 6 };
 
 __device__ __forceinline__ uint64_t gemm_smem_desc(uint32_t addr) {
   // K-major tile of 128-byte rows, 128-byte swizzle: 8-row groups 1024 bytes apart.
@@ -216,7 +217,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             const float up = fminf(fmaxf(__uint_as_float(u[j]), -glu_limit), glu_limit);
             v[j] = __fdividef(gate, 1.0f + __expf(-glu_slope * gate)) * (up + glu_offset);
           }
-          if (MODE == GEMM_GROUP_RELU2) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
+          if (MODE == GEMM_GROUP_RELU2 || MODE == GEMM_RELU2) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
           if (MODE == GEMM_GROUP_SCALE) v[j] *= factor;
         }
         if (MODE == GEMM_GROUP_SCALE) {
@@ -295,19 +296,21 @@ using namespace ifx;
 
 // act [M, K] and W [w_rows, K] bfloat16, K % 8 == 0, both 16-byte aligned; out [M, N] bfloat16.
 // mode 0: out = act . W[:N]^T.   mode 1: out = silu(act . W[:N]^T) * (act . W[up_row_offset : up_row_offset + N]^T).
+// mode 6: out = max(act . W[:N]^T, 0)^2.
 // error_flag: device int, set to non-zero if a bounded wait ran out (the output is then not valid).
 extern "C" int ifx_gemm_tcgen05(const void* act, const void* W, void* out, int M, int N, int K, int w_rows, int mode,
                                 int up_row_offset, int* error_flag, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || error_flag == nullptr || out == nullptr) return IFX_E_BADARG;
   if (mode == GEMM_SWIGLU && (up_row_offset < N || up_row_offset + N > w_rows)) return IFX_E_BADARG;
-  if (mode == GEMM_STORE && N > w_rows) return IFX_E_BADARG;
+  if ((mode == GEMM_STORE || mode == GEMM_RELU2) && N > w_rows) return IFX_E_BADARG;
   CUtensorMap ma, mw;
   int rc = weight_tensor_map(&mw, W, w_rows, K, 128);
   if (rc) return rc;
   rc = make_tensor_map_bf16(&ma, act, M, K, kBM);
   if (rc) return rc;
   if (mode == GEMM_STORE) return launch_gemm<GEMM_STORE>(ma, mw, out, M, N, K, 0, error_flag, stream);
+  if (mode == GEMM_RELU2) return launch_gemm<GEMM_RELU2>(ma, mw, out, M, N, K, 0, error_flag, stream);
   if (mode == GEMM_SWIGLU) return launch_gemm<GEMM_SWIGLU>(ma, mw, out, M, N, K, up_row_offset, error_flag, stream);
   return IFX_E_BADARG;
 }

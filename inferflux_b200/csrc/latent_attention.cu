@@ -13,7 +13,8 @@
 // cached latents, and the head's value projection is applied once to the sum.  Scores,
 // softmax weights, the running maximum, sum and accumulator are float32.  A sink is
 // a learned score per head with no key and no value: it only enlarges the
-// denominator, once.  Without sinks (null) the softmax is the usual one.
+// denominator, once.  Without sinks (null) the softmax is the usual one.  A gate per token and head (null: none)
+// multiplies the weighted sum of latents, and with it the head's output, which is linear in it.
 //
 // latent_attention_generic: one warp per (token, head), keys in chunks of 32 from
 // the window's start in increasing position, so the order of every addition depends
@@ -65,7 +66,8 @@ __global__ void latent_norm_append_kernel(const T* __restrict__ rows, int ld, in
 // dim + rot in `q`, rows ldq apart) are turned the same way and written to q_out (rows ld_out apart, heads head_stride
 // apart, at `out_offset` in a head): q itself, or the tail of a query in latent space.  The first `rot_used` of the
 // `rot` elements turn (pair i is (2i, 2i + 1) when interleaved, else (i, i + rot_used / 2)); angle = position *
-// inv_freq[i] in float32, cos and sin times `magnitude`.
+// inv_freq[i] in float32, cos and sin times `magnitude`.  With `gate_out` [T, heads]: sigmoid of the columns gate_col ..
+// gate_col + heads of `rows`, in float32.
 template <typename T>
 __device__ __forceinline__ void turn_store(const T* src, T* dst, int rot, int rot_used, int interleaved,
                                            const float* __restrict__ cs, float* __restrict__ held, int lane) {
@@ -93,7 +95,8 @@ __global__ void latent_rope_append_kernel(const T* __restrict__ rows, int ld, in
                                           const int* __restrict__ positions, const int* __restrict__ token_req,
                                           const int* __restrict__ req_slot, const int* __restrict__ block_table,
                                           int max_blocks, int page_size, int num_pages, T* __restrict__ pool,
-                                          int num_tokens, int lat, int rot, int heads, int dim) {
+                                          int num_tokens, int lat, int rot, int heads, int dim,
+                                          float* __restrict__ gate_out, int gate_col) {
   extern __shared__ float cs_s[];                        // per warp: cos and sin of the token's angles, then `rot` staged numbers
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -108,6 +111,9 @@ __global__ void latent_rope_append_kernel(const T* __restrict__ rows, int ld, in
     cs[i] = c * magnitude;
     cs[half + i] = sn * magnitude;
   }
+  if (gate_out != nullptr)
+    for (int h = lane; h < heads; h += 32)
+      gate_out[(size_t)t * heads + h] = 1.0f / (1.0f + expf(-to_f32(rows[(size_t)t * ld + gate_col + h])));
   __syncwarp();
   const T* x = rows + (size_t)t * ld + col0;
   float ss = 0.0f;
@@ -141,7 +147,7 @@ __global__ void __launch_bounds__(kLatentWarps * 32) latent_attention_generic_ke
     const float* __restrict__ sinks, const T* __restrict__ pool, const int* __restrict__ block_table,
     const int* __restrict__ positions, const int* __restrict__ token_req, const int* __restrict__ req_slot,
     const int* __restrict__ rows, T* __restrict__ out, int num_tokens, int heads, int dim, int vdim, int lat,
-    int page_size, int max_blocks, int num_pages, int window, float scale, int rot) {
+    int page_size, int max_blocks, int num_pages, int window, float scale, int rot, const float* __restrict__ gate) {
   // `lat`: numbers of a latent; `rot`: numbers behind it in every cached row and behind the `dim` plain ones of every
   // query head, which meet each other directly.  `rank` is the cached row: the kernel's sums run over all of it.
   extern __shared__ float lat_s[];                       // per warp: `rank` floats (query in latent space, then the sum)
@@ -225,7 +231,7 @@ __global__ void __launch_bounds__(kLatentWarps * 32) latent_attention_generic_ke
 #pragma unroll
     for (int i = 0; i < NR; ++i) acc[i] *= corr;
   }
-  const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+  const float inv = (l > 0.0f ? 1.0f / l : 0.0f) * (gate != nullptr ? gate[(size_t)t * heads + h] : 1.0f);
   __syncwarp();
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
@@ -281,8 +287,9 @@ int ifx_latent_rope_append(const void* rows, int ld, int col0, const float* w, f
                            int ld_out, int head_stride, int out_offset, const float* inv_freq, int rot_used, int interleaved,
                            float magnitude, const int* positions, const int* token_req, const int* req_slot,
                            const int* block_table, int max_blocks, int page_size, int num_pages, void* pool, int T, int lat,
-                           int rot, int heads, int dim, int dtype, cudaStream_t stream) {
+                           int rot, int heads, int dim, float* gate_out, int gate_col, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (gate_out != nullptr && (gate_col < 0 || gate_col + heads > ld)) return IFX_E_BADARG;
   if (lat <= 0 || rot < 0 || col0 < 0 || ld < col0 + lat + rot || heads <= 0 || dim < 0 || ldq < heads * (dim + rot) ||
       rot_used < 0 || rot_used > rot || (rot_used & 1) || (rot_used > 0 && inv_freq == nullptr))
     return IFX_E_BADARG;
@@ -294,12 +301,12 @@ int ifx_latent_rope_append(const void* rows, int ld, int col0, const float* w, f
     latent_rope_append_kernel<float><<<blocks, warps * 32, smem, stream>>>(
         (const float*)rows, ld, col0, w, eps, (const float*)q, ldq, (float*)q_out, ld_out, head_stride, out_offset, inv_freq,
         rot_used, interleaved, magnitude, positions, token_req, req_slot, block_table, max_blocks, page_size, num_pages,
-        (float*)pool, T, lat, rot, heads, dim);
+        (float*)pool, T, lat, rot, heads, dim, gate_out, gate_col);
   else if (dtype == IFX_DT_BF16)
     latent_rope_append_kernel<__nv_bfloat16><<<blocks, warps * 32, smem, stream>>>(
         (const __nv_bfloat16*)rows, ld, col0, w, eps, (const __nv_bfloat16*)q, ldq, (__nv_bfloat16*)q_out, ld_out,
         head_stride, out_offset, inv_freq, rot_used, interleaved, magnitude, positions, token_req, req_slot, block_table,
-        max_blocks, page_size, num_pages, (__nv_bfloat16*)pool, T, lat, rot, heads, dim);
+        max_blocks, page_size, num_pages, (__nv_bfloat16*)pool, T, lat, rot, heads, dim, gate_out, gate_col);
   else return IFX_E_DTYPE;
   IFX_CHECK_LAUNCH();
   return 0;
@@ -311,8 +318,8 @@ int ifx_latent_attention_generic_rot(const void* q, int ldq, const void* w_uk, c
                                      const void* pool, const int* block_table, const int* positions,
                                      const int* token_req, const int* req_slot, const int* rows, void* out,
                                      int num_tokens, int heads, int dim, int vdim, int lat, int page_size,
-                                     int max_blocks, int num_pages, int window, float scale, int rot, int dtype,
-                                     cudaStream_t stream);
+                                     int max_blocks, int num_pages, int window, float scale, int rot, const float* gate,
+                                     int dtype, cudaStream_t stream);
 
 int ifx_latent_attention_generic(const void* q, int ldq, const void* w_uk, const void* w_uv, const float* sinks,
                                  const void* pool, const int* block_table, const int* positions,
@@ -322,17 +329,18 @@ int ifx_latent_attention_generic(const void* q, int ldq, const void* w_uk, const
                                  cudaStream_t stream) {
   return ifx_latent_attention_generic_rot(q, ldq, w_uk, w_uv, sinks, pool, block_table, positions, token_req, req_slot, rows,
                                           out, num_tokens, heads, dim, vdim, rank, page_size, max_blocks, num_pages, window,
-                                          scale, 0, dtype, stream);
+                                          scale, 0, nullptr, dtype, stream);
 }
 
 // The same with `rot` numbers behind the latent in every cached row (rows of lat + rot) and behind the `dim` plain
 // elements of every query head (heads of dim + rot in q); w_uk [heads * dim, lat], w_uv [heads * vdim, lat].
+// gate: null, or float32 [num_tokens, heads].
 int ifx_latent_attention_generic_rot(const void* q, int ldq, const void* w_uk, const void* w_uv, const float* sinks,
                                      const void* pool, const int* block_table, const int* positions,
                                      const int* token_req, const int* req_slot, const int* rows, void* out,
                                      int num_tokens, int heads, int dim, int vdim, int lat, int page_size,
-                                     int max_blocks, int num_pages, int window, float scale, int rot, int dtype,
-                                     cudaStream_t stream) {
+                                     int max_blocks, int num_pages, int window, float scale, int rot, const float* gate,
+                                     int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (heads <= 0 || dim <= 0 || vdim <= 0 || lat <= 0 || rot < 0 || page_size <= 0 || max_blocks <= 0 ||
       ldq < heads * (dim + rot))
@@ -346,7 +354,7 @@ int ifx_latent_attention_generic_rot(const void* q, int ldq, const void* w_uk, c
   latent_attention_generic_kernel<TT, NR><<<blocks, kLatentWarps * 32, smem, stream>>>(                            \
       (const TT*)q, ldq, (const TT*)w_uk, (const TT*)w_uv, sinks, (const TT*)pool, block_table, positions,         \
       token_req, req_slot, rows, (TT*)out, num_tokens, heads, dim, vdim, lat, page_size, max_blocks, num_pages,    \
-      window, scale, rot)
+      window, scale, rot, gate)
 #define IFX_BY_RANK(TT)                          \
   do {                                           \
     if (rank <= 64) IFX_LAUNCH(TT, 2);           \

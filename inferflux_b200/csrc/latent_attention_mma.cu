@@ -65,7 +65,8 @@ __global__ void __launch_bounds__(128, 3) latent_attention_mma_kernel(   // 32 .
     const __nv_bfloat16* __restrict__ ql, const __nv_bfloat16* __restrict__ pool, const int* __restrict__ block_table,
     const int4* __restrict__ items, const float* __restrict__ sinks, __nv_bfloat16* __restrict__ out,
     float* __restrict__ part_o, float2* __restrict__ part_ml, int total_rows, int heads, int rank, int page_size,
-    int max_blocks, int num_pages, int window, float scale_log2, int QT, int HC, int subs, int splits, int rot) {
+    int max_blocks, int num_pages, int window, float scale_log2, int QT, int HC, int subs, int splits, int rot,
+    const float* __restrict__ gate) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int kw = rank + rot;                                           // a cached row, a query row
   const int stride = kw + kPad;                                        // elements per shared row
@@ -276,7 +277,7 @@ __global__ void __launch_bounds__(128, 3) latent_attention_mma_kernel(   // 32 .
         c = exp2f(m - mn);
         l = l * c + exp2f(sk - mn);
       }
-      const float inv = l > 0.0f ? c / l : 0.0f;
+      const float inv = (l > 0.0f ? c / l : 0.0f) * (gate != nullptr ? gate[grow] : 1.0f);
       __nv_bfloat16* orow = out + grow * rank;
 #pragma unroll
       for (int i = 0; i < NT; ++i)
@@ -295,7 +296,7 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const float* __restri
                                                            const float2* __restrict__ part_ml,
                                                            const float* __restrict__ sinks,
                                                            __nv_bfloat16* __restrict__ out, int total_rows, int heads,
-                                                           int rank, int splits) {
+                                                           int rank, int splits, const float* __restrict__ gate) {
   __shared__ float w_s[kMaxSplits];
   __shared__ float inv_s;
   const int row = blockIdx.x, c = threadIdx.x;
@@ -320,7 +321,7 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const float* __restri
     }
     l = warp_sum(l);
     if (sk != -INFINITY) l += exp2f(sk - m);
-    if (c == 0) inv_s = l > 0.0f ? 1.0f / l : 0.0f;
+    if (c == 0) inv_s = (l > 0.0f ? 1.0f / l : 0.0f) * (gate != nullptr ? gate[row] : 1.0f);
   }
   __syncthreads();
   if (c >= rank) return;
@@ -359,11 +360,11 @@ long long ifx_latent_attention_mma_workspace(int total_rows, int rank, int split
 
 // ql: [T, heads, rank + rot], out: [T, heads, rank] bfloat16; cached rows of rank + rot.  items: [num_items, 4]
 // (slot, first flat token, tokens <= 64, first position).  max_item_tokens: the largest token count among the items.
-// workspace: as ifx_latent_attention_mma_workspace says.
+// workspace: as ifx_latent_attention_mma_workspace says.  gate: null, or float32 [T, heads], which multiplies the sums.
 int ifx_latent_attention_mma_rot(const void* ql, const void* pool, const int* block_table, const int* items, int num_items,
                                  int max_item_tokens, const float* sinks, void* out, void* workspace, int T, int heads,
                                  int rank, int rot, int page_size, int max_blocks, int num_pages, int window, float scale,
-                                 int splits, cudaStream_t stream) {
+                                 int splits, const float* gate, cudaStream_t stream) {
   if (num_items <= 0 || T <= 0) return 0;
   if (!ifx_latent_attention_mma_supports_rot(rank, rot) || heads <= 0 || page_size <= 0 || max_blocks <= 0 || splits < 1 ||
       max_item_tokens < 1 || max_item_tokens > 64 || splits > kMaxSplits)
@@ -388,7 +389,7 @@ int ifx_latent_attention_mma_rot(const void* ql, const void* pool, const int* bl
     kern<<<grid, nwarps * 32, smem, stream>>>((const __nv_bfloat16*)ql, (const __nv_bfloat16*)pool, block_table,            \
                                       (const int4*)items, sinks, (__nv_bfloat16*)out, part_o, part_ml, total_rows,  \
                                       heads, rank, page_size, max_blocks, num_pages, window, scale_log2, QT, HC,    \
-                                      subs, splits, rot);                                                           \
+                                      subs, splits, rot, gate);                                                         \
   } while (0)
   if (rot == 0) {
     if (rank <= 64) IFX_LAUNCH(64, 0);
@@ -403,7 +404,7 @@ int ifx_latent_attention_mma_rot(const void* ql, const void* pool, const int* bl
   IFX_CHECK_LAUNCH();
   if (splits > 1) {
     latent_merge_kernel<<<total_rows, 256, 0, stream>>>(
-        part_o, part_ml, sinks, (__nv_bfloat16*)out, total_rows, heads, rank, splits);
+        part_o, part_ml, sinks, (__nv_bfloat16*)out, total_rows, heads, rank, splits, gate);
     IFX_CHECK_LAUNCH();
   }
   return 0;
@@ -414,7 +415,7 @@ int ifx_latent_attention_mma(const void* ql, const void* pool, const int* block_
                              int rank, int page_size, int max_blocks, int num_pages, int window, float scale,
                              int splits, cudaStream_t stream) {
   return ifx_latent_attention_mma_rot(ql, pool, block_table, items, num_items, max_item_tokens, sinks, out, workspace, T,
-                                      heads, rank, 0, page_size, max_blocks, num_pages, window, scale, splits, stream);
+                                      heads, rank, 0, page_size, max_blocks, num_pages, window, scale, splits, nullptr, stream);
 }
 
 }  // extern "C"

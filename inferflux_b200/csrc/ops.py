@@ -165,7 +165,7 @@ class CudaKernels:
                    "ifx_rmsnorm_pair", "ifx_gate_mul", "ifx_gated_groupnorm", "ifx_pair_combine", "ifx_residual_add_vectors",
                    "ifx_attention_prefill_tcgen05_sink", "ifx_attention_prefill_bf16_sink", "ifx_attention_decode_bf16_sink",
                    "ifx_norm_of_sum", "ifx_row_norm_rope_append", "ifx_rotate_rows", "ifx_gated_scan", "ifx_decay_scan_rate",
-                   "ifx_geglu_mul", "ifx_gemm_skinny_geglu", "ifx_gemm_tcgen05_geglu"):
+                   "ifx_geglu_mul", "ifx_gemm_skinny_geglu", "ifx_gemm_tcgen05_geglu", "ifx_relu2", "ifx_silu_columns"):
             getattr(self.lib, fn).restype = ctypes.c_int
         self.lib.ifx_delta_rule_scratch_floats.restype = ctypes.c_longlong
         self.lib.ifx_sample_scratch_bytes.restype = ctypes.c_longlong
@@ -453,6 +453,40 @@ class CudaKernels:
             self.launches += 1
             return out
         return self.xielu(self.linear(a, w, allow_partial=True), a_pos, a_neg)
+
+    def linear_relu2(self, a, w):
+        """max(a . w^T, 0)^2: the activation on the product's result inside the weight-streaming kernel (few bfloat16 rows, a
+        product wide enough without K slices) or the tcgen05 tiles (many), else by the kernel that adds the slices."""
+        T, K = a.shape
+        N = w.shape[0]
+        if (T and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and K % 8 == 0 and a.is_contiguous() and w.is_contiguous()
+                and w.shape[1] == K and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
+            out = None
+            if T <= self.SKINNY_MAX_ROWS and -(-N // 128) >= 74:
+                out = torch.empty((T, N), dtype=torch.bfloat16, device=a.device)
+                _check(self.lib.ifx_gemm_skinny_act(_ptr(a), _ptr(w), _ptr(None), _ptr(out), T, N, K, N, 0, _ptr(None), 0,
+                                                    ctypes.c_float(0.0), 3, ctypes.c_float(0.0), ctypes.c_float(0.0),
+                                                    _ptr(self.error_flag), _stream()), "gemm_skinny (relu2)")
+            elif T > self.SKINNY_MAX_ROWS and self.swiglu_tiles and K <= self.SWIGLU_TILES_MAX_K:
+                out = torch.empty((T, N), dtype=torch.bfloat16, device=a.device)
+                _check(self.lib.ifx_gemm_tcgen05(_ptr(a), _ptr(w), _ptr(out), T, N, K, N, 6, 0, _ptr(self.error_flag), _stream()),
+                       "gemm_tcgen05 (relu2)")
+            if out is not None:
+                self.launches += 1
+                return out
+        return self.relu2(self.linear(a, w, allow_partial=True))
+
+    def relu2(self, z):
+        """max(z, 0)^2, element by element, in z's dtype; a PartialSum's slices are added first, in the same pass."""
+        splits, out_dtype = 1, z.dtype
+        if isinstance(z, PartialSum):
+            out_dtype, splits, z = z.dtype, z.splits, z.parts
+        _need(z.is_contiguous(), "relu2: contiguous input")
+        out = torch.empty(tuple(z.shape[-2:]), dtype=out_dtype, device=z.device)
+        _check(self.lib.ifx_relu2(_ptr(z), _ptr(out), ctypes.c_longlong(out.numel()), _DT[z.dtype], _DT[out_dtype], splits,
+                                  _stream()), "relu2")
+        self.launches += 1
+        return out
 
     def check_errors(self):
         """Raise if a kernel reported that one of its bounded waits ran out (reads the device flag)."""
@@ -752,7 +786,8 @@ class CudaKernels:
         self.launches += 1
         return q_out
 
-    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None, turn_back=None):
+    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None, turn_back=None,
+                  keep_first=0, head_gate=None):
         """Every token attends its request's keys up to its own position (or the last
         `window` of them) through the block table.  float32: the per-token kernel
         whose additions depend on the position only.  bfloat16: the tiled kernels,
@@ -760,11 +795,13 @@ class CudaKernels:
         `chunk`: a query at position p sees keys from (p // chunk) * chunk on; `sink`: one more unit in the
         softmax's denominator (True), or exp of a learned number per head (a float32 tensor [nq]); `dv`: the values'
         head size if it is not `d`; `turn_back`: what `row_norm_rope_append` returned for values that were turned, so that
-        every head's output is turned back by the query's position before it is rounded."""
-        if (turn_back is not None or chunk or torch.is_tensor(sink) or sink or (dv is not None and dv != d)
+        every head's output is turned back by the query's position before it is rounded; `keep_first`: the first keys of a
+        sequence that every query sees besides its window or chunk; `head_gate` (float32 [T, nq]): every head's output is
+        multiplied by it before it is rounded."""
+        if (turn_back is not None or keep_first or head_gate is not None or chunk or torch.is_tensor(sink) or sink or (dv is not None and dv != d)
                 or (cache.kv is not None and cache.kv.shape[-1] != d)):      # cache rows longer than a head
             return self._attention_masked(q, nq, nkv, d, d if dv is None else dv, window, chunk, sink, scale, ctx, cache,
-                                          turn_back)
+                                          turn_back, int(keep_first), head_gate)
         T = q.shape[0]
         kv, table = cache.kv, cache.block_table
         _need(kv is not None and table is not None, "attention: the mixer has no key/value cache")
@@ -825,9 +862,10 @@ class CudaKernels:
             splits = 8
         return splits
 
-    def _attention_masked(self, q, nq, nkv, d, dv, window, chunk, sink, scale, ctx, cache, turn_back=None):
-        """Attention with a chunk mask, a sink, values of their own size or turned values: the tiled kernels where they take
-        the sizes, else the per-token kernel."""
+    def _attention_masked(self, q, nq, nkv, d, dv, window, chunk, sink, scale, ctx, cache, turn_back=None, keep_first=0,
+                          head_gate=None):
+        """Attention with a chunk mask, kept first keys, a sink, values of their own size, turned values or gated heads: the
+        tiled kernels where they take the sizes, else the per-token kernel."""
         T = q.shape[0]
         kv, table = cache.kv, cache.block_table
         _need(kv is not None and table is not None, "attention: the mixer has no key/value cache")
@@ -845,6 +883,8 @@ class CudaKernels:
         back, neighbours = (None, 0) if turn_back is None else (turn_back[0], int(bool(turn_back[1])))
         _need(back is None or (back.dtype == torch.float32 and back.is_contiguous() and tuple(back.shape) == (T, dv // 2, 2)),
               "attention: cos and sin of the values' angles are float32 [tokens, dv / 2, 2]")
+        _need(head_gate is None or (head_gate.dtype == torch.float32 and head_gate.is_contiguous()
+                                    and tuple(head_gate.shape) == (T, nq)), "attention: a gate per head is float32 [tokens, heads]")
         if (q.dtype == torch.bfloat16 and d == dv == d_row and nq // nkv <= 16 and self.lib.ifx_attention_mma_supports(d)
                 and os.environ.get("INFERFLUX_B200_MASKED_TILES", "1") != "0"):
             # the tiled kernels: prompt portions on mma.sync tiles, single tokens on the cluster kernel
@@ -854,7 +894,8 @@ class CudaKernels:
                     ctx.extra_len[name] = len(vals)
             num_tiles = ctx.extra_len["attn.prefill_tiles"] // 4
             common = (cache.page_size, table.shape[1], kv.shape[0], win, int(chunk or 0),
-                      int(sink_values is not None or bool(sink)), _ptr(sink_values), ctypes.c_float(scale), _ptr(back), neighbours)
+                      int(sink_values is not None or bool(sink)), _ptr(sink_values), ctypes.c_float(scale), _ptr(back), neighbours,
+                      keep_first, _ptr(head_gate))
             if num_tiles and self.tensor_core_prefill and self.lib.ifx_attention_prefill_tcgen05_supports(d, cache.page_size):
                 _check(self.lib.ifx_attention_prefill_tcgen05_sink(
                     _ptr(q), T, _ptr(kv), _ptr(table), _ptr(ctx.extra["attn.prefill_tiles"]), _ptr(ctx.req_slot), _ptr(out),
@@ -874,6 +915,8 @@ class CudaKernels:
                     max_keys = min(max_keys, win)
                 if chunk:
                     max_keys = min(max_keys, int(chunk))
+                if keep_first:                              # (both ends in whole tiles of 16)
+                    max_keys = min(int(ctx.max_kv_len), max_keys + -(-keep_first // 16) * 16)
                 splits = self.decode_splits(n, nkv, max_keys, int(self.lib.ifx_attention_decode_max_splits(d, cache.page_size)))
                 _check(self.lib.ifx_attention_decode_bf16_sink(
                     _ptr(q), _ptr(kv), _ptr(table), _ptr(ctx.extra["attn.decode_meta"]), _ptr(out), n, nq, nkv, d, *common,
@@ -884,7 +927,8 @@ class CudaKernels:
             _ptr(q), _ptr(kv), _ptr(table), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(ctx.req_slot), _ptr(None),
             _ptr(out), T, nq, nkv, d, dv, d_row, cache.page_size, table.shape[1], kv.shape[0],
             0 if window is None else int(window), int(chunk or 0), int(sink_values is not None or bool(sink)),
-            _ptr(sink_values), ctypes.c_float(scale), _ptr(back), neighbours, _DT[q.dtype], _stream()), "attention (masked)")
+            _ptr(sink_values), ctypes.c_float(scale), _ptr(back), neighbours, keep_first, _ptr(head_gate),
+            _DT[q.dtype], _stream()), "attention (masked)")
         self.launches += 1
         return out
 
@@ -1129,13 +1173,15 @@ class CudaKernels:
             _ptr(None), T, rank, _DT[rows.dtype], _stream()), "latent_norm_append")
         self.launches += 1
 
-    def latent_rope_append(self, rows, col0, rank, rot, w, eps, q, heads, dim, rotary, ctx, cache, vdim=None):
+    def latent_rope_append(self, rows, col0, rank, rot, w, eps, q, heads, dim, rotary, ctx, cache, vdim=None, gate_col=None):
         """The cached row of every token: [columns col0 .. + rank of `rows`, RMS-normed with `w`; the `rot` columns
         behind them, turned by the token's position], written at the token's position.  Returns `q`
         [T, heads (dim + rot)] with every head's last `rot` elements turned the same way (in place), or, where the
         tiled attention kernel takes the sizes (`vdim` given), a `TurnedQueries`: the turned parts then lie in the
-        rows of queries in latent space, [T, heads (rank + rot)], whose other columns `latent_attention` fills."""
+        rows of queries in latent space, [T, heads (rank + rot)], whose other columns `latent_attention` fills.  With
+        `gate_col` returns (that, sigmoid of the `heads` columns of `rows` from gate_col on as float32 [T, heads])."""
         T, ld = rows.shape
+        gate = None if gate_col is None else torch.empty((T, heads), dtype=torch.float32, device=rows.device)
         kv, table = cache.kv, cache.block_table
         _need(kv is not None and table is not None and kv.dtype == rows.dtype and q.dtype == rows.dtype,
               "latent_rope_append: no cache of the run's dtype")
@@ -1158,14 +1204,16 @@ class CudaKernels:
             _ptr(rows), ld, int(col0), _ptr(w), ctypes.c_float(eps), _ptr(q), q.shape[1], _ptr(dst), ld_dst, head_stride, offset,
             _ptr(freq), used, inter, ctypes.c_float(mag), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(ctx.req_slot),
             _ptr(table), table.shape[1], cache.page_size, kv.shape[0], _ptr(kv if write else None), T, rank, rot, heads, dim,
-            _DT[rows.dtype], _stream()), "latent_rope_append")
+            _ptr(gate), int(gate_col or 0), _DT[rows.dtype], _stream()), "latent_rope_append")
         self.launches += 1
-        return result
+        return result if gate_col is None else (result, gate)
 
-    def latent_attention(self, q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache, rot=0):
+    def latent_attention(self, q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache, rot=0,
+                         head_gate=None):
         """Attention over cached latents (see csrc/latent_attention.cu).  `q_rows`: [T, >= heads * (dim + rot)], the
         queries in its first columns, every head's `rot` turned elements behind its `dim` plain ones; cached rows
-        are [latent of `rank`; turned key part of `rot`].  Returns [T, heads * vdim]."""
+        are [latent of `rank`; turned key part of `rot`].  `head_gate` (float32 [T, heads]) multiplies the heads' outputs.
+        Returns [T, heads * vdim]."""
         turned = None
         if isinstance(q_rows, TurnedQueries):
             q_rows, turned = q_rows.rows, q_rows.latent
@@ -1178,19 +1226,23 @@ class CudaKernels:
         _need(kv.shape[4] == rank + rot and ldq >= heads * (dim + rot), "latent_attention: rows do not hold the turned part")
         if turned is not None:
             return self._latent_attention_tiles(q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache,
-                                                rot=rot, ql=turned)
-        if rot:
+                                                rot=rot, ql=turned, head_gate=head_gate)
+        _need(head_gate is None or (head_gate.dtype == torch.float32 and tuple(head_gate.shape) == (T, heads)
+                                    and head_gate.is_contiguous()), "latent_attention: a gate per head is float32 [tokens, heads]")
+        tiled = (self.latent_tiles and not rot and q_rows.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0
+                 and ldq % 8 == 0 and self.lib.ifx_latent_attention_mma_supports(rank))
+        if rot or (head_gate is not None and not tiled):
             out = torch.empty((T, heads * vdim), dtype=q_rows.dtype, device=q_rows.device)
             _check(self.lib.ifx_latent_attention_generic_rot(
                 _ptr(q_rows), ldq, _ptr(w_uk), _ptr(w_uv), _ptr(sinks), _ptr(kv), _ptr(table), _ptr(ctx.positions),
                 _ptr(ctx.token_req), _ptr(ctx.req_slot), _ptr(None), _ptr(out), T, heads, dim, vdim, rank, cache.page_size,
                 table.shape[1], kv.shape[0], 0 if window is None else int(window), ctypes.c_float(scale), int(rot),
-                _DT[q_rows.dtype], _stream()), "latent_attention (turned part)")
+                _ptr(head_gate), _DT[q_rows.dtype], _stream()), "latent_attention (turned part)")
             self.launches += 1
             return out
-        if (self.latent_tiles and q_rows.dtype == torch.bfloat16 and self.lib.ifx_latent_attention_mma_supports(rank)
-                and dim % 8 == 0 and vdim % 8 == 0 and ldq % 8 == 0):
-            return self._latent_attention_tiles(q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache)
+        if tiled:
+            return self._latent_attention_tiles(q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache,
+                                                head_gate=head_gate)
         out = torch.empty((T, heads * vdim), dtype=q_rows.dtype, device=q_rows.device)
         _check(self.lib.ifx_latent_attention_generic(
             _ptr(q_rows), ldq, _ptr(w_uk), _ptr(w_uv), _ptr(sinks), _ptr(kv), _ptr(table), _ptr(ctx.positions),
@@ -1201,7 +1253,7 @@ class CudaKernels:
         return out
 
     def _latent_attention_tiles(self, q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache, rot=0,
-                                ql=None):
+                                ql=None, head_gate=None):
         """bfloat16: queries into latent space (a product per head), the tensor-core kernel over cached latents
         with all heads of a token tile in one block, the value projection per head on the weighted latents.
         With `rot`, `ql` [T, heads (rank + rot)] holds the turned query parts already, behind the columns that the
@@ -1239,7 +1291,7 @@ class CudaKernels:
         _check(self.lib.ifx_latent_attention_mma_rot(
             _ptr(ql), _ptr(kv), _ptr(table), _ptr(items), num_items, int(min(self.LATENT_TILE, ctx.max_span)), _ptr(sinks),
             _ptr(olat), _ptr(ws), T, heads, rank, int(rot), cache.page_size, table.shape[1], kv.shape[0], win,
-            ctypes.c_float(scale), splits, _stream()), "latent_attention (tiles)")
+            ctypes.c_float(scale), splits, _ptr(head_gate), _stream()), "latent_attention (tiles)")
         self.launches += 1 + int(splits > 1)
         return self.linear_heads(olat, w_uv, heads, rank, vdim, w_is_nk=True)               # [T, heads * vdim]
 
@@ -1519,17 +1571,19 @@ class CudaKernels:
         self.launches += 1 + int(scratch is not None)
         return out
 
-    def gated_groupnorm(self, y, gate, w, eps, groups, gate_first, out_dtype):
+    def gated_groupnorm(self, y, gate, w, eps, groups, gate_first, out_dtype, kind="silu"):
         """Rows of y (float32 [T, C]) in `groups` equal parts, each over its own root mean square, times w (of size C, or
         of a part's size and then the same for every part; None: no weight) and silu(gate) (float32 rows, maybe a slice of wider ones):
-        the gate multiplies before the norm (`gate_first`) or behind it."""
+        the gate multiplies before the norm (`gate_first`) or behind it.  `kind` "sigmoid": sigmoid(gate) in its place."""
         T, C = y.shape
         _need(y.dtype == torch.float32 and y.is_contiguous() and tuple(gate.shape) == (T, C) and C % groups == 0
-              and (w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() in (C, C // groups))), "gated_groupnorm: bad operands")
+              and (w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() in (C, C // groups)))
+              and kind in ("silu", "sigmoid"), "gated_groupnorm: bad operands")
         out = torch.empty((T, C), dtype=out_dtype, device=y.device)
         gp, gs = self._rows_f32(gate, "gated_groupnorm gate")
         _check(self.lib.ifx_gated_groupnorm(_ptr(y), gp, gs, _ptr(w), 0 if w is None else int(w.numel()), ctypes.c_float(eps), _ptr(out), T, C,
-                                            int(groups), int(bool(gate_first)), _DT[out_dtype], _stream()), "gated_groupnorm")
+                                            int(groups), int(bool(gate_first)), int(kind == "sigmoid"), _DT[out_dtype], _stream()),
+               "gated_groupnorm")
         self.launches += 1
         return out
 
@@ -1598,16 +1652,19 @@ class CudaKernels:
         return _ptr(rows), _DT[rows.dtype], _ptr(None), 1, rows.shape[-1]
 
     def row_norm_rope_append(self, rows, col0, bias, rotary, turn, temp, nq, nkv, d, dv, ctx, cache, q_norm=None, k_norm=None,
-                             norm_eps=0.0):
+                             norm_eps=0.0, v_from_k=False, gate_col=None):
         """Columns col0 .. of `rows` (a tensor or PartialSum): [nq heads of d | nkv key heads of d | nkv value heads of dv],
         plus `bias`; the query part and the key part RMS-normed as a whole (weights of their full size; None: no norm),
         turned by `rotary`, the queries times `temp` per head; the values turned by `turn` over their whole heads; keys and
-        values to the cache.  Returns (queries [T, nq d] in the cache's dtype, what `attention` takes as `turn_back`)."""
+        values to the cache.  Returns (queries [T, nq d] in the cache's dtype, what `attention` takes as `turn_back`).
+        `v_from_k`: no value columns, the values are the keys with their bias, in front of norm and rotation.  With `gate_col`
+        returns a third: sigmoid of the nq columns from col0 + gate_col on, float32 [T, nq] (no bias)."""
         T = rows.shape[0]
         kv, table = cache.kv, cache.block_table
         _need(kv is not None and table is not None and kv.shape[1] == 2 and kv.shape[2] == nkv and kv.shape[-1] >= max(d, dv),
               "row_norm_rope_append: the cache does not fit the heads")
-        for v, n in ((bias, nq * d + nkv * (d + dv)), (q_norm, nq * d), (k_norm, nkv * d), (temp, nq)):
+        _need(not v_from_k or dv == d, "row_norm_rope_append: values that are the keys have their size")
+        for v, n in ((bias, nq * d + nkv * (d if v_from_k else d + dv)), (q_norm, nq * d), (k_norm, nkv * d), (temp, nq)):
             _need(v is None or (v.dtype == torch.float32 and v.numel() == n and v.is_contiguous()),
                   "row_norm_rope_append: biases, norm weights and factors are float32 of their full size")
         for table_, size in ((rotary, d), (turn, dv)):
@@ -1617,15 +1674,30 @@ class CudaKernels:
         dev = kv.device
         q_out = torch.empty((T, nq * d), dtype=kv.dtype, device=dev)
         back = None if turn is None else torch.empty((T, dv // 2, 2), dtype=torch.float32, device=dev)
+        gate = None if gate_col is None else torch.empty((T, nq), dtype=torch.float32, device=dev)
         _check(self.lib.ifx_row_norm_rope_append(
             src, code, part, splits, _LL(ld), int(col0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), ctypes.c_float(norm_eps),
             _ptr(None if rotary is None else rotary.inv_freq), 0 if rotary is None else int(rotary.rotary_dim),
             int(rotary is not None and rotary.interleaved), _ptr(None if turn is None else turn.inv_freq),
             int(turn is not None and turn.interleaved), _ptr(temp), _ptr(ctx.positions), _ptr(ctx.token_req), _ptr(ctx.req_slot),
             _ptr(table), table.shape[1], cache.page_size, kv.shape[0], _ptr(kv), _ptr(q_out), _ptr(back), T, nq, nkv, d, dv,
-            kv.shape[-1], int(bool(cache.writes)), _DT[kv.dtype], _stream()), "row_norm_rope_append")
+            kv.shape[-1], int(bool(cache.writes)), int(bool(v_from_k)), _ptr(gate), int(gate_col or 0), _DT[kv.dtype], _stream()),
+            "row_norm_rope_append")
         self.launches += 1
-        return q_out, (None if back is None else (back, turn.interleaved))
+        turned = None if back is None else (back, turn.interleaved)
+        return (q_out, turned) if gate_col is None else (q_out, turned, gate)
+
+    def silu_columns(self, rows, acted, ctx):
+        """float32 rows from `rows` (a float32 tensor, changed in place, or a PartialSum): z sigmoid(z) on the first `acted`
+        columns, the others as they are."""
+        T = rows.shape[0]
+        src, code, part, splits, ld = self._row_source(rows)
+        plain = not isinstance(rows, PartialSum)
+        _need(not plain or rows.dtype == torch.float32, "silu_columns: float32 rows")
+        out = rows if plain else torch.empty((T, ld), dtype=torch.float32, device=rows.parts.device)
+        _check(self.lib.ifx_silu_columns(src, part, splits, _LL(ld), 0, _ptr(out), T, int(ld), int(acted), _stream()), "silu_columns")
+        self.launches += 1
+        return out
 
     def rotate_rows(self, rows, col0, width, heads, dk, rotary, k_scale, ctx):
         """float32 [T, width] from columns col0 .. of `rows` (a float32 tensor, which is then changed in place where it has

@@ -4,8 +4,8 @@
 //                         the token before a span's first one is the request's state, which takes the span's last token
 //   rmsnorm_pair          two RMS norms of the same float32 rows (one sum of squares, two weights)
 //   gate_mul              a * sigmoid(g) or a * silu(g)
-//   gated_groupnorm       rows in equal parts, each over its own root mean square, times a weight (or none) and silu(gate), the
-//                         gate in front of the norm or behind it
+//   gated_groupnorm       rows in equal parts, each over its own root mean square, times a weight (or none) and silu(gate),
+//                         or sigmoid(gate), the gate in front of the norm or behind it
 //   pair_combine          c_a a + c_b b, or c_a a / rms(a) * w_a + c_b b / rms(b) * w_b; the result is float32
 //   residual_add_vectors  x += s_a * a + s_b * (b + b2), vectors along the row
 //
@@ -94,11 +94,13 @@ __global__ void gate_mul_kernel(const void* __restrict__ a, const void* __restri
   }
 }
 
+__device__ __forceinline__ float gate_value(float g, int sigmoid) { return (sigmoid ? 1.0f : g) / (1.0f + expf(-g)); }
+
 // One block a row, a warp a part at a time.  y [T, C] float32 contiguous; gate float32 with a row stride.
 __global__ void __launch_bounds__(256) gated_groupnorm_kernel(const float* __restrict__ y, const float* __restrict__ gate,
                                                               long long gate_stride, const float* __restrict__ w, int w_size,
                                                               float eps, void* __restrict__ out, int C, int groups,
-                                                              int gate_first, int out_dtype) {
+                                                              int gate_first, int sigmoid, int out_dtype) {
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   const int part = C / groups;
   const float* yr = y + (size_t)t * C;
@@ -109,8 +111,7 @@ __global__ void __launch_bounds__(256) gated_groupnorm_kernel(const float* __res
       const int c = p * part + e;
       float v = yr[c];
       if (gate_first) {
-        const float gv = gr[c];
-        v *= gv / (1.0f + expf(-gv));
+        v *= gate_value(gr[c], sigmoid);
       }
       ss = fmaf(v, v, ss);
     }
@@ -118,8 +119,7 @@ __global__ void __launch_bounds__(256) gated_groupnorm_kernel(const float* __res
     const float inv = rsqrtf(ss / (float)part + eps);
     for (int e = lane; e < part; e += 32) {
       const int c = p * part + e;
-      const float gv = gr[c];
-      const float sg = gv / (1.0f + expf(-gv));
+      const float sg = gate_value(gr[c], sigmoid);
       float v = yr[c];
       if (gate_first) v *= sg;
       v = v * inv * (w ? w[w_size == C ? c : e] : 1.0f);
@@ -133,7 +133,7 @@ __global__ void __launch_bounds__(256) gated_groupnorm_kernel(const float* __res
 __global__ void __launch_bounds__(512) gated_groupnorm_wide_kernel(const float* __restrict__ y, const float* __restrict__ gate,
                                                                    long long gate_stride, const float* __restrict__ w,
                                                                    int w_size, float eps, void* __restrict__ out, int C,
-                                                                   int groups, int gate_first, int out_dtype) {
+                                                                   int groups, int gate_first, int sigmoid, int out_dtype) {
   __shared__ float scratch[32];
   const int t = blockIdx.x;
   const int part = C / groups;
@@ -145,8 +145,7 @@ __global__ void __launch_bounds__(512) gated_groupnorm_wide_kernel(const float* 
       const int c = p * part + e;
       float v = yr[c];
       if (gate_first) {
-        const float gv = gr[c];
-        v *= gv / (1.0f + expf(-gv));
+        v *= gate_value(gr[c], sigmoid);
       }
       ss = fmaf(v, v, ss);
     }
@@ -154,8 +153,7 @@ __global__ void __launch_bounds__(512) gated_groupnorm_wide_kernel(const float* 
     const float inv = rsqrtf(ss / (float)part + eps);
     for (int e = threadIdx.x; e < part; e += blockDim.x) {
       const int c = p * part + e;
-      const float gv = gr[c];
-      const float sg = gv / (1.0f + expf(-gv));
+      const float sg = gate_value(gr[c], sigmoid);
       float v = yr[c];
       if (gate_first) v *= sg;
       v = v * inv * (w ? w[w_size == C ? c : e] : 1.0f);
@@ -260,7 +258,7 @@ int ifx_gate_mul(const void* a, const void* g, void* out, long long total, int d
 }
 
 int ifx_gated_groupnorm(const float* y, const float* gate, long long gate_stride, const float* w, int w_size, float eps,
-                        void* out, int T, int C, int groups, int gate_first, int out_dtype, cudaStream_t stream) {
+                        void* out, int T, int C, int groups, int gate_first, int sigmoid, int out_dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (C <= 0 || groups <= 0 || C % groups || (w != nullptr && w_size != C && w_size != C / groups) || gate_stride < C) return IFX_E_BADARG;
   if (out_dtype != IFX_DT_F32 && out_dtype != IFX_DT_BF16) return IFX_E_DTYPE;
@@ -268,11 +266,11 @@ int ifx_gated_groupnorm(const float* y, const float* gate, long long gate_stride
   if (groups < 8 && part > 64) {                            // few long parts: a block per row takes them in turn
     const int threads = part >= 2048 ? 512 : (part >= 256 ? 256 : ((part + 31) / 32) * 32);
     gated_groupnorm_wide_kernel<<<T, threads, 0, stream>>>(y, gate, gate_stride, w, w_size, eps, out, C, groups, gate_first,
-                                                           out_dtype);
+                                                           sigmoid, out_dtype);
   } else {
     const int warps = groups >= 8 ? 8 : groups;
     gated_groupnorm_kernel<<<T, warps * 32, 0, stream>>>(y, gate, gate_stride, w, w_size, eps, out, C, groups, gate_first,
-                                                        out_dtype);
+                                                        sigmoid, out_dtype);
   }
   IFX_CHECK_LAUNCH();
   return 0;

@@ -6,6 +6,7 @@
 //                          h  = x in the output's dtype       (out given, w_next null: the next sublayer reads x itself)
 //                          y may arrive as the float32 partial sums [splits, rows, hidden] of a K-split product
 //   concat_cast            out[t] = [a[t]; b[t]] in the run's dtype, a and b float32
+//   relu2                  z -> max(z, 0)^2
 //   xielu                  z -> a_pos z^2 + z/2 (z > 0), a_neg (e^z - 1 - z) + z/2 (z <= 0)
 //   softcap                v -> cap tanh(v / cap), float32 in place
 //
@@ -233,14 +234,22 @@ __device__ __forceinline__ float xielu_f(float z, float a_pos, float a_neg) {
   return z > 0.0f ? fmaf(a_pos * z, z, 0.5f * z) : fmaf(a_neg, expm1f(z) - z, 0.5f * z);
 }
 
+enum { ELEM_XIELU = 0, ELEM_RELU2 = 1 };
+
+template <int ACT>
+__device__ __forceinline__ float element_act(float z, float a_pos, float a_neg) {
+  if (ACT == ELEM_RELU2) return fmaxf(z, 0.0f) * fmaxf(z, 0.0f);
+  return xielu_f(z, a_pos, a_neg);
+}
+
 // splits > 1: z is float32 [splits, n], the partial sums of a K-split product, added in split order first.
-template <typename TI, typename TO>
-__global__ void xielu_kernel(const TI* __restrict__ z, TO* __restrict__ out, long long n, float a_pos, float a_neg,
+template <typename TI, typename TO, int ACT>
+__global__ void element_act_kernel(const TI* __restrict__ z, TO* __restrict__ out, long long n, float a_pos, float a_neg,
                              int splits) {
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     float v = to_f32(z[i]);
     for (int s = 1; s < splits; ++s) v += to_f32(z[(long long)s * n + i]);
-    out[i] = from_f32<TO>(xielu_f(v, a_pos, a_neg));
+    out[i] = from_f32<TO>(element_act<ACT>(v, a_pos, a_neg));
   }
 }
 
@@ -251,7 +260,8 @@ __device__ __forceinline__ float xielu_fast(float z, float a_pos, float a_neg) {
 }
 
 // The same, eight bfloat16 (16 bytes) per thread and step, for element counts that are multiples of 8.
-__global__ void xielu_bf16x8_kernel(const __nv_bfloat16* __restrict__ z, __nv_bfloat16* __restrict__ out, long long n8,
+template <int ACT>
+__global__ void element_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ z, __nv_bfloat16* __restrict__ out, long long n8,
                                     float a_pos, float a_neg) {
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n8; i += (long long)gridDim.x * blockDim.x) {
     uint4 raw = reinterpret_cast<const uint4*>(z)[i];
@@ -259,7 +269,8 @@ __global__ void xielu_bf16x8_kernel(const __nv_bfloat16* __restrict__ z, __nv_bf
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       const float2 f = __bfloat1622float2(h2[k]);
-      h2[k] = __floats2bfloat162_rn(xielu_fast(f.x, a_pos, a_neg), xielu_fast(f.y, a_pos, a_neg));
+      if (ACT == ELEM_XIELU) h2[k] = __floats2bfloat162_rn(xielu_fast(f.x, a_pos, a_neg), xielu_fast(f.y, a_pos, a_neg));
+      else h2[k] = __floats2bfloat162_rn(element_act<ACT>(f.x, a_pos, a_neg), element_act<ACT>(f.y, a_pos, a_neg));
     }
     reinterpret_cast<uint4*>(out)[i] = raw;
   }
@@ -273,6 +284,27 @@ __global__ void softcap_kernel(float* __restrict__ v, long long n, float cap) {
 inline unsigned grid_for(long long n, int threads) {
   long long b = (n + threads - 1) / threads;
   return (unsigned)(b < 1 ? 1 : (b > 148 * 16 ? 148 * 16 : b));
+}
+
+template <int ACT>
+static int launch_element_act(const void* z, void* out, long long n, float a_pos, float a_neg, int in_dtype, int out_dtype,
+                              int splits, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (splits < 1 || (splits > 1 && in_dtype != IFX_DT_F32)) return IFX_E_BADARG;
+  const __nv_bfloat16* zb = (const __nv_bfloat16*)z;
+  __nv_bfloat16* ob = (__nv_bfloat16*)out;
+  if (in_dtype == IFX_DT_F32 && out_dtype == IFX_DT_F32)
+    element_act_kernel<float, float, ACT><<<grid_for(n, 256), 256, 0, stream>>>((const float*)z, (float*)out, n, a_pos, a_neg, splits);
+  else if (in_dtype == IFX_DT_BF16 && out_dtype == IFX_DT_BF16 && n % 8 == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)out % 16 == 0)
+    element_act_bf16x8_kernel<ACT><<<grid_for(n / 8, 256), 256, 0, stream>>>(zb, ob, n / 8, a_pos, a_neg);
+  else if (in_dtype == IFX_DT_BF16 && out_dtype == IFX_DT_BF16)
+    element_act_kernel<__nv_bfloat16, __nv_bfloat16, ACT><<<grid_for(n, 256), 256, 0, stream>>>(zb, ob, n, a_pos, a_neg, splits);
+  else if (in_dtype == IFX_DT_F32 && out_dtype == IFX_DT_BF16)
+    element_act_kernel<float, __nv_bfloat16, ACT><<<grid_for(n, 256), 256, 0, stream>>>((const float*)z, ob, n, a_pos, a_neg, splits);
+  else
+    return IFX_E_DTYPE;
+  IFX_CHECK_LAUNCH();
+  return 0;
 }
 
 }  // namespace ifx
@@ -345,23 +377,11 @@ int ifx_concat_cast(const float* a, const float* b, void* out, int T, int hidden
 
 int ifx_xielu(const void* z, void* out, long long n, float a_pos, float a_neg, int in_dtype, int out_dtype, int splits,
               cudaStream_t stream) {
-  if (n <= 0) return 0;
-  if (splits < 1 || (splits > 1 && in_dtype != IFX_DT_F32)) return IFX_E_BADARG;
-  if (in_dtype == IFX_DT_F32 && out_dtype == IFX_DT_F32)
-    xielu_kernel<float, float><<<grid_for(n, 256), 256, 0, stream>>>((const float*)z, (float*)out, n, a_pos, a_neg, splits);
-  else if (in_dtype == IFX_DT_BF16 && out_dtype == IFX_DT_BF16 && n % 8 == 0 && (uintptr_t)z % 16 == 0 &&
-           (uintptr_t)out % 16 == 0)
-    xielu_bf16x8_kernel<<<grid_for(n / 8, 256), 256, 0, stream>>>((const __nv_bfloat16*)z, (__nv_bfloat16*)out, n / 8,
-                                                                  a_pos, a_neg);
-  else if (in_dtype == IFX_DT_BF16 && out_dtype == IFX_DT_BF16)
-    xielu_kernel<__nv_bfloat16, __nv_bfloat16><<<grid_for(n, 256), 256, 0, stream>>>(
-        (const __nv_bfloat16*)z, (__nv_bfloat16*)out, n, a_pos, a_neg, splits);
-  else if (in_dtype == IFX_DT_F32 && out_dtype == IFX_DT_BF16)
-    xielu_kernel<float, __nv_bfloat16><<<grid_for(n, 256), 256, 0, stream>>>((const float*)z, (__nv_bfloat16*)out, n,
-                                                                             a_pos, a_neg, splits);
-  else return IFX_E_DTYPE;
-  IFX_CHECK_LAUNCH();
-  return 0;
+  return launch_element_act<ELEM_XIELU>(z, out, n, a_pos, a_neg, in_dtype, out_dtype, splits, stream);
+}
+
+int ifx_relu2(const void* z, void* out, long long n, int in_dtype, int out_dtype, int splits, cudaStream_t stream) {
+  return launch_element_act<ELEM_RELU2>(z, out, n, 0.0f, 0.0f, in_dtype, out_dtype, splits, stream);
 }
 
 int ifx_softcap(float* v, long long n, float cap, cudaStream_t stream) {

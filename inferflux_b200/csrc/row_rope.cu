@@ -4,12 +4,15 @@
 //                            queries: n_q(all of them together) * weight, turned, times a factor per head -> q_out
 //                            keys:    n_k(all of them together) * weight, turned                          -> cache
 //                            values:  turned by their own position over the whole head (optional)       -> cache
+//                          With v_from_k there are no value columns: the values are the keys as projected (with their bias,
+//                          in front of norm and rotation).  With gate_out: sigmoid of nq more columns, in float32.
 //                          and the cosines and sines of the values' angles, for whoever turns a sum of values back.
 //                          One block, or a cluster of blocks that share the heads, per token.
 //   rotate_rows            rows [heads of d | heads of d | rest] -> float32: both groups of heads turned, the second one
 //                          scaled behind it, the rest as it is.
+//   silu_columns           rows -> float32, z / (1 + e^-z) on the first columns, the rest as it is.
 //
-// Both read plain rows (wider ones than needed, from a column on) or the float32 partial sums of a K-split product.
+// All read plain rows (wider ones than needed, from a column on) or the float32 partial sums of a K-split product.
 // Angles are position * frequency in float32 with precise sines; norms, rotations and factors are float32.
 #include <cooperative_groups.h>
 
@@ -48,6 +51,10 @@ struct RowSource {
     }
     return s;
   }
+  __device__ __forceinline__ float load_one(size_t token, int c) const {
+    if (partial == nullptr && is_bf16) return __bfloat162float(static_cast<const __nv_bfloat16*>(rows)[token * ld + col0 + c]);
+    return partial == nullptr ? load1<false>(token, c) : load1<true>(token, c);
+  }
   // float32 only; SLICED false (plain rows): a caller's loads are one straight run without a branch between them
   template <bool SLICED>
   __device__ __forceinline__ float load1(size_t token, int c) const {
@@ -77,6 +84,17 @@ struct RowRopeArgs {
   int max_blocks, page_size, num_pages;
   void* kv_pool; void* q_out; float2* turn_out;
   int nq, nkv, d, dv, d_row, write_cache;
+  int v_from_k;                                // value head g is read from key head g's columns
+  float* gate_out; int gate_col;               // [tokens, nq] = sigmoid of the columns from gate_col on; null: no gate
+
+  __device__ __forceinline__ int column(int u) const {        // the first column of unit u: queries, keys, values
+    if (u < nq + nkv) return u * d;
+    return v_from_k ? (u - nkv) * d : (nq + nkv) * d + (u - nq - nkv) * dv;
+  }
+  __device__ __forceinline__ void store_gate(int t) const {   // by all threads of a block
+    if (gate_out == nullptr) return;
+    for (int h = threadIdx.x; h < nq; h += blockDim.x) gate_out[(size_t)t * nq + h] = 1.0f / (1.0f + expf(-src.load_one(t, gate_col + h)));
+  }
 };
 
 // element indices of pair j among a head's `size` elements of which `rot` turn
@@ -116,13 +134,14 @@ __global__ void __launch_bounds__(1024) row_norm_rope_append_kernel(const RowRop
   if (z == 0 && a.turn_out)
     for (int j = threadIdx.x; j < half_rot + half_v; j += blockDim.x)
       if (j >= half_rot) a.turn_out[(size_t)t * half_v + (j - half_rot)] = cs[j];      // this thread's own
+  if (z == C - 1) a.store_gate(t);
 
   // ---- the rows, with their biases, and the sums of squares of all queries and of all keys
   float ss_q = 0.0f, ss_k = 0.0f;
   for (int u = z + warp * C, l = warp; u < units; u += nwarps * C, l += nwarps) {
     const bool is_v = u >= a.nq + a.nkv;
     const int size = is_v ? a.dv : a.d;
-    const int col = is_v ? (a.nq + a.nkv) * a.d + (u - a.nq - a.nkv) * a.dv : u * a.d;
+    const int col = a.column(u);
     float ss = 0.0f;
     for (int e = 2 * lane; e < size; e += 64) {
       float2 v = a.src.load2(t, col + e);
@@ -216,9 +235,10 @@ __global__ void __launch_bounds__(1024) row_norm_rope_append_kernel(const RowRop
   }
 }
 
-// The same work for many tokens in the common case: plain bfloat16 rows, whole heads turned in halves, sizes that are
-// multiples of 4 up to 128.  A lane holds elements (2l, 2l + 1) and their partners half a head away, all of a warp's UPW
-// heads in registers, fetched before anything is waited for.
+// The same work for many tokens in the common case: plain bfloat16 rows, heads turned in halves, sizes and turned parts that
+// are multiples of 4, up to 128.  A lane holds two pairs of every head of its warp: elements (2l, 2l + 1) and their partners
+// half the turned part away, or, behind the turned part, the four elements from 4l on; all UPW heads in registers, fetched
+// before anything is waited for.
 template <int UPW>
 __global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeArgs a) {
   __shared__ __align__(16) float2 cs[128];                                 // [d / 2] then [dv / 2]
@@ -237,16 +257,17 @@ __global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeAr
   for (int k = 0; k < UPW; ++k) {
     const int u = warp + k * nwarps;
     const bool is_v = u >= a.nq + a.nkv;
-    const int half = (is_v ? a.dv : a.d) / 2;
-    const int col = is_v ? (a.nq + a.nkv) * a.d + (u - a.nq - a.nkv) * a.dv : u * a.d;
+    const int half = (is_v ? a.dv : a.d) / 2, turned = is_v ? half_v : half_rot;
+    const int e_lo = 2 * lane < turned ? 2 * lane : 4 * lane, e_hi = 2 * lane < turned ? 2 * lane + turned : 4 * lane + 2;
+    const int col = a.column(u);
     lo_raw[k] = hi_raw[k] = __floats2bfloat162_rn(0.0f, 0.0f);
     lo[k] = hi[k] = make_float2(0.0f, 0.0f);
     if (u < units && 2 * lane < half) {
-      lo_raw[k] = *reinterpret_cast<const __nv_bfloat162*>(row + col + 2 * lane);
-      hi_raw[k] = *reinterpret_cast<const __nv_bfloat162*>(row + col + half + 2 * lane);
+      lo_raw[k] = *reinterpret_cast<const __nv_bfloat162*>(row + col + e_lo);
+      hi_raw[k] = *reinterpret_cast<const __nv_bfloat162*>(row + col + e_hi);
       if (a.bias) {
-        lo[k] = *reinterpret_cast<const float2*>(a.bias + col + 2 * lane);
-        hi[k] = *reinterpret_cast<const float2*>(a.bias + col + half + 2 * lane);
+        lo[k] = *reinterpret_cast<const float2*>(a.bias + col + e_lo);
+        hi[k] = *reinterpret_cast<const float2*>(a.bias + col + e_hi);
       }
     }
   }
@@ -256,6 +277,7 @@ __global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeAr
     cs[j] = make_float2(c, sn);
     if (j >= half_rot && a.turn_out) a.turn_out[(size_t)t * half_v + (j - half_rot)] = make_float2(c, sn);
   }
+  a.store_gate(t);
   float ss_q = 0.0f, ss_k = 0.0f;
 #pragma unroll
   for (int k = 0; k < UPW; ++k) {
@@ -280,7 +302,8 @@ __global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeAr
   for (int k = 0; k < UPW; ++k) {
     const int u = warp + k * nwarps;
     const bool is_q = u < a.nq, is_v = u >= a.nq + a.nkv;
-    const int half = (is_v ? a.dv : a.d) / 2;
+    const int half = (is_v ? a.dv : a.d) / 2, turned = is_v ? half_v : half_rot;
+    const int e_lo = 2 * lane < turned ? 2 * lane : 4 * lane, e_hi = 2 * lane < turned ? 2 * lane + turned : 4 * lane + 2;
     if (u >= units || 2 * lane >= half) continue;
     __nv_bfloat16* dst;
     if (is_q) {
@@ -295,11 +318,11 @@ __global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeAr
     const float* nw = is_q ? a.q_norm : (is_v ? nullptr : a.k_norm);
     if (nw) {
       const float inv = is_q ? inv_q : inv_k;
-      nw += (size_t)(is_q ? u : u - a.nq) * a.d + 2 * lane;
-      const float2 wl = *reinterpret_cast<const float2*>(nw), wh = *reinterpret_cast<const float2*>(nw + half);
+      nw += (size_t)(is_q ? u : u - a.nq) * a.d;
+      const float2 wl = *reinterpret_cast<const float2*>(nw + e_lo), wh = *reinterpret_cast<const float2*>(nw + e_hi);
       x.x *= inv * wl.x; x.y *= inv * wl.y; y.x *= inv * wh.x; y.y *= inv * wh.y;
     }
-    if (!is_v || half_v) {
+    if (2 * lane < turned) {
       const float4 c = *reinterpret_cast<const float4*>(&cs[(is_v ? half_rot : 0) + 2 * lane]);      // cos, sin of two pairs
       const float2 rx = make_float2(x.x * c.x - y.x * c.y, x.y * c.z - y.y * c.w);
       y = make_float2(y.x * c.x + x.x * c.y, y.y * c.z + x.y * c.w);
@@ -314,8 +337,8 @@ __global__ void __launch_bounds__(512) row_norm_rope_rows_kernel(const RowRopeAr
       y.x = isfinite(y.x) ? y.x : 0.0f;
       y.y = isfinite(y.y) ? y.y : 0.0f;
     }
-    *reinterpret_cast<__nv_bfloat162*>(dst + 2 * lane) = __floats2bfloat162_rn(x.x, x.y);
-    *reinterpret_cast<__nv_bfloat162*>(dst + half + 2 * lane) = __floats2bfloat162_rn(y.x, y.y);
+    *reinterpret_cast<__nv_bfloat162*>(dst + e_lo) = __floats2bfloat162_rn(x.x, x.y);
+    *reinterpret_cast<__nv_bfloat162*>(dst + e_hi) = __floats2bfloat162_rn(y.x, y.y);
   }
 }
 
@@ -367,6 +390,28 @@ __global__ void __launch_bounds__(128) rotate_rows_kernel(const RowSource src, c
     for (int c = c0 + lane; c < min(c0 + 128, width); c += 32) o[c] = src.load1<SLICED>(t, c);
 }
 
+// A warp takes 128 columns of one token at a time, four a lane.  `acted` columns get the activation; in place, only they
+// are touched.
+template <bool SLICED>
+__global__ void __launch_bounds__(128) silu_columns_kernel(const RowSource src, float* __restrict__ out, int width, int acted,
+                                                           int in_place) {
+  pdl_launch_dependents();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int stop = in_place ? acted : width;
+  float* o = out + (size_t)t * width;
+  pdl_wait();
+  for (int c0 = (blockIdx.y * 4 + warp) * 128 + lane; c0 - lane < stop; c0 += gridDim.y * 512) {
+    float v[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) v[k] = c0 + 32 * k < stop ? src.load1<SLICED>(t, c0 + 32 * k) : 0.0f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int c = c0 + 32 * k;
+      if (c < stop) o[c] = c < acted ? v[k] / (1.0f + expf(-v[k])) : v[k];
+    }
+  }
+}
+
 static int make_source(RowSource* s, const void* rows, int dtype, const float* partial, int splits, int tokens, long long ld, int col0) {
   if ((rows == nullptr) == (partial == nullptr) || ld <= 0 || col0 < 0) return IFX_E_BADARG;
   if (partial != nullptr && splits < 1) return IFX_E_BADARG;
@@ -383,18 +428,21 @@ extern "C" {
 
 // Rows: `rows` (dtype src_dtype) or `partial` [splits, num_tokens, ld]; columns col0 .. col0 + (nq + nkv) d + nkv dv are read.
 // turn_out: float2 [num_tokens, dv / 2] when v_inv_freq is given.  dtype: of q_out and the cache.
+// v_from_k: columns col0 .. col0 + (nq + nkv) d are read, bias has that size, dv == d.
+// gate_out: null, or float32 [num_tokens, nq]; its columns begin at col0 + gate_col.
 int ifx_row_norm_rope_append(const void* rows, int src_dtype, const float* partial, int splits, long long ld, int col0,
                              const float* bias, const float* q_norm, const float* k_norm, float eps, const float* inv_freq,
                              int rot, int interleaved, const float* v_inv_freq, int v_interleaved, const float* temp,
                              const int* positions, const int* token_req, const int* req_slot, const int* block_table,
                              int max_blocks, int page_size, int num_pages, void* kv_pool, void* q_out, float* turn_out,
-                             int num_tokens, int nq, int nkv, int d, int dv, int d_row, int write_cache, int dtype,
-                             cudaStream_t stream) {
+                             int num_tokens, int nq, int nkv, int d, int dv, int d_row, int write_cache, int v_from_k,
+                             float* gate_out, int gate_col, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv || d <= 0 || d % 2 || dv <= 0 || dv % 2 || rot < 0 || rot > d || rot % 2 || ld % 2 || col0 % 2 ||
       (rot > 0 && inv_freq == nullptr) || q_out == nullptr)
     return IFX_E_BADARG;
-  if (col0 + (long long)(nq + nkv) * d + (long long)nkv * dv > ld) return IFX_E_BADARG;
+  if (col0 + (long long)(nq + nkv) * d + (v_from_k ? 0 : (long long)nkv * dv) > ld || (v_from_k && dv != d)) return IFX_E_BADARG;
+  if (gate_out != nullptr && (gate_col < 0 || (long long)col0 + gate_col + nq > ld)) return IFX_E_BADARG;
   if (write_cache && (page_size <= 0 || max_blocks <= 0 || kv_pool == nullptr || block_table == nullptr || d_row < d || d_row < dv))
     return IFX_E_BADARG;
   if (dtype != IFX_DT_F32 && dtype != IFX_DT_BF16) return IFX_E_DTYPE;
@@ -407,10 +455,10 @@ int ifx_row_norm_rope_append(const void* rows, int src_dtype, const float* parti
   a.v_inv_freq = v_inv_freq; a.v_interleaved = v_interleaved; a.temp = temp; a.positions = positions; a.token_req = token_req;
   a.req_slot = req_slot; a.block_table = block_table; a.max_blocks = max_blocks; a.page_size = page_size; a.num_pages = num_pages;
   a.kv_pool = kv_pool; a.q_out = q_out; a.turn_out = reinterpret_cast<float2*>(turn_out); a.nq = nq; a.nkv = nkv; a.d = d; a.dv = dv;
-  a.d_row = d_row; a.write_cache = write_cache;
+  a.d_row = d_row; a.write_cache = write_cache; a.v_from_k = v_from_k; a.gate_out = gate_out; a.gate_col = gate_col;
   const int units = nq + 2 * nkv, dmax = d > dv ? d : dv;
   auto aligned = [](const void* p, int n) { return reinterpret_cast<uintptr_t>(p) % n == 0; };
-  if (dtype == IFX_DT_BF16 && rows != nullptr && src_dtype == IFX_DT_BF16 && num_tokens > 32 && rot == d && !interleaved &&
+  if (dtype == IFX_DT_BF16 && rows != nullptr && src_dtype == IFX_DT_BF16 && num_tokens > 32 && rot % 4 == 0 && !interleaved &&
       (v_inv_freq == nullptr || !v_interleaved) && d % 4 == 0 && dv % 4 == 0 && dmax <= 128 && units <= 64 && d_row % 2 == 0 &&
       aligned(bias, 8) && aligned(q_norm, 8) && aligned(k_norm, 8) && aligned(q_out, 4) && aligned(kv_pool, 4)) {
     const int per_warp = (units + 15) / 16, warps = (units + per_warp - 1) / per_warp;
@@ -460,6 +508,24 @@ int ifx_rotate_rows(const float* rows, const float* partial, int splits, long lo
   if (blocks > 1024) blocks = 1024;
   return launch_pdl(partial ? rotate_rows_kernel<true> : rotate_rows_kernel<false>, dim3(num_tokens, blocks), dim3(128), 0, stream, 1, src, inv_freq, rot, interleaved,
                     positions, out, width, heads, d, k_scale, in_place);
+}
+
+// float32 rows in (plain or partial sums), float32 [num_tokens, width] out: silu on the first `acted` columns, the others as
+// they are; out may be `rows` itself when ld == width and col0 == 0.
+int ifx_silu_columns(const float* rows, const float* partial, int splits, long long ld, int col0, float* out, int num_tokens,
+                     int width, int acted, cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (width <= 0 || acted < 0 || acted > width || col0 + (long long)width > ld || out == nullptr) return IFX_E_BADARG;
+  const int in_place = rows == out;
+  if (in_place && (ld != width || col0 != 0)) return IFX_E_BADARG;
+  RowSource src;
+  const int rc = make_source(&src, rows, IFX_DT_F32, partial, splits, num_tokens, ld, col0);
+  if (rc) return rc;
+  int blocks = ((in_place ? acted : width) + 511) / 512;
+  if (blocks < 1) blocks = 1;
+  if (blocks > 1024) blocks = 1024;
+  return launch_pdl(partial ? silu_columns_kernel<true> : silu_columns_kernel<false>, dim3(num_tokens, blocks), dim3(128), 0, stream, 1, src,
+                    out, width, acted, in_place);
 }
 
 }  // extern "C"

@@ -40,12 +40,14 @@ class KVCacheSpec:
     `head_dim`; `window` None keeps every key, an integer only the last `window`.
     `planes` 2 stores keys and values; 1 stores one vector per head that serves as
     both (a latent from which keys and values are made).  `chunk`: positions are cut into stretches of that
-    many and no query ever reads a key of an earlier stretch than its own, so those pages can go."""
+    many and no query ever reads a key of an earlier stretch than its own, so those pages can go.  `keep_first`: the
+    first so many positions stay readable whatever window and chunk say."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     planes: int = 2
     chunk: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
