@@ -25,6 +25,10 @@ query rows and of the key rows as a whole, all heads together, in front of the r
 (`qk_norm` with `over: "row"`); a learned factor per head on the scores (`head_temp`, multiplied into the queries); and values
 that are turned by their own position over their whole head (`value_position`), cached so, with each head's output turned
 back by the query's position.  A bias on the output projection (`o_bias`) travels with the unadded output.
+So do values that are the keys as projected, before the rotation (`v_from_k`; there is no value projection, q and k may
+have biases), and a gate of one number per head, sigmoid(W_g h) (`gate` "head"): its rows are stacked behind the projections
+and the attention kernels multiply it into each head's output.  With `keep_first` the first so many tokens of a sequence
+stay visible whatever the window or chunk.
 """
 from __future__ import annotations
 
@@ -49,7 +53,8 @@ class Attention(Mixer):
     "if_present"), invent_bias (with "if_present": whether random-weights mode makes
     the biases up; default True), scale (None for 1/sqrt(head_dim)), v_head_dim (None: head_dim),
     qk_norm (None, or {eps, over: "head" (default) or "row"}), chunk (None or int), sink (bool, or "learned": a tensor [heads]), own_kv (default True),
-    conv_taps (None or int), q_temp (None, or {coef, every}), gate (None or "sigmoid"),
+    conv_taps (None or int), q_temp (None, or {coef, every}), gate (None, "sigmoid": a number per output element, or "head"),
+    v_from_k (bool), keep_first (int, default 0),
     head_temp (bool), value_position (a PartSpec of role `position` that turns whole value heads, or None), o_bias (bool),
     names (tensor names of q, k, v, o, q_bias, k_bias, v_bias, o_bias, q_norm, k_norm, sink, gate, temp, q_conv, k_conv,
     v_conv)."""
@@ -81,9 +86,17 @@ class Attention(Mixer):
         self.o_bias = bool(p.get("o_bias", False))
         vpos = p.get("value_position")
         self.value_position = build_part("position", vpos) if vpos is not None else None
-        self.by_rows = self.row_norm or self.head_temp or self.value_position is not None      # row_norm_rope_append's options
+        self.v_from_k = bool(p.get("v_from_k", False))
+        if self.v_from_k and self.dv != self.d:
+            raise ValueError(f"attention: values that are the keys have size {self.d}, not {self.dv}")
+        self.keep_first = int(p.get("keep_first") or 0)
+        if self.keep_first < 0:
+            raise ValueError(f"attention: keep_first must not be negative, got {self.keep_first}")
+        self.head_gate = p.get("gate") == "head"
+        self.by_rows = (self.row_norm or self.head_temp or self.value_position is not None or self.v_from_k
+                        or self.head_gate)                                             # row_norm_rope_append's options
         self.general = (any(p.get(k) for k in ("qk_norm", "chunk", "sink", "conv_taps", "q_temp", "gate"))
-                        or self.dv != self.d or not p.get("own_kv", True) or self.by_rows or self.o_bias)
+                        or self.dv != self.d or not p.get("own_kv", True) or self.by_rows or self.o_bias or self.keep_first)
         if self.general:                   # the general kernels take any even size up to 256
             for size in (self.d, self.dv):
                 if size <= 0 or size % 2 or size > 256:
@@ -113,16 +126,16 @@ class Attention(Mixer):
         if self.q_temp is not None and self.q_temp[1] < 1:
             raise ValueError(f"attention: q_temp.every must be at least 1, got {self.q_temp[1]}")
         self.gate = p.get("gate") or None
-        if self.gate not in (None, "sigmoid"):
-            raise ValueError(f"attention: unknown gate {self.gate!r} (known: sigmoid)")
+        if self.gate not in (None, "sigmoid", "head"):
+            raise ValueError(f"attention: unknown gate {self.gate!r} (known: sigmoid, head)")
         if self.general and self.qkv_bias == "if_present":
             self.qkv_bias = False
         if self.general and self.qkv_bias and not self.by_rows:
             raise ValueError("attention: biases together with head norms, chunks, a sink or a shared cache are not built")
         if self.by_rows and (not self.own_kv or self.taps is not None or self.q_temp is not None
                              or (self.qk_norm_eps is not None and not self.row_norm)):
-            raise ValueError("attention: a norm over rows, a factor per head or turned values beside a shared cache, a "
-                             "convolution, a query multiplier or a norm per head are not built")
+            raise ValueError("attention: a norm over rows, a factor or a gate per head, turned values or values that are the keys "
+                             "beside a shared cache, a convolution, a query multiplier or a norm per head are not built")
         self.names = dict(self._NAMES)
         self.names.update(p.get("names") or {})
         self.w_qkv = self.b_qkv = self.w_o = self.q_norm_w = self.k_norm_w = None
@@ -133,7 +146,7 @@ class Attention(Mixer):
         """Rows that hold a key or a value, whichever is longer (a multiple of 8 elements); the cache of a layer
         that stores nothing is never asked for (its schedule entry names the storing layer's)."""
         row = self.d if not self.general else -(-max(self.d, self.dv) // 8) * 8
-        return KVCacheSpec(self.nkv, row, self.window, chunk=self.retain_chunk)
+        return KVCacheSpec(self.nkv, row, self.window, chunk=self.retain_chunk, keep_first=self.keep_first)
 
     # The stretch of positions after which the cache may drop pages: the mask's own chunk, unless the
     # configuration says that a reader of this cache looks further back (it then sets this to None).
@@ -150,7 +163,12 @@ class Attention(Mixer):
     def _sizes(self):
         """Rows of the stacked projection: (query rows, key rows, value rows)."""
         kv = self.nkv if self.own_kv else 0
-        return self.nq * self.d, kv * self.d, kv * self.dv
+        return self.nq * self.d, kv * self.d, 0 if self.v_from_k else kv * self.dv
+
+    def _gate_rows(self):
+        """Rows behind them for a gate per head; zeros fill up to a multiple of 8, which keeps rows of results aligned."""
+        rows = sum(self._sizes())
+        return -(-(rows + self.nq) // 8) * 8 - rows if self.head_gate else 0
 
     def param_specs(self):
         n = self.names
@@ -158,10 +176,13 @@ class Attention(Mixer):
         specs = {n["q"]: TensorSpec((q, self.hidden)), n["o"]: TensorSpec((self.hidden, self.nq * self.dv))}
         if self.own_kv:
             specs[n["k"]] = TensorSpec((k, self.hidden))
-            specs[n["v"]] = TensorSpec((v, self.hidden))
+            if v:
+                specs[n["v"]] = TensorSpec((v, self.hidden))
         if self.qkv_bias is not False:
             optional = self.qkv_bias == "if_present"
             for side, size in (("q", q), ("k", k), ("v", v)):
+                if not size:
+                    continue
                 specs[n[side + "_bias"]] = TensorSpec((size,), optional=optional, invent=self.invent_bias)
         if self.qk_norm_eps is not None:
             specs[n["q_norm"]] = TensorSpec((q if self.row_norm else self.d,), init="ones")
@@ -174,7 +195,7 @@ class Attention(Mixer):
         if self.learned_sink:
             specs[n["sink"]] = TensorSpec((self.nq,))
         if self.gate is not None:
-            specs[n["gate"]] = TensorSpec((self.nq * self.dv, self.hidden))
+            specs[n["gate"]] = TensorSpec((self.nq if self.head_gate else self.nq * self.dv, self.hidden))
         if self.taps is not None:
             for side, size in (("q", q), ("k", k), ("v", v)):
                 specs[n[side + "_conv"]] = TensorSpec((size, self.taps))
@@ -182,17 +203,19 @@ class Attention(Mixer):
 
     def projection_rows(self) -> int:
         """Rows of the stacked projection, for a mixer that stacks it with another one's."""
-        return sum(self._sizes())
+        return sum(self._sizes()) + self._gate_rows()
 
     def load(self, tensors, dtype, device, projection=None):
         """`projection`: room for the stacked projection that somebody else owns (see `projection_rows`)."""
         n = self.names
         q, k, v = self._sizes()
         sides = [("q", q)] + ([("k", k), ("v", v)] if self.own_kv else [])
+        sides = [(side, size) for side, size in sides if size]
+        gate_rows = self._gate_rows()
         has_bias = any(n[side + "_bias"] in tensors for side, _ in sides)
         layout = {"w_o": ((self.hidden, self.nq * self.dv), dtype)}
         if projection is None:
-            layout["w_qkv"] = ((q + k + v, self.hidden), dtype)
+            layout["w_qkv"] = ((q + k + v + gate_rows, self.hidden), dtype)
         if has_bias:
             layout["b_qkv"] = ((q + k + v,), torch.float32)               # added in float32
         if self.qk_norm_eps is not None:
@@ -204,7 +227,7 @@ class Attention(Mixer):
             layout["b_o"] = ((self.hidden,), torch.float32)
         if self.learned_sink:
             layout["sink"] = ((self.nq,), torch.float32)
-        if self.gate is not None:
+        if self.gate is not None and not self.head_gate:
             layout["w_gate"] = ((self.nq * self.dv, self.hidden), dtype)
         if self.taps is not None:
             layout["w_conv"] = ((q + k + v, self.taps), torch.float32)
@@ -218,7 +241,7 @@ class Attention(Mixer):
         if self.learned_sink:
             buf["sink"].copy_(tensors[n["sink"]])
             self.sink_values = buf["sink"]
-        if self.gate is not None:
+        if self.gate is not None and not self.head_gate:
             buf["w_gate"].copy_(tensors[n["gate"]])
             self.w_gate = buf["w_gate"]
         if self.taps is not None:                                          # the three convolutions as one over the stacked rows
@@ -238,6 +261,9 @@ class Attention(Mixer):
                 else:
                     buf["b_qkv"][at:at + size].copy_(b)
             at += size
+        if gate_rows:
+            w_qkv[at:at + self.nq].copy_(tensors[n["gate"]])
+            w_qkv[at + self.nq:].zero_()
         buf["w_o"].copy_(tensors[n["o"]])
         self.w_qkv, self.w_o = w_qkv, buf["w_o"]
         self.b_qkv = buf["b_qkv"] if has_bias else None
@@ -276,7 +302,8 @@ class Attention(Mixer):
         q = k.rope_append(qkv, None, rotary, self.nq, self.nkv, self.d, ctx, cache, q_norm=self.q_norm_w,
                           k_norm=self.k_norm_w, norm_eps=self.qk_norm_eps or 0.0, dv=self.dv, own_kv=self.own_kv, **more)
         a = k.attention(q, self.nq, self.nkv, self.d, self.window, self.scale, ctx, cache, chunk=self.chunk,
-                        sink=self.sink_values if self.learned_sink else self.sink, dv=self.dv)   # [T, nq dv]
+                        sink=self.sink_values if self.learned_sink else self.sink, dv=self.dv,
+                        **({"keep_first": self.keep_first} if self.keep_first else {}))          # [T, nq dv]
         if self.gate is not None:
             a = k.gate_mul(a, k.linear(materialized_rows(k, h), self.w_gate), self.gate)
         return self._output(k, a)
@@ -290,11 +317,19 @@ class Attention(Mixer):
         rows, col0 = (k.linear(h, self.w_qkv, allow_partial=True), 0) if projected is None else projected
         rotary = self.position.rotary(ctx.device) if self.position is not None else None
         turn = self.value_position.rotary(ctx.device) if self.value_position is not None else None
-        # the queries, and what turns the values' sum back: (cos, sin) of every token's angles
-        q, back = k.row_norm_rope_append(rows, col0, self.b_qkv, rotary, turn, self.temp, self.nq, self.nkv, self.d, self.dv,
-                                         ctx, cache, q_norm=self.q_norm_w, k_norm=self.k_norm_w, norm_eps=self.qk_norm_eps or 0.0)
+        more = {"v_from_k": True} if self.v_from_k else {}
+        if self.head_gate:
+            more["gate_col"] = sum(self._sizes())
+        # the queries, what turns the values' sum back ((cos, sin) of every token's angles), and the heads' gates
+        q, back, *gate = k.row_norm_rope_append(rows, col0, self.b_qkv, rotary, turn, self.temp, self.nq, self.nkv, self.d, self.dv,
+                                                ctx, cache, q_norm=self.q_norm_w, k_norm=self.k_norm_w,
+                                                norm_eps=self.qk_norm_eps or 0.0, **more)
+        more = {"keep_first": self.keep_first} if self.keep_first else {}
+        if gate:
+            more["head_gate"] = gate[0]
         a = k.attention(q, self.nq, self.nkv, self.d, self.window, self.scale, ctx, cache, chunk=self.chunk,
-                        sink=self.sink_values if self.learned_sink else self.sink, dv=self.dv, turn_back=back)   # [T, nq dv]
-        if self.gate is not None:
+                        sink=self.sink_values if self.learned_sink else self.sink, dv=self.dv, turn_back=back,
+                        **more)                                                                      # [T, nq dv]
+        if self.w_gate is not None:
             a = k.gate_mul(a, k.linear(materialized_rows(k, h), self.w_gate), self.gate)
         return self._output(k, a)

@@ -19,6 +19,9 @@ that all heads share; both are turned by the token's position, and
 
 The cached row is then [c; k_turned] (kv_rank + rot_dim numbers), and a query in latent space
 [Wuk_h^T q_plain; q_turned] meets it in one dot product.
+
+`gate` "head": every head's output is multiplied by sigmoid(W_g x)_h, one number per head; W_g is stacked below the
+down-projections, and the factor is multiplied into the head's weighted sum of latents, in front of Wuv_h.
 """
 from __future__ import annotations
 
@@ -36,11 +39,11 @@ class LatentAttention(Mixer):
     """params: hidden_size, num_heads, qk_dim, v_dim, kv_rank, window (None or int), scale (None for
     1/sqrt(qk_dim)), latent_norm_eps, sink (whether heads have a learned sink), q_rank (None: queries straight
     from the input), rot_dim (default 0) with position (a PartSpec of a position encoding that turns those
-    elements), names (tensor names of q, dkv, dkv_norm, uk, uv, sink, o, dq, dq_norm, uq; default: those words
+    elements), gate (None or "head"), names (tensor names of q, dkv, dkv_norm, uk, uv, sink, o, dq, dq_norm, uq, gate; default: those words
     with `_` as `.`)."""
 
     _NAMES = {"q": "q", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "sink": "sink", "o": "o",
-              "dq": "dq", "dq_norm": "dq.norm", "uq": "uq"}
+              "dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "gate": "g"}
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -71,6 +74,9 @@ class LatentAttention(Mixer):
         self.scale = float(p["scale"]) if p.get("scale") is not None else 1.0 / math.sqrt(self.dk)
         self.eps = float(p.get("latent_norm_eps", 1e-6))
         self.has_sink = bool(p.get("sink", False))
+        if p.get("gate") not in (None, "head"):
+            raise ValueError(f"latent_attention: unknown gate {p['gate']!r} (known: head)")
+        self.head_gate = p.get("gate") == "head"
         self.names = dict(self._NAMES)
         self.names.update(p.get("names") or {})
         self.w_q_dkv = self.w_uk = self.w_uv = self.w_o = self.latent_norm = self.sinks = None
@@ -92,6 +98,8 @@ class LatentAttention(Mixer):
             n["uv"]: TensorSpec((H * self.dv, self.rank)),
             n["o"]: TensorSpec((self.hidden, H * self.dv)),
         })
+        if self.head_gate:
+            specs[n["gate"]] = TensorSpec((H, self.hidden))
         if self.has_sink:
             specs[n["sink"]] = TensorSpec((H,), init="zeros")
         return specs
@@ -99,15 +107,20 @@ class LatentAttention(Mixer):
     def load(self, tensors, dtype, device):
         n, H = self.names, self.heads
         q = H * (self.dk + self.rot) if self.q_rank is None else self.q_rank      # rows in front of the latent's
+        down = q + self.rank + self.rot
+        stacked = -(-(down + H) // 8) * 8 if self.head_gate else down              # zeros fill up: rows of results stay aligned
         layout = {
-            "w_q_dkv": ((q + self.rank + self.rot, self.hidden), dtype), "w_uk": ((H * self.dk, self.rank), dtype),
+            "w_q_dkv": ((stacked, self.hidden), dtype), "w_uk": ((H * self.dk, self.rank), dtype),
             "w_uv": ((H * self.dv, self.rank), dtype), "w_o": ((self.hidden, H * self.dv), dtype),
             "latent_norm": ((self.rank,), torch.float32), "sinks": ((H,), torch.float32)}
         if self.q_rank is not None:
             layout.update({"w_uq": ((H * (self.dk + self.rot), self.q_rank), dtype), "q_norm": ((self.q_rank,), torch.float32)})
         self.buffers = buf = WeightBuffers(device, layout)
         buf["w_q_dkv"][:q].copy_(tensors[n["q"] if self.q_rank is None else n["dq"]])
-        buf["w_q_dkv"][q:].copy_(tensors[n["dkv"]])
+        buf["w_q_dkv"][q:down].copy_(tensors[n["dkv"]])
+        if self.head_gate:
+            buf["w_q_dkv"][down:down + H].copy_(tensors[n["gate"]])
+            buf["w_q_dkv"][down + H:].zero_()
         self.w_uq = self.q_norm = None
         if self.q_rank is not None:
             buf["w_uq"].copy_(tensors[n["uq"]])
@@ -131,7 +144,7 @@ class LatentAttention(Mixer):
     # --------------------------------------------------------------------- forward
     def forward(self, h, ctx, cache):
         k = ctx.kernels
-        if self.q_rank is not None or self.rot:
+        if self.q_rank is not None or self.rot or self.head_gate:
             return self._forward_with_options(h, ctx, cache)
         q_dkv = k.materialize(k.linear(h, self.w_q_dkv, allow_partial=True))   # [T, H dk + rank]
         k.latent_norm_append(q_dkv, self.heads * self.dk, self.rank, self.latent_norm, self.eps, ctx, cache)
@@ -151,8 +164,13 @@ class LatentAttention(Mixer):
             q = down
         rotary = self.position.rotary(ctx.device) if self.position is not None else None
         # norms the latent, turns the shared key part and every query head's last `rot` elements, stores [c; k_turned]
-        q = k.latent_rope_append(down, col0, self.rank, self.rot, self.latent_norm, self.eps, q, H, self.dk, rotary, ctx, cache,
-                                 vdim=self.dv)
+        more = {}
+        if self.head_gate:                                                     # and the heads' gates, from the columns behind
+            q, more["head_gate"] = k.latent_rope_append(down, col0, self.rank, self.rot, self.latent_norm, self.eps, q, H, self.dk,
+                                                        rotary, ctx, cache, vdim=self.dv, gate_col=col0 + self.rank + self.rot)
+        else:
+            q = k.latent_rope_append(down, col0, self.rank, self.rot, self.latent_norm, self.eps, q, H, self.dk, rotary, ctx,
+                                     cache, vdim=self.dv)
         a = k.latent_attention(q, self.w_uk, self.w_uv, self.sinks, H, self.dk, self.dv, self.rank, self.window,
-                               self.scale, ctx, cache, rot=self.rot)            # [T, H dv]
+                               self.scale, ctx, cache, rot=self.rot, **more)    # [T, H dv]
         return k.linear(a, self.w_o, allow_partial=True)

@@ -19,6 +19,11 @@ writes to, S <- diag(w_t) S + k_t v_t^T, and reads with the new S, o_t = S^T q_t
     q = rot(W_q h),  k = rot(W_k h) / sqrt(key_dim),  v = W_v h;  w = decay[head]
     y = W_o ((o / rms(o) per head) * silu(W_g h))
 
+`lightning`: a decay per head that is a constant of the design, activated queries, keys and values, one norm over all heads,
+
+    q = silu(W_q h),  k = silu(W_k h),  v = silu(W_v h);  w = decay[head]
+    y = W_o ((o / rms(o) over all heads) * norm * sigmoid(W_g h))
+
 S (float32) and the convolution's last taps - 1 input rows are the request's state: a slot of fixed size, whatever the
 length, zeroed when a request is admitted.  The projections take h in the run's dtype and hand their results over
 in float32; the decays, the step size, the state, the norms and the gates are float32.
@@ -243,4 +248,66 @@ class Retention(Mixer):
         o = k.decay_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], None, cache.state, ctx, heads=self.heads,
                          groups=self.heads, dk=self.dk, dv=self.dv, decay="constant", rate=self.decay)                # [T, V] float32
         y = k.gated_groupnorm(o, proj[:, 2 * K + V:], None, self.eps, groups=self.heads, gate_first=False, out_dtype=ctx.dtype)
+        return k.linear(y, self.w_o, allow_partial=True)
+
+
+@register_part("mixer", "lightning")
+class Lightning(Mixer):
+    """params: hidden_size, num_heads, key_dim, value_dim, decay (one number a head), norm_eps, names (tensor names of q, k, v,
+    g, norm, o)."""
+
+    _NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "norm": "norm", "o": "o"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = spec.params
+        self.hidden = int(p["hidden_size"])
+        self.heads = int(p["num_heads"])
+        self.dk = int(p["key_dim"])
+        self.dv = int(p["value_dim"])
+        if min(self.hidden, self.heads, self.dk, self.dv) <= 0:
+            raise ValueError("lightning: sizes must be positive")
+        if self.dk > 512:
+            raise ValueError(f"lightning: a key size of {self.dk} is beyond the kernel's 512")
+        self.decay_values = [float(v) for v in p["decay"]]
+        if len(self.decay_values) != self.heads:
+            raise ValueError(f"lightning: {len(self.decay_values)} decays for {self.heads} heads")
+        self.eps = float(p.get("norm_eps", 1e-6))
+        self.names = dict(self._NAMES)
+        self.names.update(p.get("names") or {})
+        self.w_stack = self.w_o = self.norm_w = self.decay = None
+
+    def state_spec(self):
+        """S of every head as [head, value channel, key channel]."""
+        return StateSpec((self.heads * self.dk * self.dv,), torch.float32)
+
+    def param_specs(self):
+        n, K, V, C = self.names, self.heads * self.dk, self.heads * self.dv, self.hidden
+        return {n["q"]: TensorSpec((K, C)), n["k"]: TensorSpec((K, C)), n["v"]: TensorSpec((V, C)), n["g"]: TensorSpec((V, C)),
+                n["norm"]: TensorSpec((V,), init="ones"), n["o"]: TensorSpec((C, V))}
+
+    def load(self, tensors, dtype, device):
+        n, K, V, C = self.names, self.heads * self.dk, self.heads * self.dv, self.hidden
+        self.buffers = buf = WeightBuffers(device, {
+            "stack": ((2 * K + 2 * V, C), dtype), "o": ((C, V), dtype),        # q, k, v, g one below the other: one product
+            "norm": ((V,), torch.float32), "decay": ((self.heads,), torch.float32)})
+        at = 0
+        for s, rows in (("q", K), ("k", K), ("v", V), ("g", V)):
+            buf["stack"][at:at + rows].copy_(tensors[n[s]])
+            at += rows
+        buf["o"].copy_(tensors[n["o"]])
+        buf["norm"].copy_(tensors[n["norm"]])
+        buf["decay"].copy_(torch.tensor(self.decay_values, dtype=torch.float64))
+        self.w_stack, self.w_o, self.norm_w, self.decay = buf["stack"], buf["o"], buf["norm"], buf["decay"]
+
+    def forward(self, h, ctx, cache):
+        k = ctx.kernels
+        f32 = torch.float32
+        K, V = self.heads * self.dk, self.heads * self.dv
+        rows = k.linear(materialized_rows(k, h), self.w_stack, out_dtype=f32, allow_partial=True)
+        proj = k.silu_columns(rows, 2 * K + V, ctx)                                       # [T, q | k | v | g], g as it is
+        o = k.decay_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], None, cache.state, ctx, heads=self.heads,
+                         groups=self.heads, dk=self.dk, dv=self.dv, decay="constant", rate=self.decay)       # [T, V] float32
+        y = k.gated_groupnorm(o, proj[:, 2 * K + V:], self.norm_w, self.eps, groups=1, gate_first=False, out_dtype=ctx.dtype,
+                              kind="sigmoid")
         return k.linear(y, self.w_o, allow_partial=True)

@@ -111,7 +111,8 @@ class ActivationMLP(FeedForward):
     params: hidden_size, intermediate_size, activation, names (tensor names of up, down, act).
 
     activation `xielu`: two learned numbers (p, q) in the tensor `act`;
-    act(z) = softplus(p) z^2 + z/2 for z > 0, (1/2 + softplus(q)) (e^z - 1 - z) + z/2 for z <= 0."""
+    act(z) = softplus(p) z^2 + z/2 for z > 0, (1/2 + softplus(q)) (e^z - 1 - z) + z/2 for z <= 0.
+    activation `relu2`: max(z, 0)^2, no numbers of its own."""
 
     _NAMES = {"up": "up", "down": "down", "act": "act"}
 
@@ -120,8 +121,8 @@ class ActivationMLP(FeedForward):
         self.hidden = int(spec.params["hidden_size"])
         self.inter = int(spec.params["intermediate_size"])
         self.activation = str(spec.params.get("activation", "xielu"))
-        if self.activation != "xielu":
-            raise ValueError(f"up_act_down: unknown activation {self.activation!r} (known: xielu)")
+        if self.activation not in ("xielu", "relu2"):
+            raise ValueError(f"up_act_down: unknown activation {self.activation!r} (known: xielu, relu2)")
         self.names = dict(self._NAMES)
         self.names.update(spec.params.get("names") or {})
         self.w_up = self.w_down = None
@@ -129,8 +130,10 @@ class ActivationMLP(FeedForward):
 
     def param_specs(self):
         n = self.names
-        return {n["up"]: TensorSpec((self.inter, self.hidden)), n["down"]: TensorSpec((self.hidden, self.inter)),
-                n["act"]: TensorSpec((2,), init="zeros")}
+        specs = {n["up"]: TensorSpec((self.inter, self.hidden)), n["down"]: TensorSpec((self.hidden, self.inter))}
+        if self.activation == "xielu":
+            specs[n["act"]] = TensorSpec((2,), init="zeros")
+        return specs
 
     def load(self, tensors, dtype, device):
         n = self.names
@@ -139,10 +142,13 @@ class ActivationMLP(FeedForward):
         buf["w_up"].copy_(tensors[n["up"]])
         buf["w_down"].copy_(tensors[n["down"]])
         self.w_up, self.w_down = buf["w_up"], buf["w_down"]
+        if self.activation == "relu2":
+            return
         p, q = (float(v) for v in tensors[n["act"]].to(torch.float32).cpu().tolist())
         self.a_pos, self.a_neg = _softplus(p), 0.5 + _softplus(q)
 
     def forward(self, h, ctx):
         k = ctx.kernels
-        act = k.linear_xielu(h, self.w_up, self.a_pos, self.a_neg)     # the activation in the product's epilogue where it can be
+        # the activation in the product's epilogue where it can be
+        act = k.linear_relu2(h, self.w_up) if self.activation == "relu2" else k.linear_xielu(h, self.w_up, self.a_pos, self.a_neg)
         return k.linear(act, self.w_down, allow_partial=True)

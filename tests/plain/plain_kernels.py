@@ -168,13 +168,15 @@ class PlainKernels:
         return q.to(qkv.dtype).reshape(T, nq * d).contiguous()
 
     def row_norm_rope_append(self, rows, col0, bias, rotary, turn, temp, nq, nkv, d, dv, ctx, cache, q_norm=None, k_norm=None,
-                             norm_eps=0.0):
+                             norm_eps=0.0, v_from_k=False, gate_col=None):
         """Columns col0 .. of `rows`: [nq heads of d | nkv key heads of d | nkv value heads of dv], plus `bias`; the query part
         and the key part RMS-normed as a whole (weights of their full size; None: no norm), turned by `rotary`, the queries
         times `temp` per head; the values turned by `turn`; keys and values to the cache.  Returns (queries [T, nq d] in the
-        cache's dtype, what turns a sum of values back: None, or (float32 [T, dv/2, 2] of cos and sin, interleaved))."""
+        cache's dtype, what turns a sum of values back: None, or (float32 [T, dv/2, 2] of cos and sin, interleaved)).
+        `v_from_k`: no value columns, the values are the keys in front of norm and rotation.  With `gate_col` a third result:
+        sigmoid of nq columns, float32."""
         A, T = self.acc, rows.shape[0]
-        nQ, nK, nV = nq * d, nkv * d, nkv * dv
+        nQ, nK, nV = nq * d, nkv * d, 0 if v_from_k else nkv * dv
         x = rows[:, col0:col0 + nQ + nK + nV].to(A)
         if bias is not None:
             x = x + bias.to(A)
@@ -186,7 +188,7 @@ class PlainKernels:
         if temp is not None:
             q = q * temp.to(A)[None, :, None]
         k = self._turn(row_norm(x[:, nQ:nQ + nK], k_norm).view(T, nkv, d), rotary, pos)
-        v = self._turn(x[:, nQ + nK:].view(T, nkv, dv), turn, pos)
+        v = self._turn((x[:, nQ:nQ + nK] if v_from_k else x[:, nQ + nK:]).view(T, nkv, dv), turn, pos)
         if cache.writes:
             P = cache.page_size
             slot = ctx.req_slot.long()[ctx.token_req.long()]
@@ -197,7 +199,16 @@ class PlainKernels:
         if turn is not None:
             ang = pos.to(torch.float32)[:, None] * turn.inv_freq[None, :]
             back = (torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1), turn.interleaved)
-        return q.to(cache.kv.dtype).reshape(T, nQ).contiguous(), back
+        q = q.to(cache.kv.dtype).reshape(T, nQ).contiguous()
+        if gate_col is None:
+            return q, back
+        return q, back, torch.sigmoid(rows[:, col0 + gate_col:col0 + gate_col + nq].to(A)).to(torch.float32).contiguous()
+
+    def silu_columns(self, rows, acted, ctx):
+        out = rows.to(torch.float32).clone()
+        z = out[:, :acted].to(self.acc)
+        out[:, :acted] = (z * torch.sigmoid(z)).to(torch.float32)
+        return out
 
     @staticmethod
     def _turn_back(out, turn_back):
@@ -209,14 +220,20 @@ class PlainKernels:
         a, b = u * cos + v * sin, v * cos - u * sin
         return torch.stack([a, b], dim=-1).flatten(-2) if interleaved else torch.cat([a, b], dim=-1)
 
-    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None, turn_back=None):
+    def attention(self, q, nq, nkv, d, window, scale, ctx, cache, chunk=None, sink=False, dv=None, turn_back=None,
+                  keep_first=0, head_gate=None):
         dv = d if dv is None else dv
+        if head_gate is not None:                            # in the accumulation's dtype, rounded once
+            wide = self.attention(q.to(self.acc), nq, nkv, d, window, scale, ctx, cache, chunk=chunk, sink=sink, dv=dv,
+                                  turn_back=turn_back, keep_first=keep_first)
+            return (wide.view(-1, nq, dv) * head_gate.to(self.acc)[:, :, None]).to(q.dtype).reshape(-1, nq * dv)
         if turn_back is not None:                            # in the accumulation's dtype, rounded once
-            wide = self.attention(q.to(self.acc), nq, nkv, d, window, scale, ctx, cache, chunk=chunk, sink=sink, dv=dv)
+            wide = self.attention(q.to(self.acc), nq, nkv, d, window, scale, ctx, cache, chunk=chunk, sink=sink, dv=dv,
+                                  keep_first=keep_first)
             return self._turn_back(wide.view(-1, nq, dv), turn_back).to(q.dtype).reshape(-1, nq * dv)
         T = q.shape[0]
         P = cache.page_size
-        if chunk or torch.is_tensor(sink) or sink or dv != d or cache.kv.shape[-1] != d:
+        if chunk or keep_first or torch.is_tensor(sink) or sink or dv != d or cache.kv.shape[-1] != d:
             out = torch.empty((T, nq, dv), dtype=q.dtype, device=q.device)
             qv = q.view(T, nq, d).to(self.acc)
             pos_all, req_all, slots = ctx.positions.tolist(), ctx.token_req.tolist(), ctx.req_slot.tolist()
@@ -225,7 +242,7 @@ class PlainKernels:
                 first = max(0, pos - window + 1) if window else 0
                 if chunk:
                     first = max(first, pos // chunk * chunk)
-                keys = torch.arange(first, pos + 1, device=q.device)
+                keys = torch.tensor(list(range(min(keep_first, first))) + list(range(first, pos + 1)), device=q.device)
                 pages = cache.block_table[slot, keys // P].long()
                 K = cache.kv[pages, 0, :, keys % P, :d].to(self.acc)
                 V = cache.kv[pages, 1, :, keys % P, :dv].to(self.acc)
@@ -277,6 +294,10 @@ class PlainKernels:
 
     def linear_xielu(self, a, w, a_pos, a_neg):
         return self.xielu(self.linear(a, w), a_pos, a_neg)
+
+    def linear_relu2(self, a, w):
+        z = self.linear(a, w).to(self.acc)
+        return (torch.clamp(z, min=0.0) ** 2).to(a.dtype)
 
     def softcap(self, logits, cap):
         logits.copy_(cap * torch.tanh(logits.to(self.acc) / cap))
@@ -432,13 +453,13 @@ class PlainKernels:
             out = out + skip.to(A)[None, :, None] * va
         return out.reshape(T, heads * dv).to(torch.float32)
 
-    def gated_groupnorm(self, y, gate, w, eps, groups, gate_first, out_dtype):
+    def gated_groupnorm(self, y, gate, w, eps, groups, gate_first, out_dtype, kind="silu"):
         """Rows of y [T, C] in `groups` equal parts, each over its own root mean square, times w (of size C, or of a
         part's size and then the same for every part) and silu(gate): the gate multiplies before the norm
-        (`gate_first`) or behind it."""
+        (`gate_first`) or behind it.  `kind` "sigmoid": sigmoid(gate) in its place."""
         A = self.acc
         ya, ga = y.to(A), gate.to(A)
-        ga = ga * torch.sigmoid(ga)
+        ga = torch.sigmoid(ga) * (1.0 if kind == "sigmoid" else ga)
         if gate_first:
             ya = ya * ga
         T, C = ya.shape
@@ -567,7 +588,8 @@ class PlainKernels:
             page = cache.block_table[slot, pos // P].long()
             cache.kv[page, 0, 0, pos % P, :] = c.to(cache.kv.dtype)
 
-    def latent_rope_append(self, rows, col0, rank, rot, w, eps, q, heads, dim, rotary, ctx, cache, vdim=None):
+    def latent_rope_append(self, rows, col0, rank, rot, w, eps, q, heads, dim, rotary, ctx, cache, vdim=None,
+                           gate_col=None):
         """The cached row of every token: [columns col0 .. + rank of `rows`, RMS-normed with `w`; the `rot` columns
         behind them, turned by the token's position].  Returns `q` [T, heads (dim + rot)] with every head's last `rot`
         elements turned the same way (q itself may be changed)."""
@@ -599,9 +621,17 @@ class PlainKernels:
             cache.kv[page, 0, 0, p % P, :] = torch.cat([c, kt], dim=-1).to(cache.kv.dtype)
         qa = q[:, :heads * (dim + rot)].to(A).reshape(T, heads, dim + rot).clone()
         qa[:, :, dim:] = turn(qa[:, :, dim:])
-        return qa.reshape(T, heads * (dim + rot)).to(q.dtype)
+        result = qa.reshape(T, heads * (dim + rot)).to(q.dtype)
+        if gate_col is None:
+            return result
+        return result, torch.sigmoid(rows[:, gate_col:gate_col + heads].to(A)).to(torch.float32)
 
-    def latent_attention(self, q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache, rot=0):
+    def latent_attention(self, q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache, rot=0,
+                         head_gate=None):
+        if head_gate is not None:                            # in the accumulation's dtype, rounded once
+            wide = self.latent_attention(q_rows.to(self.acc), w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx,
+                                         cache, rot=rot)
+            return (wide.view(-1, heads, vdim) * head_gate.to(self.acc)[:, :, None]).to(q_rows.dtype).reshape(-1, heads * vdim)
         if rot:
             return self._latent_attention_rot(q_rows, w_uk, w_uv, sinks, heads, dim, vdim, rank, window, scale, ctx, cache, rot)
         T, P = q_rows.shape[0], cache.page_size
