@@ -2,7 +2,9 @@
 batching, nothing shared with the package.  Slow on purpose; the tests hold the engine to it.
 
 A model is (raw, W): config.json as a dict and name -> tensor.  Every function computes in the dtype of
-its inputs (the tests use float64).
+its inputs (the tests use float64).  In bfloat16, what the design keeps in 32 bits is float32 here too: the residual
+stream, norms, rotations, scores and softmax, gates, the recurrence; such a run is the yardstick for what rounding the
+rest does.
 
     x = scale * embed[tokens]
     per layer run:  x += n(mixer(n(x)));   x += n(ff(n(x)))   (ff may be absent; every n has a weight 1 + w of its own)
@@ -25,14 +27,20 @@ from .plain_vononex import load_model_dir            # noqa: F401  (reads config
 
 # ------------------------------------------------------------------------------ small pieces
 
+def wide(x):
+    """Float32 for bfloat16, anything else as it is."""
+    return x.to(torch.float32) if x.dtype == torch.bfloat16 else x
+
+
 def unit_rms(x, eps):
     """x divided by its root mean square over the last axis, eps under the root."""
+    x = wide(x)
     return x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps)
 
 
 def norm(x, w, eps):
     """The model's norm: the stored weight is the distance from one."""
-    return unit_rms(x, eps) * (1.0 + w)
+    return unit_rms(x, eps) * (1.0 + wide(w))
 
 
 def silu(z):
@@ -45,7 +53,7 @@ def squared_relu(z):
 
 def gate_heads(o, logits):
     """o: [n, H, dv] heads' outputs, logits: [n, H]."""
-    return o * torch.sigmoid(logits)[:, :, None]
+    return (wide(o) * torch.sigmoid(wide(logits))[:, :, None]).to(logits.dtype)
 
 
 # ------------------------------------------------------------------------------ positions
@@ -58,19 +66,21 @@ def _angles(positions, dims, base, dtype):
 
 def rotate_halves(x, positions, dims, base):
     """x: [n, H, d]; elements i and i + dims/2 of the first `dims` turn by position * base^(-2i/dims)."""
+    dtype, x = x.dtype, wide(x)
     c, s = _angles(positions, dims, base, x.dtype)
     u, v = x[:, :, :dims // 2], x[:, :, dims // 2:dims]
-    return torch.cat([u * c - v * s, v * c + u * s, x[:, :, dims:]], dim=-1)
+    return torch.cat([u * c - v * s, v * c + u * s, x[:, :, dims:]], dim=-1).to(dtype)
 
 
 def rotate_neighbours(x, positions, dims, base):
     """The same for elements 2i and 2i + 1."""
+    dtype, x = x.dtype, wide(x)
     c, s = _angles(positions, dims, base, x.dtype)
     out = x.clone()
     u, v = x[:, :, 0:dims:2], x[:, :, 1:dims:2]
     out[:, :, 0:dims:2] = u * c - v * s
     out[:, :, 1:dims:2] = v * c + u * s
-    return out
+    return out.to(dtype)
 
 
 # ------------------------------------------------------------------------------ masks and softmax
@@ -106,8 +116,9 @@ def attend(q, k, v, scale, seen, sinks):
     out = []
     for h in range(H):
         g = h // (H // G)
-        s = (q[:, h] @ k[:, g].T) * scale
-        out.append(softmax_rows(s, seen, None if sinks is None else sinks[h]) @ v[:, g])
+        s = (wide(q[:, h]) @ wide(k[:, g]).T) * scale
+        w = softmax_rows(s, seen, None if sinks is None else wide(sinks[h]))
+        out.append((w.to(q.dtype) @ v[:, g]))
     return torch.stack(out, dim=1)
 
 
@@ -130,10 +141,10 @@ def latent_attention(h, W, p, m, eps, positions):
     n = h.shape[0]
     H, d, dr, dv, r = int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"])
     base = float(m["rot"]["base"])
-    cq = unit_rms(h @ W[p + "dq"].T, eps) * W[p + "dq.norm"]
+    cq = (unit_rms(h @ W[p + "dq"].T, eps) * wide(W[p + "dq.norm"])).to(h.dtype)
     q = (cq @ W[p + "uq"].T).reshape(n, H, d + dr)
     down = h @ W[p + "dkv"].T
-    c = unit_rms(down[:, :r], eps) * W[p + "dkv.norm"]
+    c = (unit_rms(down[:, :r], eps) * wide(W[p + "dkv.norm"])).to(h.dtype)
     k = (c @ W[p + "uk"].T).reshape(n, H, d)
     v = (c @ W[p + "uv"].T).reshape(n, H, dv)
     kr = rotate_neighbours(down[:, r:].reshape(n, 1, dr), positions, dr, base)
@@ -159,11 +170,11 @@ def decay_scan(q, k, v, decay):
 def lightning(h, W, p, m, eps):
     n = h.shape[0]
     H, d, dv = int(m["heads"]), int(m["dim"]), int(m["vdim"])
-    q, k = (silu(h @ W[p + s].T).reshape(n, H, d) for s in ("q", "k"))
-    v = silu(h @ W[p + "v"].T).reshape(n, H, dv)
-    o = decay_scan(q, k, v, torch.tensor([float(x) for x in m["decay"]], dtype=h.dtype)).reshape(n, H * dv)
-    o = unit_rms(o, eps) * W[p + "norm"]
-    return (o * torch.sigmoid(h @ W[p + "g"].T)) @ W[p + "o"].T
+    q, k = (silu(wide(h @ W[p + s].T)).reshape(n, H, d) for s in ("q", "k"))
+    v = silu(wide(h @ W[p + "v"].T)).reshape(n, H, dv)
+    o = decay_scan(q, k, v, torch.tensor([float(x) for x in m["decay"]], dtype=q.dtype)).reshape(n, H * dv)
+    o = unit_rms(o, eps) * wide(W[p + "norm"])
+    return (o * torch.sigmoid(wide(h @ W[p + "g"].T))).to(h.dtype) @ W[p + "o"].T
 
 
 # ------------------------------------------------------------------------------ the layer
@@ -190,14 +201,14 @@ def forward(raw, W, tokens, dtype=torch.float64, streams=None):
     W = {k: (v.to(dtype) if v.is_floating_point() else v) for k, v in W.items()}
     eps = float(raw["norm"]["eps"])
     positions = list(range(len(tokens)))
-    x = W["embed"][list(tokens)] * float(raw["embedding"]["scale"])
+    x = wide(W["embed"][list(tokens)]) * float(raw["embedding"]["scale"])
     for i, layer in enumerate(raw["layers"]):
         p = f"l{i if layer.get('weights_of') is None else layer['weights_of']}."
-        y = mixer(norm(x, W[p + "norm1"], eps), W, p + "mix.", layer, eps, positions)
+        y = mixer(norm(x, W[p + "norm1"], eps).to(dtype), W, p + "mix.", layer, eps, positions)
         x = x + norm(y, W[p + "norm1b"], eps)
         if layer.get("mlp") is not None:
-            y = feed_forward(norm(x, W[p + "norm2"], eps), W, p + "mlp.")
+            y = feed_forward(norm(x, W[p + "norm2"], eps).to(dtype), W, p + "mlp.")
             x = x + norm(y, W[p + "norm2b"], eps)
         if streams is not None:
             streams.append(x.clone())
-    return float(raw["logit_scale"]) * (norm(x, W["final.norm"], eps) @ W["head"].T)
+    return float(raw["logit_scale"]) * wide(norm(x, W["final.norm"], eps).to(dtype) @ W["head"].T)
