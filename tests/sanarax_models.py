@@ -49,11 +49,11 @@ def configs():
     a = [_attention(4, 2, 16, 0.3, 500.0, 8, 24, 5, _dense(88)), _latent(3, 12, 4, 10, 20, 24, 0.25, 300.0, _dense(40)),
          _lightning([0.9, 0.999, 0.5], 12, 20, None)]
     a += [_again(a, 0), _attention(2, 2, 24, 0.21, 40.0, 24, 7, 0, None), _again(a, 2), _again(a, 1)]
-    b = [_lightning([0.97, 0.75], 24, 6, _dense(64)), _attention(6, 1, 8, 0.5, 2000.0, 4, 1, 33, _dense(200)),
+    b = [_lightning([0.97], 24, 26, _dense(64)), _attention(6, 1, 8, 0.5, 2000.0, 4, 1, 33, _dense(200)),
          _latent(1, 16, 16, 8, 32, 16, 0.3, 50.0, None), _lightning([0.999, 0.3, 1.0, 0.6, 0.9], 8, 8, _dense(24))]
     b += [_again(b, 1), _again(b, 3)]
     c = [_latent(2, 7, 6, 5, 9, 11, 0.4, 90.0, _dense(33)), _attention(3, 3, 10, 0.45, 25.0, 2, 16, 16, None)]
-    c += [_again(c, 0), _attention(5, 1, 14, 0.27, 700.0, 10, 90, 3, _dense(75)), _lightning([0.98], 5, 3, _dense(21))]
+    c += [_again(c, 0), _attention(5, 1, 14, 0.27, 700.0, 10, 90, 3, _dense(75)), _lightning([0.98, 0.6, 0.995], 11, 9, _dense(21))]
     return {"A": (_config(310, 72, 1e-6, 3.0, 0.7, a), 8), "B": (_config(259, 96, 2e-4, 1.0, 1.0, b), 4),
             "C": (_config(151, 50, 1e-5, 0.6, 2.5, c), 16)}
 
