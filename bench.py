@@ -1509,6 +1509,243 @@ def run_design_vononex(args, pk):
     return 0
 
 
+def sanarax_config(shape, layers=0):
+    """Sanarax at the sizes of the other designs, its three layer kinds taking turns: attention (the Qwen2 shape's heads of 128
+    over its key/value heads, half of every head rotated, a window of 2,048 beside 64 kept first tokens), latent attention
+    (heads of 128 + 64 rotated, a latent of 256, queries through a latent of 1,536) and lightning attention (heads of
+    128 x 128); every layer with a squared-ReLU feed-forward that has as many parameters as the Qwen2 shape's gated one."""
+    from inferflux_b200.config import SanaraxConfig
+    s = DESIGN_SHAPES[shape]
+    q = qwen7b_config(s["qwen"])
+    w, n = s["width"], layers or q.num_hidden_layers
+    mlp = {"kind": "dense", "ff": q.intermediate_size * 3 // 2}
+    heads = w // 128
+    kinds = [
+        {"type": "attention", "mlp": mlp, "mixer": {
+            "heads": s["heads"], "kv_heads": q.num_key_value_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "rot": {"base": 500000.0, "dims": 64}, "mask": {"size": 2048, "keep_first": 64}}},
+        {"type": "latent_attention", "mlp": mlp, "mixer": {
+            "heads": s["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 256, "q_rank": 1536, "scale": 192 ** -0.5,
+            "rot": {"base": 10000.0, "dims": 64}}},
+        {"type": "lightning", "mlp": mlp, "mixer": {
+            "heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5.0 - 5.0 * h / heads) for h in range(heads)]}}]
+    return SanaraxConfig.from_dict({"architecture": "Sanarax", "vocab": s["vocab"], "width": w, "norm": {"eps": 1e-6},
+                                    "embedding": {"scale": 8.0}, "logit_scale": 0.5, "layers": [kinds[i % 3] for i in range(n)]})
+
+
+def sanarax_costs(cfg, batch, context, tokens):
+    """(bytes a decode step must read or write, FLOPs of a prefill of `tokens`): matrices, recurrent state in and out, cached
+    rows that a token sees."""
+    w, step_bytes, flops = cfg.width, 0, 0
+    for layer in cfg.layers:
+        m = layer["mixer"]
+        params = 2 * w * layer["mlp"]["ff"] if layer["mlp"] else 0
+        if layer["type"] == "attention":
+            qd, kd = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+            size, keep = m["mask"]["size"], m["mask"]["keep_first"]
+            seen = lambda n: min(n, size + keep)
+            params += w * (2 * qd + kd + m["heads"])
+            step_bytes += batch * seen(context) * 2 * kd * 2
+            flops += 4 * qd * sum(seen(n) for n in range(1, tokens + 1))
+        elif layer["type"] == "latent_attention":
+            H, dq, row = m["heads"], m["dim"] + m["rot_dim"], m["kv_rank"] + m["rot_dim"]
+            params += w * (m["q_rank"] + row + H) + m["q_rank"] * H * dq + H * (m["dim"] + m["vdim"]) * m["kv_rank"] + H * m["vdim"] * w
+            step_bytes += batch * context * row * 2
+            flops += 2 * H * (2 * m["kv_rank"] + m["rot_dim"]) * (tokens * (tokens + 1) // 2)
+        else:
+            state = m["heads"] * m["dim"] * m["vdim"]
+            params += w * m["heads"] * (2 * m["dim"] + 3 * m["vdim"])
+            step_bytes += 2 * batch * state * 4
+            flops += 4 * tokens * state
+        step_bytes += 2 * params
+        flops += 2 * tokens * params
+    return step_bytes + 2 * cfg.vocab * w, flops + 2 * cfg.vocab * w
+
+
+def sanarax_kernels(kernels, scfg, pk, batch, context, tokens):
+    """The new design's kernels beside the like kernels of the closest models, each alone at the layer's sizes: attention with
+    kept first tokens and gates beside a plain window with a sink and plain attention, its rows beside bias and rotation, gated
+    latent attention beside Benarax's, activated columns beside rotated ones, the scan, the norm over all heads beside the
+    norm per head, the sum with both norms, the squared-ReLU product beside the SiLU-gated one and xIELU's."""
+    import torch
+    from inferflux_b200.cache import CacheManager
+    from inferflux_b200.config import ScheduleEntry
+    from inferflux_b200.csrc.ops import PartialSum
+    from inferflux_b200.engine.batch import StepContext, StepEntry
+    from inferflux_b200.parts import KVCacheSpec
+    from inferflux_b200.parts.base import RotaryTable
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    at, lat, lig = (next(l for l in scfg.layers if l["type"] == k)["mixer"] for k in ("attention", "latent_attention", "lightning"))
+    w, ff = scfg.width, scfg.layers[0]["mlp"]["ff"]
+    page, out = 16, {}
+
+    def row(name, fn, bytes_=0, flops=0):
+        ms = _event_times(fn)
+        roof = max(bytes_ / hbm, flops / tf)
+        out[name] = {"us": round(ms * 1000, 1), "roofline_us": round(roof * 1e6, 1), "frac": round(roof / (ms * 1e-3), 3),
+                     "bound": "hbm" if bytes_ / hbm >= flops / tf else "tensor"}
+
+    class _Sections:                                       # asks the kernel table for both attentions' work lists
+        def step_sections(self, ctx):
+            return {**ctx.kernels.attention_sections(ctx), **ctx.kernels.latent_attention_sections(ctx)}
+
+    def ctx_for(cache, spans):
+        entries, starts, slots = [], [], []
+        for rid, n in spans:
+            if rid not in cache:
+                cache.add_request(rid)
+            start = cache.length(rid)
+            cache.reserve(rid, start + n)
+            entries.append(StepEntry(rid, [0] * n, []))
+            starts.append(start)
+            slots.append(cache.slot(rid))
+        ctx = StepContext.build(kernels, bf, dev, entries, starts, slots, cache.drain_table_updates(), providers=[_Sections()])
+        for g, (idx, pg) in zip(cache.groups, ctx.table_updates):
+            kernels.scatter_i32(g.table, idx, pg)
+        for (rid, n), start in zip(spans, starts):
+            cache.commit(rid, start + n)
+        return ctx
+
+    nq, nkv, d = at["heads"], at["kv_heads"], at["dim"]
+    size_, keep = at["mask"]["size"], at["mask"]["keep_first"]
+    rdims = at["rot"]["dims"]
+    rot = RotaryTable(torch.tensor([at["rot"]["base"] ** (-2.0 * i / rdims) for i in range(rdims // 2)], device=dev), rdims, False)
+    sinks = torch.zeros(nq, device=dev)
+    AH, ldk, lrot, ldv, rank = lat["heads"], lat["dim"], lat["rot_dim"], lat["vdim"], lat["kv_rank"]
+    ltable = RotaryTable(torch.rand(lrot // 2, device=dev), lrot, True, 1.0)
+    for what, spans_a, spans_b in (("decode", [(f"r{i}", context - 1) for i in range(batch)], [(f"r{i}", 1) for i in range(batch)]),
+                                   ("prefill", [], [("p", tokens)])):
+        T, R = sum(n for _r, n in spans_b), len(spans_b)
+        tag = f"{T} rows" if what == "decode" else f"{T} rows "
+        pages = (batch * context if what == "decode" else tokens) // page + 2 * batch + 2
+        cached = batch * context if what == "decode" else tokens
+        cache = CacheManager([(KVCacheSpec(nkv, d, size_, keep_first=keep), None), (KVCacheSpec(1, rank + lrot, None, planes=1), None)],
+                             page_size=page, num_pages=pages, max_seqs=batch, max_seq_len=max(context, tokens) + 16, dtype=bf, device=dev)
+        for g in cache.groups:
+            g.pool.normal_()
+        if spans_a:
+            ctx_for(cache, spans_a)
+        ctx = ctx_for(cache, spans_b)
+        view, lview = cache.view(ScheduleEntry(0, 0)), cache.view(ScheduleEntry(1, 1))
+        splits = 8 if what == "decode" else 0
+        mk = lambda n, dt=bf: PartialSum(torch.randn(splits, T, n, device=dev), dt) if splits else torch.randn(T, n, device=dev).to(dt)
+        size = lambda n, dt=bf: T * n * (4 * splits if splits else (2 if dt == bf else 4))
+        # rows in front of attention
+        used = (nq + nkv) * d
+        width = -(-(used + nq) // 8) * 8
+        qk, qkv, bias = mk(width), mk((nq + 2 * nkv) * d), torch.randn((nq + 2 * nkv) * d, device=dev)
+        run = lambda: kernels.row_norm_rope_append(qk, 0, bias[:used], rot, None, None, nq, nkv, d, d, ctx, view, v_from_k=True, gate_col=used)
+        row(f"bias, partial rotation, values from keys, gates, cache write, {tag}", run, bytes_=size(width) + 2 * T * (nq + 2 * nkv) * d + T * nq * 4)
+        row(f"bias, rotation, cache write (the Qwen2 model's), {tag}", lambda: kernels.rope_append(qkv, bias, rot, nq, nkv, d, ctx, view),
+            bytes_=size((nq + 2 * nkv) * d) + 2 * T * (nq + 2 * nkv) * d)
+        # attention over the window, alone and beside kept tokens
+        q, _back, gate = run()
+        for name, kw, seen in (("attention, window and kept first tokens, sink, gates", dict(window=size_, keep_first=keep, sink=sinks, head_gate=gate), size_ + keep),
+                               ("attention, window, sink (Radalix's kernels)", dict(window=size_, sink=sinks), size_),
+                               ("attention, plain window (the Qwen2 model's)", dict(window=size_), size_)):
+            kw = dict(kw)
+            win = kw.pop("window")
+            keys = batch * min(context, seen) if what == "decode" else sum(min(i, seen) for i in range(1, tokens + 1))
+            row(f"{name}, {what}", lambda: kernels.attention(q, nq, nkv, d, win, d ** -0.5, ctx, view, **kw),
+                bytes_=min(cached, R * seen) * nkv * 2 * d * 2 + 2 * T * nq * d * 2, flops=4 * nq * d * keys)
+        # latent attention
+        uk, uv = (torch.randn(AH * ldk, rank, device=dev) * 0.05).to(bf), (torch.randn(AH * ldv, rank, device=dev) * 0.05).to(bf)
+        lq, lw = (torch.randn(T, AH * (ldk + lrot), device=dev) * 0.3).to(bf), torch.ones(rank, device=dev)
+        down = torch.randn(T, -(-(rank + lrot + AH) // 8) * 8, device=dev).to(bf)
+        append = lambda col: kernels.latent_rope_append(down, 0, rank, lrot, lw, 1e-6, lq, AH, ldk, ltable, ctx, lview, vdim=ldv, gate_col=col)
+        for name, col in (("with gates", rank + lrot), ("(Benarax's)", None)):
+            row(f"latent row: norm, rotation, append {name}, {tag}", lambda: append(col), bytes_=T * (2 * (rank + lrot) * 2 + 2 * AH * lrot * 2))
+        queries, lgate = append(rank + lrot)
+        keys = batch * context if what == "decode" else tokens * (tokens + 1) // 2
+        for name, g in (("latent attention with gates", lgate), ("latent attention (Benarax's)", None)):
+            row(f"{name}, {what}", lambda: kernels.latent_attention(queries, uk, uv, None, AH, ldk, ldv, rank, None, 192 ** -0.5, ctx, lview, rot=lrot, head_gate=g),
+                bytes_=cached * (rank + lrot) * 2 + 2 * T * AH * (ldk + ldv) * 2 + AH * (ldk + ldv) * rank * 2,
+                flops=2 * AH * (2 * rank + lrot) * keys + 2 * T * AH * (ldk + ldv) * rank)
+        # lightning: activated columns, the scan, the gated norm over all heads
+        H, dk, dv = lig["heads"], lig["dim"], lig["vdim"]
+        K, V = H * dk, H * dv
+        rw = 2 * K + 2 * V
+        proj = mk(rw, f32)
+        rot_r = RotaryTable(torch.rand(dk // 2, device=dev), dk, False)
+        row(f"activated columns, {tag}", lambda: kernels.silu_columns(proj, 2 * K + V, ctx), bytes_=(size(rw, f32) + T * rw * 4) if splits else T * (2 * K + V) * 8)
+        row(f"turned columns (Vononex's), {tag}", lambda: kernels.rotate_rows(proj, 0, rw, H, dk, rot_r, 1.0, ctx),
+            bytes_=(size(rw, f32) + T * rw * 4) if splits else T * 2 * K * 8)
+        state, wide = torch.zeros(batch, H * dk * dv, device=dev), torch.randn(T, rw, device=dev) * 0.1
+        rate, raw = torch.full((H,), 0.99, device=dev), torch.randn(T, K, device=dev)
+        cut = (wide[:, :K], wide[:, K:2 * K], wide[:, 2 * K:2 * K + V])
+        row(f"scan, constant decay (also Vononex's), {tag}", lambda: kernels.decay_scan(*cut, None, state, ctx, heads=H, groups=H, dk=dk, dv=dv, decay="constant", rate=rate),
+            bytes_=2 * R * H * dk * dv * 4 + T * H * (2 * dk + 2 * dv) * 4)
+        row(f"scan, decay per key channel (Radalix's), {tag}", lambda: kernels.decay_scan(*cut, raw, state, ctx, heads=H, groups=H, dk=dk, dv=dv, decay="sigmoid_root", tau=16.0),
+            bytes_=2 * R * H * dk * dv * 4 + T * H * (3 * dk + 2 * dv) * 4)
+        o, wn = torch.randn(T, V, device=dev), torch.ones(V, device=dev)
+        row(f"norm over all heads, sigmoid gate, {tag}", lambda: kernels.gated_groupnorm(o, wide[:, 2 * K + V:], wn, 1e-6, 1, False, bf, kind="sigmoid"), bytes_=T * V * 10)
+        row(f"norm per head, SiLU gate (Vononex's), {tag}", lambda: kernels.gated_groupnorm(o, wide[:, 2 * K + V:], None, 1e-6, H, False, bf), bytes_=T * V * 10)
+        del cache, proj, wide
+        # sums and norms
+        x, wr, y1 = torch.randn(T, w, device=dev), torch.ones(w, device=dev), mk(w)
+        row(f"norm of the output, sum, next norm (also Dafolorn's), {tag}", lambda: kernels.postnorm_add(x, y1, wr, 1e-6, wr, 1e-6, bf), bytes_=size(w) + T * w * 10)
+        row(f"norm of a sum (Vononex's), {tag}", lambda: kernels.norm_of_sum(x, 2.0, [(1.0, y1, None)], wr, 1e-6, out_dtype=bf), bytes_=size(w) + T * w * 10)
+        # the feed-forward's first product
+        h = torch.randn(T, w, device=dev).to(bf)
+        up = (torch.randn(ff, w, device=dev) * 0.02).to(bf)
+        gu = (torch.randn(2 * (ff * 2 // 3), w, device=dev) * 0.02).to(bf)
+        cost = dict(bytes_=ff * w * 2 + T * (w + ff) * 2, flops=2 * T * ff * w)
+        row(f"squared-ReLU product, {tag}", lambda: kernels.linear_relu2(h, up), **cost)
+        row(f"xIELU product (Dafolorn's), {tag}", lambda: kernels.linear_xielu(h, up, 1.0, 1.0), **cost)
+        row(f"SiLU-gated product (the Qwen2 model's), {tag}", lambda: kernels.linear_swiglu(h, gu), bytes_=gu.numel() * 2 + T * (w + gu.shape[0] // 2) * 2,
+            flops=2 * T * gu.numel())
+        del up, gu
+    kernels.check_errors()
+    return out
+
+
+def run_design_sanarax(args, pk):
+    """`--design sanarax`: decode and prefill throughput of the design at real layer sizes beside Benarax (the closest model:
+    latent attention and a matrix-state scan, but mixtures of experts), Vononex (attention beside the same scan, dense
+    feed-forwards) and the Qwen2 shape at equal width, layer count and vocabulary, and its kernels beside the like kernels,
+    one JSON line."""
+    import torch
+    page, batch, context = 16, args.batch, min(args.context, 4096)
+    steps, warmup = max(1, args.steps), max(3, args.warmup)
+    result = {"metric": "decode and prefill tokens/s of another design beside the closest models at equal size",
+              "design": args.design, "dtype": "bf16", "n_gpus": 1, "data": "synthetic: random weights, uniform random token ids",
+              "batch": batch, "context": context, "prefill_tokens": PREFILL_TOKENS, "peaks": pk["source"], "shapes": {}}
+    makers = {"sanarax": (sanarax_config, sanarax_costs), "benarax": (benarax_config, benarax_costs), "vononex": (vononex_config, vononex_costs)}
+    kernels_table = None
+    for shape in ([args.shape] if args.shape in DESIGN_SHAPES and args.shape != "7b" else sorted(DESIGN_SHAPES)):
+        entry = {}
+        for name in ("sanarax", "benarax", "vononex", "qwen2"):
+            longest = context + 4 * (warmup + 3 * steps) + 16 + batch
+            if name == "qwen2":
+                cfg = qwen7b_config(DESIGN_SHAPES[shape]["qwen"])
+                cfg.num_hidden_layers = args.layers or cfg.num_hidden_layers
+                cfg.max_position_embeddings = max(cfg.max_position_embeddings, longest)
+            else:
+                cfg = makers[name][0](shape, args.layers)
+            engine = _engine(cfg, page, batch, longest)
+            r = time_decode(engine, cfg, batch, steps, warmup, repeats=3, context=context, e2e=False)
+            pre_ms = time_prefill(engine, cfg, PREFILL_TOKENS, warmup=2, reps=5)
+            if name == "qwen2":
+                step_bytes = weight_bytes(cfg, batch) + batch * r["ctx"] * kv_bytes_per_token(cfg)
+                flops = prefill_flops(cfg, PREFILL_TOKENS)
+            else:
+                step_bytes, flops = makers[name][1](cfg, batch, r["ctx"], PREFILL_TOKENS)
+            entry[name] = {"decode_tok_s": round(batch * 1000.0 / r["dev_ms"], 1), "decode_ms_per_step": round(r["dev_ms"], 3),
+                           "decode_hbm_frac": round(step_bytes / (r["dev_ms"] * 1e-3) / 1e9 / pk["hbm_gbs"], 3),
+                           "launches_per_step": round(r["launches"], 1),
+                           "prefill_tok_s": round(PREFILL_TOKENS * 1000.0 / pre_ms, 1), "prefill_ms": round(pre_ms, 2),
+                           "prefill_tensor_frac": round(flops / (pre_ms * 1e-3) / 1e12 / pk["bf16_tflops"], 3)}
+            if name == "sanarax" and kernels_table is None:
+                kernels_table = sanarax_kernels(engine.kernels, cfg, pk, batch, context, PREFILL_TOKENS)
+                entry["kernels"] = kernels_table
+            del engine
+            torch.cuda.empty_cache()
+        result["shapes"][shape] = entry
+    print(json.dumps(result))
+    return 0
+
+
 def _engine(cfg, page, slots, longest, pages=None, chunk=2048):
     import torch
     from inferflux_b200 import Engine
@@ -1542,7 +1779,7 @@ def main() -> int:
     ap.add_argument("--no-extras", action="store_true", help="skip the PyTorch baseline and the 1.5B-shape points")
     ap.add_argument("--prefill-only", action="store_true",
                     help="time only the 2,048-token prefill and print a short line (for profiling prefill)")
-    ap.add_argument("--design", default="", choices=["", "dafolorn", "zeluzen", "benarax", "radalix", "vononex"],
+    ap.add_argument("--design", default="", choices=["", "dafolorn", "zeluzen", "benarax", "radalix", "vononex", "sanarax"],
                     help="instead of the headline numbers: this design at real layer sizes beside the Qwen2 shape of equal "
                          "size (decode and prefill tokens/s, and its kernels beside the like kernels); --shape picks one size")
     args = ap.parse_args()
@@ -1558,6 +1795,8 @@ def main() -> int:
         return run_design_radalix(args, pk)
     if args.design == "vononex":
         return run_design_vononex(args, pk)
+    if args.design == "sanarax":
+        return run_design_sanarax(args, pk)
     if args.design:
         return run_design(args, pk)
     if args.gpus != 1:
