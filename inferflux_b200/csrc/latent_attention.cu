@@ -61,7 +61,8 @@ __global__ void latent_norm_append_kernel(const T* __restrict__ rows, int ld, in
 }
 
 // ------------------------------------------------- norm + rotation + append
-// One warp per token.  The cached row is [c; k_t]: c = x / rms(x) * w over `lat` columns starting at `col0` of `rows`,
+// A warp per token and stretch of `per` heads (blockIdx.y; the first stretch's also makes the cached row and the gates).  The
+// cached row is [c; k_t]: c = x / rms(x) * w over `lat` columns starting at `col0` of `rows`,
 // k_t the `rot` columns behind them turned by the token's position.  Every query head's last `rot` elements (heads of
 // dim + rot in `q`, rows ldq apart) are turned the same way and written to q_out (rows ld_out apart, heads head_stride
 // apart, at `out_offset` in a head): q itself, or the tail of a query in latent space.  The first `rot_used` of the
@@ -96,7 +97,7 @@ __global__ void latent_rope_append_kernel(const T* __restrict__ rows, int ld, in
                                           const int* __restrict__ req_slot, const int* __restrict__ block_table,
                                           int max_blocks, int page_size, int num_pages, T* __restrict__ pool,
                                           int num_tokens, int lat, int rot, int heads, int dim,
-                                          float* __restrict__ gate_out, int gate_col) {
+                                          float* __restrict__ gate_out, int gate_col, int per) {
   extern __shared__ float cs_s[];                        // per warp: cos and sin of the token's angles, then `rot` staged numbers
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -111,19 +112,19 @@ __global__ void latent_rope_append_kernel(const T* __restrict__ rows, int ld, in
     cs[i] = c * magnitude;
     cs[half + i] = sn * magnitude;
   }
-  if (gate_out != nullptr)
+  if (gate_out != nullptr && blockIdx.y == 0)
     for (int h = lane; h < heads; h += 32)
       gate_out[(size_t)t * heads + h] = 1.0f / (1.0f + expf(-to_f32(rows[(size_t)t * ld + gate_col + h])));
   __syncwarp();
   const T* x = rows + (size_t)t * ld + col0;
-  float ss = 0.0f;
-  for (int e = lane; e < lat; e += 32) {
-    const float v = to_f32(x[e]);
-    ss = fmaf(v, v, ss);
-  }
-  ss = warp_sum(ss);
-  const float r = rsqrtf(ss / (float)lat + eps);
-  if (pool != nullptr) {
+  if (pool != nullptr && blockIdx.y == 0) {
+    float ss = 0.0f;
+    for (int e = lane; e < lat; e += 32) {
+      const float v = to_f32(x[e]);
+      ss = fmaf(v, v, ss);
+    }
+    ss = warp_sum(ss);
+    const float r = rsqrtf(ss / (float)lat + eps);
     const int slot = req_slot[token_req[t]];
     const int page = block_table[(size_t)slot * max_blocks + pos / page_size];
     if (page >= 0 && page < num_pages) {
@@ -132,7 +133,7 @@ __global__ void latent_rope_append_kernel(const T* __restrict__ rows, int ld, in
       turn_store(x + lat, dst + lat, rot, rot_used, interleaved, cs, held, lane);
     }
   }
-  for (int h = 0; h < heads; ++h)
+  for (int h = blockIdx.y * per; h < min(heads, (int)(blockIdx.y + 1) * per); ++h)
     turn_store(q + (size_t)t * ldq + (size_t)h * (dim + rot) + dim, q_out + (size_t)t * ld_out + (size_t)h * head_stride + out_offset,
                rot, rot_used, interleaved, cs, held, lane);
 }
@@ -297,16 +298,20 @@ int ifx_latent_rope_append(const void* rows, int ld, int col0, const float* w, f
   const int warps = 4;
   const unsigned blocks = (unsigned)((T + warps - 1) / warps);
   const size_t smem = (size_t)warps * (rot_used + rot + 1) * sizeof(float);
+  // few tokens: a warp a head; many: as many heads a warp as still give every SM a few blocks (a warp works out its angles)
+  int per = 1;
+  while (per < 8 && per < heads && (long long)blocks * ((heads + 2 * per - 1) / (2 * per)) >= 148 * 8) per *= 2;
+  const dim3 grid(blocks, rot > 0 ? (unsigned)((heads + per - 1) / per) : 1u);
   if (dtype == IFX_DT_F32)
-    latent_rope_append_kernel<float><<<blocks, warps * 32, smem, stream>>>(
+    latent_rope_append_kernel<float><<<grid, warps * 32, smem, stream>>>(
         (const float*)rows, ld, col0, w, eps, (const float*)q, ldq, (float*)q_out, ld_out, head_stride, out_offset, inv_freq,
         rot_used, interleaved, magnitude, positions, token_req, req_slot, block_table, max_blocks, page_size, num_pages,
-        (float*)pool, T, lat, rot, heads, dim, gate_out, gate_col);
+        (float*)pool, T, lat, rot, heads, dim, gate_out, gate_col, per);
   else if (dtype == IFX_DT_BF16)
-    latent_rope_append_kernel<__nv_bfloat16><<<blocks, warps * 32, smem, stream>>>(
+    latent_rope_append_kernel<__nv_bfloat16><<<grid, warps * 32, smem, stream>>>(
         (const __nv_bfloat16*)rows, ld, col0, w, eps, (const __nv_bfloat16*)q, ldq, (__nv_bfloat16*)q_out, ld_out,
         head_stride, out_offset, inv_freq, rot_used, interleaved, magnitude, positions, token_req, req_slot, block_table,
-        max_blocks, page_size, num_pages, (__nv_bfloat16*)pool, T, lat, rot, heads, dim, gate_out, gate_col);
+        max_blocks, page_size, num_pages, (__nv_bfloat16*)pool, T, lat, rot, heads, dim, gate_out, gate_col, per);
   else return IFX_E_DTYPE;
   IFX_CHECK_LAUNCH();
   return 0;
