@@ -616,7 +616,8 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kv_pool,
 // padding: ldmatrix reads the swizzled tiles without bank conflicts.  Keys of a tile
 // beyond the token's range get zero weight; what the page holds there is finite (the
 // pool starts as zeros and only finite values are ever written to it).
-template <int D, int STAGES, int WARPS>
+// KEPT: the mask has kept first keys.
+template <int D, int STAGES, int WARPS, bool KEPT>
 __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16* __restrict__ q,
                        const int* __restrict__ block_table, const int4* __restrict__ decode_meta,
@@ -659,16 +660,16 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
   const int* table = table_g;
   int blk_base = 0;
 
-  // Tiles start on multiples of 16 so that one lies in one page.  They are counted without the gap between the keys that
-  // stay visible and the window: index i is key i for i < kept, else key i + gap (kept and gap are multiples of 16).
+  // Tiles start on multiples of 16 so that one lies in one page.  With kept keys they are counted from 0 on without the gap
+  // between those and the window: index i is key i for i < kept, else key i + gap (both multiples of 16).
   const int kfirst = window.first(pos);
   const int kstart = kfirst & ~15;
-  const int kept = min((window.keep + 15) & ~15, kstart), gap = kstart - kept;
-  const int kend = pos + 1 - gap;
-  const int per_split = (((kend + num_splits - 1) / num_splits) + WARPS * 16 - 1) / (WARPS * 16) * (WARPS * 16);
-  const int k0 = split * per_split;
+  const int kept = KEPT ? min((window.keep + 15) & ~15, kstart) : 0, gap = KEPT ? kstart - kept : 0;
+  const int kbegin = KEPT ? 0 : kstart, kend = pos + 1 - gap;
+  const int per_split = (((kend - kbegin + num_splits - 1) / num_splits) + WARPS * 16 - 1) / (WARPS * 16) * (WARPS * 16);
+  const int k0 = kbegin + split * per_split;
   const int k1 = min(kend, k0 + per_split);
-  if (k0 < k1 && k1 > kept) {
+  if (k0 < k1 && (!KEPT || k1 > kept)) {
     const int b0 = (max(k0, kept) + gap) >> page_shift, b1 = (k1 - 1 + gap) >> page_shift;
     if (b1 - b0 + 1 <= tbl_cap) {
       for (int i = tid; i <= b1 - b0; i += THREADS) tbl_s[i] = table_g[b0 + i];
@@ -681,8 +682,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
   const uint32_t my_stage0 = smem_addr(stage_base) + warp * STAGES * STAGE_BYTES;
   const uint32_t my_bar0 = smem_addr(bars + warp * STAGES);
   auto issue_tile = [&](int base, int stage) {           // lane 0 only: the 16 keys from index `base` on
-    const int key0 = base < kept ? base : base + gap, blk = key0 >> page_shift;
-    int page = blk >= blk_base ? table[blk - blk_base] : table_g[blk];
+    const int key0 = KEPT && base < kept ? base : base + gap, blk = key0 >> page_shift;
+    int page = !KEPT || blk >= blk_base ? table[blk - blk_base] : table_g[blk];
     if (page < 0 || page >= num_pages) page = 0;
     const int off = key0 & (page_size - 1);
     const int yk = ((page * 2) * nkv + g) * page_size + off;
@@ -764,8 +765,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
     for (int n = 0; n < 2; ++n) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int idx = base + n * 8 + 2 * (lane & 3) + (e & 1), key = idx < kept ? idx : idx + gap;
-        s[n][e] = (idx < k1 && window.sees(key, kfirst)) ? s[n][e] * scale_log2 : -INFINITY;
+        const int idx = base + n * 8 + 2 * (lane & 3) + (e & 1), key = KEPT && idx < kept ? idx : idx + gap;
+        s[n][e] = (idx < k1 && (key >= kfirst || (KEPT && key < window.keep))) ? s[n][e] * scale_log2 : -INFINITY;
       }
       mx_lo = fmaxf(mx_lo, fmaxf(s[n][0], s[n][1]));
       mx_hi = fmaxf(mx_hi, fmaxf(s[n][2], s[n][3]));
@@ -933,7 +934,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap pool_map, const bf16*
   cluster.sync();
 }
 
-template <int D, int STAGES, int WARPS>
+template <int D, int STAGES, int WARPS, bool KEPT>
 int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const int* block_table, const int4* decode_meta,
                              bf16* out, int num_items, int nq, int nkv, int page_size, int page_shift, int max_blocks,
                              int num_pages, KeyMask window, HeadOutput post, float scale_log2, int num_splits, int max_keys, int* error_flag,
@@ -949,7 +950,7 @@ int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const i
   const int smem = 1024 + work_bytes + 16 * (D + 8) * 2 + WARPS * STAGES * 8 + tbl_cap * 4;
   static int configured = 0;
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_tma_kernel<D, STAGES, WARPS>,
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_tma_kernel<D, STAGES, WARPS, KEPT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
@@ -957,13 +958,13 @@ int launch_decode_tma_stages(const CUtensorMap& pool_map, const bf16* q, const i
   if (num_splits > 8) {                                   // a cluster of 16 is beyond the portable size
     static bool allowed = false;
     if (!allowed) {
-      cudaError_t e = cudaFuncSetAttribute(attn_decode_tma_kernel<D, STAGES, WARPS>,
+      cudaError_t e = cudaFuncSetAttribute(attn_decode_tma_kernel<D, STAGES, WARPS, KEPT>,
                                            cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
       if (e != cudaSuccess) return (int)e;
       allowed = true;
     }
   }
-  return launch_pdl(attn_decode_tma_kernel<D, STAGES, WARPS>, dim3(num_items, nkv, num_splits), dim3(WARPS * 32),
+  return launch_pdl(attn_decode_tma_kernel<D, STAGES, WARPS, KEPT>, dim3(num_items, nkv, num_splits), dim3(WARPS * 32),
                     (size_t)smem, stream, num_splits, pool_map, q, block_table, decode_meta, out, nq, nkv, page_size,
                     page_shift, max_blocks, num_pages, window, post, scale_log2, tbl_cap, error_flag);
 }
@@ -984,8 +985,10 @@ int launch_decode_tma(const CUtensorMap& pool_map, const bf16* q, const int* blo
   const int keys_per_block = max_keys / (num_splits > 0 ? num_splits : 1);
 #define ARGS pool_map, q, block_table, decode_meta, out, num_items, nq, nkv, page_size, page_shift, max_blocks, num_pages, \
              window, post, scale_log2, num_splits, max_keys, error_flag, stream
-  if (D <= 128 && blocks <= 104 && keys_per_block >= 8 * 16) return launch_decode_tma_stages<D, STAGES, 8>(ARGS);
-  return launch_decode_tma_stages<D, STAGES, 4>(ARGS);
+  const bool eight = D <= 128 && blocks <= 104 && keys_per_block >= 8 * 16;
+  if (window.keep > 0)
+    return eight ? launch_decode_tma_stages<D, STAGES, 8, true>(ARGS) : launch_decode_tma_stages<D, STAGES, 4, true>(ARGS);
+  return eight ? launch_decode_tma_stages<D, STAGES, 8, false>(ARGS) : launch_decode_tma_stages<D, STAGES, 4, false>(ARGS);
 #undef ARGS
 }
 

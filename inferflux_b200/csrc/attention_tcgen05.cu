@@ -128,7 +128,8 @@ struct PrefillLayout {
   static constexpr size_t SMEM = 1024 + 2 * Q_BYTES + (size_t)SLOTS * SLOT_BYTES + B_COUNT * 8 + 16;
 };
 
-template <int D>
+// KEPT: the mask has kept first keys (without them the walk over the key tiles is a plain range).
+template <int D, bool KEPT>
 __global__ void __launch_bounds__(kThreads)
 attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap pool_map,
                             const int* __restrict__ block_table, const int* __restrict__ tiles,
@@ -185,16 +186,17 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
   const int tb_0 = window.first(pos0) / kBN;
   const int te_0 = (pos0 + min(rows, kBM) + kBN - 1) / kBN;
   const int tb_1 = window.first(pos0 + kBM) / kBN;
-  const int te_1 = rows_1 > 0 ? (pos0 + rows + kBN - 1) / kBN : 0;
+  const int te_1 = rows_1 > 0 ? (pos0 + rows + kBN - 1) / kBN : tb_1;
   const int te = max(te_0, te_1);
-  // Key tiles in the order they are visited, counted without a gap: [0, nk) with the keys that stay visible in front of the
-  // windows, then [tb_0, te).  Query tile q uses those that hold kept keys and those of its own window.
-  const int keep_tiles = (window.keep + kBN - 1) / kBN, nk = min(keep_tiles, tb_0), tile_gap = tb_0 - nk;
-  const int num_kt = te - tile_gap;
-  auto tile_at = [&](int i) { return i < nk ? i : i + tile_gap; };
-  auto active = [&](int q, int i) {
-    const int kt = tile_at(i);
-    return kt < (q == 0 ? te_0 : te_1) && (kt < keep_tiles || kt >= (q == 0 ? tb_0 : tb_1));
+  // Key tiles are visited in order: with kept keys first [0, nk), then [tb_0, te); query tile q uses those that hold kept keys
+  // and those of its own window.
+  const int keep = KEPT ? window.keep : 0, keep_tiles = (keep + kBN - 1) / kBN, nk = min(keep_tiles, tb_0);
+  const int tb = KEPT && nk > 0 ? 0 : tb_0;
+  auto next_tile = [&](int kt) { return KEPT && kt + 1 == nk ? tb_0 : kt + 1; };
+  auto visited = [&](int kt) { return KEPT && kt < nk ? kt : kt - tb_0 + nk; };          // how many tiles come before kt
+  auto active = [&](int q, int kt) {
+    if (KEPT && kt < keep_tiles && kt < te_0 && (q == 0 || rows_1 > 0)) return true;      // (kept keys lie in front of te_0)
+    return q == 0 ? (kt >= tb_0 && kt < te_0) : (kt >= tb_1 && kt < te_1);
   };
   const int kfirst = window.first(pos0), kend = pos0 + rows;
 
@@ -210,20 +212,19 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     }
     bool ok = true;
     int issued = 0;                                       // slots filled so far
-    for (int i = 0; i < num_kt && ok; ++i) {
-      const int kt = tile_at(i);
+    for (int kt = tb; kt < te && ok; kt = next_tile(kt)) {
       // lanes 0-7 take one 16-key block each; its page is looked up before the wait for a free slot
       const int key = kt * kBN + lane * 16;
       int page = 0, off = 0;
       // no visible key among the 16: any valid page, its keys get weight zero
-      if (lane < kBN / 16 && key < kend && (key + 16 > kfirst || key < window.keep)) {
+      if (lane < kBN / 16 && key < kend && (key + 16 > kfirst || key < keep)) {
         page = table[key >> page_shift];
         if (page < 0 || page >= num_pages) page = 0;
         off = key & (page_size - 1);
       }
 #pragma unroll 1
       for (int kv = 0; kv < 2; ++kv) {                     // the keys, then the values
-        const int j = 2 * i + kv, s = j % SLOTS;
+        const int j = 2 * visited(kt) + kv, s = j % SLOTS;
         ok = __all_sync(0xffffffffu, mbar_wait(bar(L::B_EMPTY + s), ((j / SLOTS) & 1) ^ 1));
         if (!ok) break;
         const uint32_t fb = bar(L::B_FULL + s);
@@ -250,10 +251,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                                ((uint32_t)(kBM >> 4) << 24);                       // both operands K-major
       const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(D >> 3) << 17) |
                                ((uint32_t)(kBM >> 4) << 24);                       // B (values) MN-major
-      auto last_q = [&](int i) { return active(1, i) ? 1 : 0; };      // the query tile that uses a key tile last
+      auto last_q = [&](int kt) { return active(1, kt) ? 1 : 0; };    // the query tile that uses a key tile last
       bool ok = mbar_wait(bar(L::B_Q), 0);
-      auto issue_s = [&](int q, int i) -> bool {          // S_q = Q_q . K^T with the i-th key tile
-        const int j = 2 * i, s = j % SLOTS;
+      auto issue_s = [&](int q, int kt) -> bool {         // S_q = Q_q . K(kt)^T
+        const int j = 2 * visited(kt), s = j % SLOTS;
         if (!mbar_wait(bar(L::B_FULL + s), (j / SLOTS) & 1)) return false;
         tc_fence_after();
         const uint32_t k_src = kv_s + s * SLOT_BYTES, q_src = q_s + q * Q_BYTES;
@@ -264,12 +265,12 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     desc_kmajor_sw128(k_src + half * kBN * 128) + (inner >> 4), idesc_s, k > 0 ? 1u : 0u);
         }
         umma_commit(bar(L::B_S_FULL + q));
-        if (q == last_q(i)) umma_commit(bar(L::B_EMPTY + s));       // the keys have been read
+        if (q == last_q(kt)) umma_commit(bar(L::B_EMPTY + s));      // the keys have been read
         return true;
       };
       int done[2] = {0, 0};                                // key tiles of each query tile so far
-      auto issue_pv = [&](int q, int i) -> bool {         // O_q += P_q . V with the i-th key tile
-        const int j = 2 * i + 1, s = j % SLOTS;
+      auto issue_pv = [&](int q, int kt) -> bool {        // O_q += P_q . V(kt)
+        const int j = 2 * visited(kt) + 1, s = j % SLOTS;
         if (!mbar_wait(bar(L::B_P_FULL + q), done[q] & 1) || !mbar_wait(bar(L::B_FULL + s), (j / SLOTS) & 1))
           return false;
         tc_fence_after();
@@ -279,20 +280,21 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
           umma_bf16_ts(tmem_o + q * D, tmem_s + q * kBN + k * 8, desc_mnmajor_sw128(v_src + k * 2048, kBN * 128),
                        idesc_o, (done[q] > 0 || k > 0) ? 1u : 0u);
         umma_commit(bar(L::B_O_FULL + q));
-        if (q == last_q(i)) umma_commit(bar(L::B_EMPTY + s));       // the values have been read
+        if (q == last_q(kt)) umma_commit(bar(L::B_EMPTY + s));      // the values have been read
         ++done[q];
         return true;
       };
       for (int q = 0; q < 2 && ok; ++q)
-        if (active(q, 0)) ok = issue_s(q, 0);
-      for (int i = 0; i < num_kt && ok; ++i) {
+        if (active(q, tb)) ok = issue_s(q, tb);
+      for (int kt = tb, before = tb; kt < te && ok; before = kt, kt = next_tile(kt)) {
         for (int q = 0; q < 2 && ok; ++q) {
-          if (!active(q, i)) continue;
-          if (i > 0 && !active(q, i - 1)) ok = issue_s(q, i);         // a query tile that starts, or goes on, later (window)
-          if (ok) ok = issue_pv(q, i);
+          if (!active(q, kt)) continue;
+          // a query tile that starts, or behind the kept keys goes on, later (window)
+          if (kt != tb && (KEPT ? !active(q, before) : kt == (q == 0 ? tb_0 : tb_1))) ok = issue_s(q, kt);
+          if (ok) ok = issue_pv(q, kt);
           // the next scores of this query tile go over its probabilities: the product that reads them
           // was issued just before and runs first; meanwhile the other tile's softmax is at work
-          if (ok && i + 1 < num_kt && active(q, i + 1)) ok = issue_s(q, i + 1);
+          if (ok && active(q, next_tile(kt))) ok = issue_s(q, next_tile(kt));
         }
       }
       if (!ok) atomicExch(error_flag, 8);
@@ -312,14 +314,14 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     float m_ref = -INFINITY, l_run = 0.0f;
     bool ok = true;
     int i = 0;                                            // key tiles of this query tile so far
-    for (int n = 0; n < num_kt; ++n) {
-      if (!active(q, n)) continue;
-      const int key0 = tile_at(n) * kBN;
+    for (int kt = KEPT ? tb : (q == 0 ? tb_0 : tb_1); kt < (KEPT ? te : (q == 0 ? te_0 : te_1)); kt = next_tile(kt)) {
+      if (KEPT && !active(q, kt)) continue;
+      const int key0 = kt * kBN;
       ok = __all_sync(0xffffffffu, mbar_wait(bar(L::B_S_FULL + q), i & 1));
       if (!ok) break;
       tc_fence_after();
       const bool edge = key0 + kBN - 1 > pos0_q ||
-                        (window.any() && key0 < window.first(pos0_q + kBM - 1) && key0 + kBN > window.keep);
+                        (window.any() && key0 < window.first(pos0_q + kBM - 1) && (!KEPT || key0 + kBN > keep));
       // pass 1: the row's maximum
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -332,7 +334,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 #pragma unroll
           for (int j = 0; j < 64; ++j) {
             const int key = key0 + c + j;
-            if (key > pos || !window.sees(key, wfirst)) s[j] = -INFINITY;
+            if (key > pos || (key < wfirst && (!KEPT || key >= keep))) s[j] = -INFINITY;
           }
         }
 #pragma unroll
@@ -378,7 +380,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 #pragma unroll
           for (int j = 0; j < 64; ++j) {
             const int key = key0 + c + j;
-            if (key > pos || !window.sees(key, wfirst)) s[j] = -INFINITY;
+            if (key > pos || (key < wfirst && (!KEPT || key >= keep))) s[j] = -INFINITY;
           }
         }
         uint32_t packed[32];
@@ -476,7 +478,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
   }
 }
 
-template <int D>
+template <int D, bool KEPT>
 static int launch_prefill_tcgen05(const bf16* q, int num_tokens, const bf16* kv_pool, const int* block_table,
                                   const int* tiles, const int* req_slot, bf16* out, int num_tiles, int nq, int nkv,
                                   int page_size, int page_shift, int max_blocks, int num_pages, KeyMask window, HeadOutput post,
@@ -489,12 +491,12 @@ static int launch_prefill_tcgen05(const bf16* q, int num_tokens, const bf16* kv_
   const size_t smem = PrefillLayout<D>::SMEM;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<D, KEPT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  return launch_pdl(attn_prefill_tcgen05_kernel<D>, dim3(nq, num_tiles), dim3(kThreads), smem, stream, 1, q_map,
+  return launch_pdl(attn_prefill_tcgen05_kernel<D, KEPT>, dim3(nq, num_tiles), dim3(kThreads), smem, stream, 1, q_map,
                     pool_map, block_table, tiles, req_slot, out, nq, nkv, page_size, page_shift, max_blocks,
                     num_pages, window, post, scale_log2, error_flag);
 }
@@ -530,13 +532,12 @@ int ifx_attention_prefill_tcgen05_sink(const void* q, int num_tokens, const void
   int ps = 0;
   while ((1 << ps) < page_size) ++ps;
   const float scale_log2 = scale * 1.4426950408889634f;
-  if (d == 64)
-    return launch_prefill_tcgen05<64>((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot,
-                                      (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, post,
-                                      scale_log2, error_flag, stream);
-  return launch_prefill_tcgen05<128>((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot,
-                                     (bf16*)out, num_tiles, nq, nkv, page_size, ps, max_blocks, num_pages, window, post,
-                                     scale_log2, error_flag, stream);
+  auto run = [&](auto launch) {
+    return launch((const bf16*)q, num_tokens, (const bf16*)kv_pool, block_table, tiles, req_slot, (bf16*)out, num_tiles, nq, nkv,
+                  page_size, ps, max_blocks, num_pages, window, post, scale_log2, error_flag, stream);
+  };
+  if (d == 64) return keep_first > 0 ? run(launch_prefill_tcgen05<64, true>) : run(launch_prefill_tcgen05<64, false>);
+  return keep_first > 0 ? run(launch_prefill_tcgen05<128, true>) : run(launch_prefill_tcgen05<128, false>);
 }
 
 int ifx_attention_prefill_tcgen05_ex(const void* q, int num_tokens, const void* kv_pool, const int* block_table,
