@@ -309,7 +309,7 @@ def _check(name, dtype, got, o):
         top = max(float(np.abs(v).max()) for v in o["float32"].values())
         bad = helpers.first_bad(got, o["float32"], 3e-4 + 1e-5 * top)
         assert bad is None, f"{name}: first wrong row (request, position, diff): {bad}"
-    else:                                                  # all rows together: a request of one token has one row to judge by
+    else:                                                  # all rows together: a request of one token has only one row
         rids = list(o["reqs"])
         _bf16_close(name, *(np.concatenate([x[r] for r in rids]) for x in (got, o["bfloat16"], o["yard"])))
 
